@@ -1,0 +1,385 @@
+// Shared pieces of the dense-weight library (bf16 or fp32 weights [N, K], K contiguous): element access, the row
+// preparation that precedes a projection, and the epilogues that follow one.
+//
+// Programmatic dependent launch: every kernel here calls pdl_trigger() AFTER its own pdl_wait().  A kernel can therefore
+// only start once everything two launches back has completed, and may read such data (positions, older cache rows,
+// weights) ahead of its own pdl_wait(); what its direct predecessor wrote is read after it, through L2 (__ldcg), because a
+// line may have been cached in L1 before the predecessor wrote it.
+#pragma once
+
+#include <utility>
+
+#include <cuda_bf16.h>
+
+#include "../common.cuh"
+#include "../../../include/dense_b200.h"
+
+namespace gptq {
+
+typedef __nv_bfloat16 bf16;
+
+constexpr int DN_THREADS = 256;
+constexpr int DN_WARPS = DN_THREADS / 32;
+constexpr int DN_STATUS_SLOT = DENSE_CONTROL_BYTES / 4 - 1;      // same place as in the other library's workspaces
+constexpr int DN_BAD_POSITION = 4;                                // status value: position outside the tables / the cache
+
+template <typename T> struct Elem;
+template <> struct Elem<bf16> {
+	static __device__ __forceinline__ float4 load4(const bf16 *p) {
+		const uint2 v = __ldg(reinterpret_cast<const uint2 *>(p));
+		return unpack(v);
+	}
+	static __device__ __forceinline__ float4 unpack(uint2 v) {
+		return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
+	}
+	static __device__ __forceinline__ void store4(bf16 *p, float4 v) {
+		__nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+		uint2 o;
+		o.x = *reinterpret_cast<uint32_t *>(&a);
+		o.y = *reinterpret_cast<uint32_t *>(&b);
+		*reinterpret_cast<uint2 *>(p) = o;
+	}
+	static __device__ __forceinline__ float ldcg(const bf16 *p) {
+		return __uint_as_float((uint32_t)__ldcg(reinterpret_cast<const unsigned short *>(p)) << 16);
+	}
+	static __device__ __forceinline__ void store(bf16 *p, float v) { *p = __float2bfloat16_rn(v); }
+};
+template <> struct Elem<float> {
+	static __device__ __forceinline__ float4 load4(const float *p) { return __ldg(reinterpret_cast<const float4 *>(p)); }
+	static __device__ __forceinline__ void store4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+	static __device__ __forceinline__ float ldcg(const float *p) { return __ldcg(p); }
+	static __device__ __forceinline__ void store(float *p, float v) { *p = v; }
+};
+
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+	__nv_bfloat162 a = __floats2bfloat162_rn(lo, hi);
+	return *reinterpret_cast<uint32_t *>(&a);
+}
+
+// D(16x8) += A(16x16, row) * B(16x8, col), bf16 operands; fragment ownership as in mma16816
+__device__ __forceinline__ void mma16816_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+	asm volatile(
+		"mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+		: "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+		: "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
+	asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldmatrix_x2(uint32_t (&r)[2], uint32_t addr) {
+	asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldmatrix_x2_trans(uint32_t (&r)[2], uint32_t addr) {
+	asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
+}
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+	for (int d = 16; d > 0; d >>= 1) v += __shfl_xor_sync(0xffffffffu, v, d);
+	return v;
+}
+__device__ __forceinline__ float warp_max(float v) {
+#pragma unroll
+	for (int d = 16; d > 0; d >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, d));
+	return v;
+}
+
+// Sum over the 256 threads of the CTA; `slot` (DN_WARPS floats of shared memory) must not be in use by an earlier call.
+__device__ __forceinline__ float block_sum(float v, float *slot) {
+	v = warp_sum(v);
+	if ((threadIdx.x & 31) == 0) slot[threadIdx.x >> 5] = v;
+	__syncthreads();
+	float t = 0.f;
+#pragma unroll
+	for (int i = 0; i < DN_WARPS; ++i) t += slot[i];
+	return t;
+}
+
+__device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
+
+// ---- row preparation ------------------------------------------------------------------------------------------------
+// Forms row m of the residual stream and the normalised or plain row that the next projection reads, all in fp32:
+//   x = table[token]                                      (start of a step), or
+//   x = x_in + (y - mean(y)) / sqrt(var(y) + eps) * gain + shift      (post-norm residual; gain and shift carry the
+//                                                          norm's affine part, the layer scale and the residual multiplier)
+//   out = x, or LayerNorm(x) * fin_w + fin_b               (final norm)
+// Rows are padded with zeros from `width` to `ld` columns.
+using RowPrep = dense_rows_t;
+
+constexpr int RP_REGS = 4;              // float4 units of a row that a thread keeps in registers
+
+template <typename T>
+__device__ __forceinline__ float4 rp_x(const RowPrep &p, size_t base, int u) {
+	if (p.table) return Elem<T>::load4(reinterpret_cast<const T *>(p.table) + base + 4 * u);
+	return __ldcg(reinterpret_cast<const float4 *>(p.x_in + base) + u);
+}
+__device__ __forceinline__ float rp_sqdev(float4 v, float mean, int c, int width) {
+	float s = 0.f;
+	const float a = v.x - mean, b = v.y - mean, d = v.z - mean, e = v.w - mean;
+	if (c < width) s = fmaf(a, a, s);
+	if (c + 1 < width) s = fmaf(b, b, s);
+	if (c + 2 < width) s = fmaf(d, d, s);
+	if (c + 3 < width) s = fmaf(e, e, s);
+	return s;
+}
+__device__ __forceinline__ float4 rp_affine(float4 x, float4 y, float mean, float inv, float4 g, float4 s) {
+	return make_float4(x.x + fmaf((y.x - mean) * inv, g.x, s.x), x.y + fmaf((y.y - mean) * inv, g.y, s.y), x.z + fmaf((y.z - mean) * inv, g.z, s.z),
+					   x.w + fmaf((y.w - mean) * inv, g.w, s.w));
+}
+
+// The whole CTA (256 threads) prepares one row.  dst: where the T row goes (global or shared memory); write_x: also store
+// the new residual row.  red: 4 * DN_WARPS floats of shared memory, reused across rows (callers synchronise between rows).
+template <typename T>
+__device__ void prepare_row(const RowPrep &p, int m, T *dst, bool write_x, float *red) {
+	const int tid = threadIdx.x, nu = p.ld >> 2;
+	size_t xb = (size_t)m * p.ld;
+	const size_t yb = xb;
+	if (p.table) {
+		long long t = __ldcg(reinterpret_cast<const long long *>(p.token) + m);
+		if (t < 0 || t >= p.vocab) {          // never index the table out of range
+			if (tid == 0) atomicExch(p.status, DN_BAD_POSITION);
+			t = 0;
+		}
+		xb = (size_t)t * p.ld;
+	}
+	float4 x[RP_REGS], y[RP_REGS];
+	const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+	for (int i = 0; i < RP_REGS; ++i) {
+		const int u = tid + i * DN_THREADS;
+		x[i] = u < nu ? rp_x<T>(p, xb, u) : zero;
+		y[i] = (p.y && u < nu) ? __ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u) : zero;
+	}
+	const float inv_n = 1.f / (float)p.width;
+	float mean = 0.f, inv = 0.f;
+	if (p.y) {
+		float s = 0.f;
+#pragma unroll
+		for (int i = 0; i < RP_REGS; ++i) s += (y[i].x + y[i].y) + (y[i].z + y[i].w);
+		for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) {
+			const float4 v = __ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u);
+			s += (v.x + v.y) + (v.z + v.w);
+		}
+		mean = block_sum(s, red) * inv_n;
+		s = 0.f;
+#pragma unroll
+		for (int i = 0; i < RP_REGS; ++i) s += rp_sqdev(y[i], mean, 4 * (tid + i * DN_THREADS), p.width);
+		for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS)
+			s += rp_sqdev(__ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u), mean, 4 * u, p.width);
+		inv = 1.f / sqrtf(block_sum(s, red + DN_WARPS) * inv_n + p.eps);
+	}
+	auto next_x = [&](float4 xv, float4 yv, int u) {
+		if (!p.y) return xv;
+		return rp_affine(xv, yv, mean, inv, __ldg(reinterpret_cast<const float4 *>(p.gain) + u), __ldg(reinterpret_cast<const float4 *>(p.shift) + u));
+	};
+#pragma unroll
+	for (int i = 0; i < RP_REGS; ++i) {
+		const int u = tid + i * DN_THREADS;
+		if (u < nu) {
+			x[i] = next_x(x[i], y[i], u);
+			if (write_x) reinterpret_cast<float4 *>(p.x_out + yb)[u] = x[i];
+			if (!p.fin_w) Elem<T>::store4(dst + 4 * u, x[i]);
+		}
+	}
+	auto far_x = [&](int u) {          // units beyond the registers are formed again where they are needed
+		return next_x(rp_x<T>(p, xb, u), p.y ? __ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u) : zero, u);
+	};
+	if (!p.fin_w) {
+		for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) {
+			const float4 v = far_x(u);
+			if (write_x) reinterpret_cast<float4 *>(p.x_out + yb)[u] = v;
+			Elem<T>::store4(dst + 4 * u, v);
+		}
+		return;
+	}
+	// final norm over the new row (x_out must not be x_in when rows are longer than the registers hold: the row is read again)
+	float s = 0.f;
+#pragma unroll
+	for (int i = 0; i < RP_REGS; ++i) s += (x[i].x + x[i].y) + (x[i].z + x[i].w);
+	for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) {
+		const float4 v = far_x(u);
+		s += (v.x + v.y) + (v.z + v.w);
+	}
+	const float fm = block_sum(s, red + 2 * DN_WARPS) * inv_n;
+	s = 0.f;
+#pragma unroll
+	for (int i = 0; i < RP_REGS; ++i) s += rp_sqdev(x[i], fm, 4 * (tid + i * DN_THREADS), p.width);
+	for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) s += rp_sqdev(far_x(u), fm, 4 * u, p.width);
+	const float fi = 1.f / sqrtf(block_sum(s, red + 3 * DN_WARPS) * inv_n + p.eps);
+	for (int i = 0, u = tid; u < nu; ++i, u += DN_THREADS) {
+		float4 v;
+		if (i < RP_REGS) {
+			v = i == 0 ? x[0] : i == 1 ? x[1] : i == 2 ? x[2] : x[3];
+		} else {
+			v = far_x(u);
+			if (write_x) reinterpret_cast<float4 *>(p.x_out + yb)[u] = v;
+		}
+		const float4 w = __ldg(reinterpret_cast<const float4 *>(p.fin_w) + u), b = __ldg(reinterpret_cast<const float4 *>(p.fin_b) + u);
+		Elem<T>::store4(dst + 4 * u, make_float4(fmaf((v.x - fm) * fi, w.x, b.x), fmaf((v.y - fm) * fi, w.y, b.y), fmaf((v.z - fm) * fi, w.z, b.z),
+												 fmaf((v.w - fm) * fi, w.w, b.w)));
+	}
+}
+
+// ---- epilogues ------------------------------------------------------------------------------------------------------
+// Every fp32 result of a projection belongs to a pair of columns (n, n + 1), n even (SILU: gate column and up column).
+using DenseEpi = dense_epilogue_t;
+
+__device__ __forceinline__ int epi_pos(const DenseEpi &e, int m) {
+	int pos = __ldcg(e.pos + m);
+	if (pos < 0 || pos >= e.max_pos) {
+		atomicExch(e.status, DN_BAD_POSITION);
+		pos = 0;
+	}
+	return pos;
+}
+
+// One pair of results of row m.  T is the activation type.
+template <typename T>
+__device__ __forceinline__ void epi_pair(const DenseEpi &e, int m, int n, float a, float b) {
+	switch (e.mode) {
+		case DENSE_EPI_F32:
+		case DENSE_EPI_LOGITS:
+			*reinterpret_cast<float2 *>(reinterpret_cast<float *>(e.out) + (size_t)m * e.ldo + n) = make_float2(a * e.scale, b * e.scale);
+			break;
+		case DENSE_EPI_T: {
+			T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
+			Elem<T>::store(o, a);
+			Elem<T>::store(o + 1, b);
+			break;
+		}
+		case DENSE_EPI_QKV: {
+			if (n < e.n_q) {
+				const int off = n % e.head_dim - e.rot_at;
+				if (off >= 0 && off < e.rot_dims) {
+					const size_t t = (size_t)epi_pos(e, m) * (e.rot_dims >> 1) + (off >> 1);
+					const float c = __ldg(e.cos_t + t), s = __ldg(e.sin_t + t);
+					const float u = a * c - b * s;
+					b = b * c + a * s;
+					a = u;
+				}
+				const size_t i = (size_t)m * e.n_q + n;
+				if (e.q_f32) {
+					*reinterpret_cast<float2 *>(reinterpret_cast<float *>(e.q_out) + i) = make_float2(a, b);
+				} else {
+					*reinterpret_cast<uint32_t *>(reinterpret_cast<bf16 *>(e.q_out) + i) = pack_bf16(a, b);
+				}
+			} else if (n < e.n_q + e.n_kv) {
+				*reinterpret_cast<float2 *>(e.kv_out + (size_t)m * e.n_kv + (n - e.n_q)) = make_float2(a, b);
+			} else if (n < e.n_q + e.n_kv + e.n_gate) {
+				float *g = e.gate_out + (size_t)m * e.n_gate + (n - e.n_q - e.n_kv);
+				g[0] = sigmoid_f32(a);
+				g[1] = sigmoid_f32(b);
+			}
+			break;
+		}
+	}
+}
+
+// Sixteen consecutive columns of row m (n a multiple of 16), as a tensor-core epilogue holds them.
+template <typename T>
+__device__ __forceinline__ void epi_16(const DenseEpi &e, int m, int n, const float (&v)[16]) {
+	if (e.mode == DENSE_EPI_F32 || e.mode == DENSE_EPI_LOGITS) {
+		float4 *o = reinterpret_cast<float4 *>(reinterpret_cast<float *>(e.out) + (size_t)m * e.ldo + n);
+#pragma unroll
+		for (int i = 0; i < 4; ++i) o[i] = make_float4(v[4 * i] * e.scale, v[4 * i + 1] * e.scale, v[4 * i + 2] * e.scale, v[4 * i + 3] * e.scale);
+	} else if (e.mode == DENSE_EPI_T) {
+		T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
+#pragma unroll
+		for (int i = 0; i < 4; ++i) Elem<T>::store4(o + 4 * i, make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]));
+	} else if (e.mode == DENSE_EPI_SILU) {          // eight gate columns, then the eight up columns of the same outputs
+		T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + (n >> 1);
+#pragma unroll
+		for (int i = 0; i < 2; ++i)
+			Elem<T>::store4(o + 4 * i, make_float4(silu_exact(v[4 * i]) * v[8 + 4 * i], silu_exact(v[4 * i + 1]) * v[9 + 4 * i],
+												   silu_exact(v[4 * i + 2]) * v[10 + 4 * i], silu_exact(v[4 * i + 3]) * v[11 + 4 * i]));
+	} else {          // QKV: a group of 16 columns lies in one head, on one side of rot_at, in one section
+		if (n < e.n_q) {
+			const int off = n % e.head_dim - e.rot_at;
+			float r[16];
+			if (off >= 0 && off < e.rot_dims) {
+				const size_t t = (size_t)epi_pos(e, m) * (e.rot_dims >> 1) + (off >> 1);
+#pragma unroll
+				for (int i = 0; i < 8; ++i) {
+					const bool in = off + 2 * i < e.rot_dims;
+					const float c = in ? __ldg(e.cos_t + t + i) : 1.f, s = in ? __ldg(e.sin_t + t + i) : 0.f;
+					r[2 * i] = v[2 * i] * c - v[2 * i + 1] * s;
+					r[2 * i + 1] = v[2 * i + 1] * c + v[2 * i] * s;
+				}
+			} else {
+#pragma unroll
+				for (int i = 0; i < 16; ++i) r[i] = v[i];
+			}
+			const size_t o = (size_t)m * e.n_q + n;
+			if (e.q_f32) {
+#pragma unroll
+				for (int i = 0; i < 4; ++i)
+					reinterpret_cast<float4 *>(reinterpret_cast<float *>(e.q_out) + o)[i] = make_float4(r[4 * i], r[4 * i + 1], r[4 * i + 2], r[4 * i + 3]);
+			} else {
+#pragma unroll
+				for (int i = 0; i < 2; ++i)
+					reinterpret_cast<uint4 *>(reinterpret_cast<bf16 *>(e.q_out) + o)[i] = make_uint4(pack_bf16(r[8 * i], r[8 * i + 1]), pack_bf16(r[8 * i + 2], r[8 * i + 3]),
+																									pack_bf16(r[8 * i + 4], r[8 * i + 5]), pack_bf16(r[8 * i + 6], r[8 * i + 7]));
+			}
+		} else if (n < e.n_q + e.n_kv) {
+			float4 *o = reinterpret_cast<float4 *>(e.kv_out + (size_t)m * e.n_kv + (n - e.n_q));
+#pragma unroll
+			for (int i = 0; i < 4; ++i) o[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
+		} else {
+#pragma unroll
+			for (int i = 0; i < 16; ++i) {
+				const int g = n - e.n_q - e.n_kv + i;
+				if (g < e.n_gate) e.gate_out[(size_t)m * e.n_gate + g] = sigmoid_f32(v[i]);
+			}
+		}
+	}
+}
+
+// order-preserving map of a float to an unsigned key; ties go to the lower index
+__device__ __forceinline__ unsigned long long argmax_key(float f, int idx) {
+	const uint32_t u = __float_as_uint(f);
+	const uint32_t k = (u & 0x80000000u) ? ~u : (u | 0x80000000u);
+	return ((unsigned long long)k << 32) | (uint32_t)~idx;
+}
+
+struct DenseArgs {
+	const void *x;                   // [M, ldx] T, when there is no row preparation
+	long long ldx;
+	const void *w;                   // [N, ldw] T, K columns used
+	long long ldw;
+	int M, K, N;
+	int prep;                        // 0: x, 1: rows are prepared by the kernel
+	RowPrep rp;
+	DenseEpi e;
+	int *status;
+};
+
+// launchers (dense_skinny.cu, dense_tc.cu, dense_simt.cu)
+int dense_skinny_launch(const DenseArgs &a, int dtype, cudaStream_t stream);
+bool dense_skinny_ok(int M, int K, int dtype);
+int dense_tc_launch(const DenseArgs &a, cudaStream_t stream);
+int dense_simt_launch(const DenseArgs &a, cudaStream_t stream);
+
+int dense_rows_launch(const RowPrep &p, int M, void *h, long long ldh, int dtype, cudaStream_t stream);
+
+int dn_sm_count();
+int dn_smem_opt_in(const void *kernel, size_t bytes);
+
+template <typename... KArgs, typename... Args>
+static int dn_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args &&...args) {
+	if (smem > 16 * 1024)          // static shared memory comes on top (at most 32 KB)
+		if (int rc = dn_smem_opt_in(reinterpret_cast<const void *>(kernel), smem)) return rc;
+	cudaLaunchConfig_t cfg = {};
+	cfg.gridDim = grid;
+	cfg.blockDim = block;
+	cfg.dynamicSmemBytes = smem;
+	cfg.stream = stream;
+	cudaLaunchAttribute attr[1];
+	attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+	attr[0].val.programmaticStreamSerializationAllowed = 1;
+	cfg.attrs = attr;
+	cfg.numAttrs = 1;
+	return cuda_status(cudaLaunchKernelEx(&cfg, kernel, std::forward<Args>(args)...));
+}
+
+}   // namespace gptq

@@ -1,0 +1,324 @@
+// Latent attention of a prompt portion on the 5th-generation tensor cores, expanded form: the caller has multiplied the cached
+// latents with W_uk and W_uv (keys [S, heads * dim], values transposed [heads * vdim, S]); the rotated key part that all heads
+// share comes straight from the cache rows.
+//
+// A CTA serves one head and NQ tiles of 128 query rows against key tiles of 128:
+//   softmax warps     four per query tile, a thread owns a query row: scores from tensor memory, causal mask where the tile
+//                     crosses the diagonal, online softmax in fp32 base 2, weights back to tensor memory; at the end the
+//                     division by the sum, the head's gate and the bf16 store
+//   TMA warp          Q once, then key and value tiles through rings of stages (128-byte swizzle)
+//   MMA warp          S = Q K^T (operands in shared memory), O += P V (P in tensor memory, V^T in shared memory)
+// The weights are kept at more than bf16 precision: P is split into a bf16 high part and a bf16 remainder, which together take
+// exactly the columns of the fp32 scores they replace; both parts multiply the same V tile.  The running output stays in
+// tensor memory; it is rescaled only when a row's maximum has grown by more than 2^8 since the last rescale (the weights are
+// then at most 2^8 and the result is the same, the reference point of a softmax cancels).
+// With NQ = 2 the MMAs of one query tile run under the softmax of the other.  Every wait is bounded.
+#include <algorithm>
+
+#include "../tcgen05.cuh"
+#include "latent.cuh"
+
+namespace gptq {
+
+int dense_tensor_map(const void *base, long long rows, long long cols, long long ld, int box_rows, int box_cols, CUtensorMap *out);
+
+namespace {
+
+constexpr int LP_T = 128;                               // query rows and keys per tile
+constexpr int LP_CHUNK = LP_T * 128;                    // bytes of a 128 x 64 bf16 operand chunk
+constexpr uint32_t LP_SPIN = 1u << 24;
+constexpr size_t LP_SMEM = 226 * 1024;
+
+struct LpPlan {
+	int nd, nr, sk, sv;                                   // chunks of the unrotated / rotated part, stages of K and V
+	size_t smem;
+};
+
+__device__ __forceinline__ float ex2(float x) {
+	float r;
+	asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+	return r;
+}
+// registers loaded by tcgen05.ld may be used only behind the wait: tie them to it
+template <int N>
+__device__ __forceinline__ void tmem_settle(float (&v)[N]) {
+#pragma unroll
+	for (int i = 0; i < N; ++i) asm volatile("" : "+f"(v[i]));
+}
+
+template <int NQ>
+__global__ void __launch_bounds__(NQ * 128 + 64, 1) latent_prefill_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_constant__ CUtensorMap tmk,
+																		 const __grid_constant__ CUtensorMap tmr, const __grid_constant__ CUtensorMap tmv,
+																		 const LatentPrefill p, const LpPlan pl, uint32_t tmem_cols) {
+	extern __shared__ unsigned char lp_raw[];
+	unsigned char *smem = lp_raw + ((1024u - (smem_u32(lp_raw) & 1023u)) & 1023u);
+	const int nch = pl.nd + pl.nr;
+	const uint32_t k_bytes = nch * LP_CHUNK, v_bytes = 2u * p.vdim * 128u;
+	const uint32_t sq = smem_u32(smem), sk = sq + NQ * k_bytes, sv = sk + pl.sk * k_bytes;
+	uint64_t *bars = reinterpret_cast<uint64_t *>(smem + (size_t)(NQ + pl.sk) * k_bytes + (size_t)pl.sv * v_bytes);
+	const uint32_t b0 = smem_u32(bars);
+	const uint32_t bar_q = b0, bar_drain = b0 + 8, bar_fk = b0 + 16, bar_ek = b0 + 32, bar_fv = b0 + 48, bar_ev = b0 + 64;      // two slots each for K, V
+	const uint32_t bar_s = b0 + 80, bar_p = b0 + 96, bar_o = b0 + 112;                                                          // one per query tile
+	uint32_t *s_tmem = reinterpret_cast<uint32_t *>(bars + 16);
+	volatile int *s_abort = reinterpret_cast<volatile int *>(s_tmem + 1);
+	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+	const int nqb = (p.t + NQ * LP_T - 1) / (NQ * LP_T);
+	const int head = blockIdx.x % p.heads, q0 = (nqb - 1 - (int)blockIdx.x / p.heads) * NQ * LP_T;          // the longest rows first
+	const int hd = p.dim + p.rot_dim;
+	auto tiles_of = [&](int i) {
+		const int first = q0 + i * LP_T;
+		return first >= p.t ? 0 : (p.start + min(first + LP_T, p.t) - 1) / LP_T + 1;
+	};
+	int ntile[2] = {tiles_of(0), NQ > 1 ? tiles_of(1) : 0};
+	const int nmax = max(ntile[0], ntile[1]);
+
+	if (tid == 0) {
+		mbar_init(bar_q, 1);
+		mbar_init(bar_drain, 1);
+		for (int s = 0; s < 2; ++s) {
+			mbar_init(bar_fk + 8 * s, 1);
+			mbar_init(bar_ek + 8 * s, 1);
+			mbar_init(bar_fv + 8 * s, 1);
+			mbar_init(bar_ev + 8 * s, 1);
+			mbar_init(bar_s + 8 * s, 1);
+			mbar_init(bar_p + 8 * s, 128);
+			mbar_init(bar_o + 8 * s, 1);
+		}
+		*s_abort = 0;
+		fence_mbar_init();
+	}
+	constexpr int W_TMA = NQ * 4, W_MMA = NQ * 4 + 1;
+	if (warp == W_MMA) {
+		tmem_alloc(smem_u32(s_tmem), tmem_cols);
+		tmem_relinquish();
+	}
+	tc_fence_before();
+	__syncthreads();
+	tc_fence_after();
+	const uint32_t tmem = *s_tmem;
+	auto fail = [&]() {
+		*s_abort = 1;
+		atomicExch(p.status, 3);
+	};
+	pdl_wait();
+	pdl_trigger();
+
+	if (warp == W_TMA) {
+		if (lane == 0) {
+			mbar_arrive_expect_tx(bar_q, NQ * k_bytes);
+			for (int i = 0; i < NQ; ++i)
+				for (int c = 0; c < nch; ++c)
+					tma_load_2d(sq + i * k_bytes + c * LP_CHUNK, &tmq, head * hd + (c < pl.nd ? 64 * c : p.dim + 64 * (c - pl.nd)), q0 + i * LP_T, bar_q);
+			int jk = 0, jv = 0;
+			for (int j = 0; j < nmax; ++j) {
+				const int a = j % pl.sk, b = j % pl.sv;
+				if (*s_abort || !mbar_wait_bounded(bar_ek + 8 * a, ((j / pl.sk) & 1) ^ 1, LP_SPIN)) { fail(); break; }
+				mbar_arrive_expect_tx(bar_fk + 8 * a, k_bytes);
+				for (int c = 0; c < nch; ++c) {
+					const uint32_t dst = sk + a * k_bytes + c * LP_CHUNK;
+					if (c < pl.nd) tma_load_2d(dst, &tmk, head * p.dim + 64 * c, j * LP_T, bar_fk + 8 * a);
+					else tma_load_2d(dst, &tmr, p.kv_rank + 64 * (c - pl.nd), j * LP_T, bar_fk + 8 * a);
+				}
+				jk = j + 1;
+				if (*s_abort || !mbar_wait_bounded(bar_ev + 8 * b, ((j / pl.sv) & 1) ^ 1, LP_SPIN)) { fail(); break; }
+				mbar_arrive_expect_tx(bar_fv + 8 * b, v_bytes);
+				for (int c = 0; c < 2; ++c) tma_load_2d(sv + b * v_bytes + c * (v_bytes / 2), &tmv, j * LP_T + 64 * c, head * p.vdim, bar_fv + 8 * b);
+				jv = j + 1;
+			}
+			// no copy may be in flight when the CTA ends
+			mbar_wait_bounded(bar_q, 0, LP_SPIN);
+			for (int j = max(0, jk - pl.sk); j < jk; ++j) mbar_wait_bounded(bar_fk + 8 * (j % pl.sk), (j / pl.sk) & 1, LP_SPIN);
+			for (int j = max(0, jv - pl.sv); j < jv; ++j) mbar_wait_bounded(bar_fv + 8 * (j % pl.sv), (j / pl.sv) & 1, LP_SPIN);
+		}
+		__syncwarp();
+	} else if (warp == W_MMA) {
+		if (lane == 0) {
+			const uint32_t base = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(LP_T >> 4) << 24);       // D fp32, A/B bf16 K-major, M = 128
+			const uint32_t id_qk = base | ((uint32_t)(LP_T >> 3) << 17), id_pv = base | ((uint32_t)(p.vdim >> 3) << 17);
+			auto wait = [&](uint32_t bar, int n) {
+				if (*s_abort || !mbar_wait_bounded(bar, n & 1, LP_SPIN)) { fail(); return false; }
+				tc_fence_after();
+				return true;
+			};
+			auto qk = [&](int i, int j) {
+				const int a = j % pl.sk;
+				if (!wait(bar_fk + 8 * a, j / pl.sk)) return false;
+				uint32_t acc = 0;
+				for (int c = 0; c < nch; ++c) {
+					const int steps = min(64, c < pl.nd ? p.dim - 64 * c : p.rot_dim - 64 * (c - pl.nd)) >> 4;
+					const uint32_t qa = sq + i * k_bytes + c * LP_CHUNK, ka = sk + a * k_bytes + c * LP_CHUNK;
+					for (int k = 0; k < steps; ++k, acc = 1) umma_f16(tmem + i * LP_T, smem_desc_sw128(qa + k * 32), smem_desc_sw128(ka + k * 32), id_qk, acc);
+				}
+				umma_commit(bar_s + 8 * i);
+				return true;
+			};
+			auto pv = [&](int i, int j) {
+				const int b = j % pl.sv;
+				if (!wait(bar_p + 8 * i, j) || !wait(bar_fv + 8 * b, j / pl.sv)) return false;
+				const uint32_t d = tmem + NQ * LP_T + i * p.vdim, va = sv + b * v_bytes;
+				for (int part = 0; part < 2; ++part)
+					for (int k = 0; k < 8; ++k)
+						umma_f16_ts(d, tmem + i * LP_T + part * 64 + k * 8, smem_desc_sw128(va + (k >> 2) * (v_bytes / 2) + (k & 3) * 32), id_pv, (j | part | k) ? 1u : 0u);
+				umma_commit(bar_o + 8 * i);
+				return true;
+			};
+			bool ok = wait(bar_q, 0);
+			for (int i = 0; i < NQ && ok; ++i)
+				if (ntile[i]) ok = qk(i, 0);
+			umma_commit(bar_ek);
+			for (int j = 0; j < nmax && ok; ++j) {
+				for (int i = 0; i < NQ && ok; ++i) {
+					if (j < ntile[i]) ok = pv(i, j);
+					if (ok && j + 1 < ntile[i]) ok = qk(i, j + 1);
+				}
+				umma_commit(bar_ev + 8 * (j % pl.sv));
+				if (j + 1 < nmax) umma_commit(bar_ek + 8 * ((j + 1) % pl.sk));
+			}
+			umma_commit(bar_drain);          // every MMA has completed before tensor memory goes back
+			mbar_wait_bounded(bar_drain, 0, LP_SPIN);
+		}
+		__syncwarp();
+	} else {
+		const int i = warp >> 2, n = ntile[i];
+		const int row = q0 + i * LP_T + (warp & 3) * 32 + lane, pos = p.start + row;
+		const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
+		const uint32_t ts = tmem + i * LP_T + lane_base, to = tmem + NQ * LP_T + i * p.vdim + lane_base;
+		const float sc = p.scale * 1.4426950408889634f;
+		float ref = 0.f, sum = 0.f;
+		bool ok = true;
+		auto wait = [&](uint32_t bar, int k) {
+			const bool got = !*s_abort && mbar_wait_bounded(bar, k & 1, LP_SPIN);
+			if (!__all_sync(0xffffffffu, got)) { fail(); return false; }
+			tc_fence_after();
+			return true;
+		};
+		for (int j = 0; j < n; ++j) {
+			if (!(ok = wait(bar_s + 8 * i, j))) break;
+			float s[LP_T];
+#pragma unroll
+			for (int c = 0; c < 4; ++c) tmem_ld32(ts + c * 32, reinterpret_cast<float(&)[32]>(s[c * 32]));
+			tmem_ld_wait();
+			tmem_settle(s);
+			if (j * LP_T + LP_T - 1 > p.start + q0 + i * LP_T + (warp & 3) * 32) {          // the tile reaches past this warp's first row
+				const int last = pos - j * LP_T;
+#pragma unroll
+				for (int k = 0; k < LP_T; ++k)
+					if (k > last) s[k] = -INFINITY;
+			}
+			float m0 = s[0], m1 = s[1], m2 = s[2], m3 = s[3];
+#pragma unroll
+			for (int k = 4; k < LP_T; k += 4) {
+				m0 = fmaxf(m0, s[k]);
+				m1 = fmaxf(m1, s[k + 1]);
+				m2 = fmaxf(m2, s[k + 2]);
+				m3 = fmaxf(m3, s[k + 3]);
+			}
+			// scaled maximum; a row below the diagonal of this tile sees none of its keys and keeps its reference point
+			const float mx = fmaxf(fmaxf(m0, m1), fmaxf(m2, m3)), rm = mx == -INFINITY ? (j ? ref : 0.f) : mx * sc;
+			if (j == 0) {
+				ref = rm;
+			} else if (__any_sync(0xffffffffu, rm > ref + 8.f)) {
+				if (!(ok = wait(bar_o + 8 * i, j - 1))) break;
+				const float nref = fmaxf(ref, rm), corr = ex2(ref - nref);
+				ref = nref;
+				sum *= corr;
+#pragma unroll 1
+				for (int c = 0; c < p.vdim; c += 16) {
+					float o[16];
+					tmem_ld16(to + c, o);
+					tmem_ld_wait();
+					tmem_settle(o);
+#pragma unroll
+					for (int k = 0; k < 16; ++k) o[k] *= corr;
+					tmem_st16(to + c, o);
+				}
+				tmem_st_wait();
+			}
+			float t0 = 0.f, t1 = 0.f;
+#pragma unroll
+			for (int c = 0; c < 2; ++c) {
+				uint32_t hi[32], lo[32];
+#pragma unroll
+				for (int k = 0; k < 32; ++k) {
+					const float a = ex2(fmaf(s[c * 64 + 2 * k], sc, -ref)), b = ex2(fmaf(s[c * 64 + 2 * k + 1], sc, -ref));
+					t0 += a;
+					t1 += b;
+					hi[k] = pack_bf16(a, b);
+					lo[k] = pack_bf16(a - __uint_as_float(hi[k] << 16), b - __uint_as_float(hi[k] & 0xFFFF0000u));
+				}
+				tmem_st32(ts + c * 32, hi);
+				tmem_st32(ts + 64 + c * 32, lo);
+			}
+			sum += t0 + t1;
+			tmem_st_wait();
+			tc_fence_before();
+			mbar_arrive(bar_p + 8 * i);
+		}
+		if (n && ok && wait(bar_o + 8 * i, n - 1)) {
+			const float f = row < p.t ? (p.gate ? __ldcg(p.gate + (size_t)row * p.gate_ld + head) : 1.f) / sum : 0.f;
+			bf16 *dst = reinterpret_cast<bf16 *>(p.out) + (size_t)row * p.out_ld + head * p.vdim;
+#pragma unroll 1
+			for (int c = 0; c < p.vdim; c += 16) {
+				float o[16];
+				tmem_ld16(to + c, o);
+				tmem_ld_wait();
+				tmem_settle(o);
+				if (row < p.t) {
+#pragma unroll
+					for (int k = 0; k < 2; ++k)
+						*reinterpret_cast<uint4 *>(dst + c + 8 * k) = make_uint4(pack_bf16(o[8 * k] * f, o[8 * k + 1] * f), pack_bf16(o[8 * k + 2] * f, o[8 * k + 3] * f),
+																				 pack_bf16(o[8 * k + 4] * f, o[8 * k + 5] * f), pack_bf16(o[8 * k + 6] * f, o[8 * k + 7] * f));
+				}
+			}
+		}
+	}
+	tc_fence_before();
+	__syncthreads();
+	if (warp == W_MMA) tmem_dealloc(tmem, tmem_cols);
+}
+
+// stages for nq query tiles per CTA; false: does not fit
+bool lp_plan(int nq, int dim, int rot_dim, int vdim, LpPlan *out) {
+	LpPlan pl;
+	pl.nd = (dim + 63) / 64;
+	pl.nr = (rot_dim + 63) / 64;
+	if (vdim > 256 || nq * (LP_T + vdim) > 512) return false;
+	const size_t k = (size_t)(pl.nd + pl.nr) * LP_CHUNK, v = (size_t)vdim * 256;
+	const int opts[3][2] = {{2, 2}, {2, 1}, {1, 1}};
+	for (auto &o : opts) {
+		pl.sk = o[0];
+		pl.sv = o[1];
+		pl.smem = (nq + pl.sk) * k + pl.sv * v + 1024 + 256;
+		if (pl.smem <= LP_SMEM) {
+			*out = pl;
+			return true;
+		}
+	}
+	return false;
+}
+
+}   // namespace
+
+bool latent_prefill_ok(int dim, int rot_dim, int vdim) {
+	LpPlan pl;
+	return lp_plan(1, dim, rot_dim, vdim, &pl);
+}
+
+int latent_prefill_launch(const LatentPrefill &p, cudaStream_t stream) {
+	LpPlan pl;
+	const bool two = p.t > LP_T && lp_plan(2, p.dim, p.rot_dim, p.vdim, &pl);
+	if (!two && !lp_plan(1, p.dim, p.rot_dim, p.vdim, &pl)) return GPTQ_ERR_UNSUPPORTED;
+	const int nq = two ? 2 : 1, hd = p.dim + p.rot_dim, R = p.kv_rank + p.rot_dim;
+	alignas(64) CUtensorMap tmq, tmk, tmr, tmv;
+	if (int rc = dense_tensor_map(p.q, p.t, (long long)p.heads * hd, (long long)p.heads * hd, LP_T, 64, &tmq)) return rc;
+	if (int rc = dense_tensor_map(p.k, p.S, (long long)p.heads * p.dim, (long long)p.heads * p.dim, LP_T, 64, &tmk)) return rc;
+	if (int rc = dense_tensor_map(p.cache, p.S, R, R, LP_T, 64, &tmr)) return rc;
+	if (int rc = dense_tensor_map(p.vt, (long long)p.heads * p.vdim, p.S, p.ldv, p.vdim, 64, &tmv)) return rc;
+	uint32_t cols = 32;
+	while (cols < (uint32_t)(nq * (LP_T + p.vdim))) cols *= 2;
+	const dim3 grid(p.heads * ((p.t + nq * LP_T - 1) / (nq * LP_T)));
+	if (two) return dn_launch(latent_prefill_kernel<2>, grid, dim3(320), pl.smem, stream, tmq, tmk, tmr, tmv, p, pl, cols);
+	return dn_launch(latent_prefill_kernel<1>, grid, dim3(192), pl.smem, stream, tmq, tmk, tmr, tmv, p, pl, cols);
+}
+
+}   // namespace gptq

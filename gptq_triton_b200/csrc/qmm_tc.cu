@@ -24,6 +24,7 @@
 #include <cuda.h>
 
 #include "qmm_tc.cuh"
+#include "tcgen05.cuh"
 
 namespace gptq {
 
@@ -37,62 +38,6 @@ constexpr uint32_t TC_SPIN = 1u << 24;
 // pipeline depth by tile configuration (shared memory: S * (MH * 16 KB + NSTREAM * BN * 128 B) + packed ring)
 __host__ __device__ constexpr int tc_stages(int nstream, int bn, int mh) { return (mh == 2 && nstream * bn == 256) ? 3 : TC_STAGES; }
 __host__ __device__ constexpr int tc_pstages(int nstream, int bn, int mh) { return (mh == 2) ? (nstream * bn == 256 ? 3 : 6) : (nstream * bn == 256 ? 4 : 8); }
-
-// ---- tcgen05 / TMEM wrappers -------------------------------------------------------------
-__device__ __forceinline__ void tmem_alloc(uint32_t smem_dst, uint32_t ncols) {
-	asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_dst), "r"(ncols) : "memory");
-}
-__device__ __forceinline__ void tmem_relinquish() { asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void tmem_dealloc(uint32_t taddr, uint32_t ncols) {
-	asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(ncols) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-
-// D[tmem] (+)= A[smem desc] * B[smem desc]
-__device__ __forceinline__ void umma_f16(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-	asm volatile(
-		"{\n\t.reg .pred p;\n\t"
-		"setp.ne.b32 p, %4, 0;\n\t"
-		"tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-		:
-		: "r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
-		: "memory");
-}
-// arrive on an mbarrier once all MMAs issued so far by this thread have completed
-__device__ __forceinline__ void umma_commit(uint32_t bar) {
-	asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ void mbar_arrive(uint32_t bar) {
-	asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
-}
-// 32 lanes x 32 consecutive fp32 columns: thread i receives row (lane quarter base + i)
-__device__ __forceinline__ void tmem_ld32(uint32_t taddr, float (&v)[32]) {
-	uint32_t *r = reinterpret_cast<uint32_t *>(v);
-	asm volatile(
-		"tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"
-		"%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-		: "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
-		  "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]),
-		  "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]),
-		  "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-		: "r"(taddr)
-		: "memory");
-}
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-
-// Shared-memory matrix descriptor: K-major tile, 128-byte swizzle, rows of 128 bytes, 8-row
-// groups 1024 bytes apart (SBO), LBO unused (1), descriptor version 1 (sm_100).
-__device__ __forceinline__ uint64_t smem_desc_sw128(uint32_t addr) {
-	uint64_t d = 0;
-	d |= (uint64_t)((addr & 0x3FFFFu) >> 4);            // start address, bits [0,14)
-	d |= (uint64_t)1 << 16;                             // leading byte offset (ignored for swizzled K-major)
-	d |= (uint64_t)(1024 >> 4) << 32;                   // stride byte offset, bits [32,46)
-	d |= (uint64_t)1 << 46;                             // version
-	d |= (uint64_t)2 << 61;                             // layout type: SWIZZLE_128B
-	return d;
-}
-
 
 struct TcParams {
 	TcArgs a;

@@ -21,6 +21,8 @@ import torch
 import torch.nn as nn
 import torch.nn.functional as F
 
+from .cache import StaticCache
+from .engine import StaticEngine
 from .fused_attention import (QuantLlamaAttention, attn_decode, qkv_attn_decode, qkv_attn_oproj_decode, qkv_attn_oproj_scratch,
 							  qkv_attn_supported)
 from .fused_attention import rmsnorm as rmsnorm_kernel
@@ -175,14 +177,14 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
 	return (x.float() * torch.rsqrt(v + eps)).to(x.dtype) * weight
 
 
-class DecodeEngine:
+class DecodeEngine(StaticEngine):
 	"""Greedy decoding with a static KV cache for a model whose attention and MLP blocks have
 	been fused (QuantLlamaAttention / QuantLlamaMLP).  One decode step = 32 x (RMSNorm, fused
 	QKV+rotary writing K/V into the cache, attention over the cache, o_proj + residual, RMSNorm,
 	fused gate/up, down_proj + residual), final norm, fp16 lm_head, argmax."""
 
 	def __init__(self, model: LlamaForCausalLM, batch: int, max_seq: int, use_graph: bool = True, tp_group=None):
-		self.model = model
+		super().__init__(model, batch, max_seq, model.lm_head.weight.device, use_graph)
 		# tensor parallelism: the model holds this rank's shards (tp.shard_llama); partial sums of the
 		# row-parallel projections are all-reduced, the residual is added on rank 0 only
 		self.tp_group = tp_group
@@ -190,17 +192,12 @@ class DecodeEngine:
 		self.tp_world = getattr(model, 'tp_world', 1)
 		cfg = model.config
 		self.cfg = cfg
-		dev = model.lm_head.weight.device
-		self.device = dev
-		self.batch, self.max_seq = batch, max_seq
+		dev = self.device
 		for layer in model.model.layers:
 			assert isinstance(layer.self_attn, QuantLlamaAttention), 'run make_quant_attn first'
 		H, D = model.model.layers[0].self_attn.num_heads, cfg.hidden_size // cfg.num_attention_heads      # local heads
-		self.kcache = [torch.zeros((batch, H, max_seq, D), dtype=torch.float16, device=dev) for _ in model.model.layers]
-		self.vcache = [torch.zeros((batch, H, max_seq, D), dtype=torch.float16, device=dev) for _ in model.model.layers]
-		self.pos = torch.zeros((batch, 1), dtype=torch.int32, device=dev)          # position of the token being fed
-		self.tok = torch.zeros((batch, 1), dtype=torch.int64, device=dev)          # token being fed
-		self.mask = torch.full((batch, 1, 1, max_seq), float('-inf'), dtype=torch.float16, device=dev)
+		self.cache = StaticCache([{'k': (H, max_seq, D), 'v': (H, max_seq, D)} for _ in model.model.layers], batch, torch.float16, dev)
+		self.kcache, self.vcache = self.cache.tensors('k'), self.cache.tensors('v')
 		# tensor parallelism, decode steps: the all-reduce after o_proj / down_proj is fused into those kernels
 		# over peer memory (one exchange buffer per projection); GPTQ_B200_TP_FUSED=0 keeps NCCL
 		self.ar_o = self.ar_down = None
@@ -217,7 +214,6 @@ class DecodeEngine:
 				if self.ar_o is not None:
 					self.ar_o.close()
 				self.ar_o = self.ar_down = None          # NCCL all-reduce instead
-		self.use_graph = use_graph
 		# RMSNorm folded into the decode kernels: o_proj / down_proj leave per-tile sums of squares of
 		# the hidden state, the next QKV / gate-up kernel scales x while staging it (one GPU only)
 		self.fuse_norm = True
@@ -225,14 +221,9 @@ class DecodeEngine:
 		self.ss_attn = torch.zeros((batch, tiles), dtype=torch.float32, device=dev)
 		self.ss_mlp = torch.zeros((batch, tiles), dtype=torch.float32, device=dev)
 		self.len_hint = max_seq
-		self.graph = None
-		self.launches_per_step = None
 		self._qao_scratch = None
-		# captures of the decode step to choose from (see step()); 1 = take the first
-		self.graph_candidates = int(os.environ.get('GPTQ_B200_GRAPH_CANDIDATES', '6'))
 		self.used_qkv_attn = False          # set when a decode step ran the one-kernel QKV + attention path
 		self.used_fused_oproj = False       # ... with o_proj and the residual add in the same kernel
-		self.next_pos = 0          # host-side copy of the position the next step() writes (the cache has max_seq rows)
 		# One persistent kernel per decode step (gptq_decode_chain) + the lm_head / arg-max kernel, where the model
 		# allows it (one GPU, batch <= 8, no act-order, no bias, one group size); opt-in with GPTQ_B200_CHAIN=1 (default: the
 		# kernel-per-projection path).
@@ -398,26 +389,18 @@ class DecodeEngine:
 			all_reduce_(h, self.tp_group)
 		return h, ss_out
 
-	@torch.no_grad()
-	def prefill(self, input_ids: torch.Tensor) -> torch.Tensor:
-		"""Runs the prompt [b, t], fills the cache, returns the first generated token [b, 1]."""
+	def _portion(self, input_ids: torch.Tensor, start: int, want):
 		b, t = input_ids.shape
-		assert b == self.batch and t < self.max_seq
-		pos = torch.arange(t, device=self.device, dtype=torch.int32).unsqueeze(0).expand(b, t).contiguous()
-		mask = causal_mask(t, 0, self.device)
+		pos = torch.arange(start, start + t, device=self.device, dtype=torch.int32).unsqueeze(0).expand(b, t).contiguous()
+		mask = causal_mask(t, start, self.device)
 		h = self.model.model.embed_tokens(input_ids)
 		for i in range(len(self.model.model.layers)):
-			h, _ = self._layer(i, h, pos, mask, t)
-		h = rmsnorm(h[:, -1:, :], self.model.model.norm.weight, self.model.model.norm.variance_epsilon)
-		logits = self.model.lm_head(h)
-		self.logits = logits
-		self.tok.copy_(logits.argmax(-1))
-		self.pos.fill_(t)
-		self.next_pos = t
-		self.len_hint = t + 1
-		self.mask.fill_(float('-inf'))
-		self.mask[..., :t + 1] = 0
-		return self.tok.clone()
+			h, _ = self._layer(i, h, pos, mask, start + t)
+		self.len_hint = start + t + 1
+		if not want:
+			return None
+		h = rmsnorm(h[:, list(want), :], self.model.model.norm.weight, self.model.model.norm.variance_epsilon)
+		return self.model.lm_head(h)
 
 	def _one_kernel_attention(self, attn) -> bool:
 		"""Whether the layer's QKV projection and attention run as one kernel in a decode step of one sequence
@@ -478,13 +461,13 @@ class DecodeEngine:
 											   float(ln.variance_epsilon), _lib.stream_ptr(self.device))
 			_lib.check(rc, 'gptq_embed_rmsnorm')
 			h = ends['h0']
-			h, ss = self._layer(0, h, self.pos, self.mask, self.max_seq, None, x_normed=ends['x0'])
+			h, ss = self._layer(0, h, self.pos, None, self.max_seq, None, x_normed=ends['x0'])
 			rest = range(1, len(m.layers))
 		else:
 			h = m.embed_tokens(self.tok)
 			rest = range(len(m.layers))
 		for i in rest:
-			h, ss = self._layer(i, h, self.pos, self.mask, self.max_seq, ss)
+			h, ss = self._layer(i, h, self.pos, None, self.max_seq, ss)
 		eps = float(m.norm.variance_epsilon)
 		if ends is not None and ss is not None:
 			# final norm (from the sums of squares the last down_proj left), lm_head, arg-max, next token and position
@@ -502,87 +485,17 @@ class DecodeEngine:
 		self.tok.copy_(nxt)
 		self.pos.add_(1)
 
-	@torch.no_grad()
-	def step(self) -> torch.Tensor:
-		"""Feeds self.tok at self.pos, returns the next token [b, 1] (device tensor)."""
-		if self.next_pos >= self.max_seq:
-			raise RuntimeError(f'DecodeEngine: the static KV cache holds {self.max_seq} positions and is full; build the engine with a larger max_seq')
-		self.next_pos += 1
-		if not self.use_graph:
-			self._step_body()
-			return self.tok
-		if self.graph is None:
-			if self.ar_o is not None:
-				# the fused exchange waits at most two seconds for a peer: start the ranks together
-				import torch.distributed as dist
-				torch.cuda.synchronize()
-				dist.barrier(group=self.tp_group)
-			# warm up on a side stream (allocations, workspaces), then capture
-			saved = (self.tok.clone(), self.pos.clone(), self.mask.clone())
-			s = torch.cuda.Stream()
-			s.wait_stream(torch.cuda.current_stream())
-			best, best_ms, best_logits = None, None, None
-			with torch.cuda.stream(s):
-				for _ in range(2):
-					self._step_body()
-					self.tok.copy_(saved[0]); self.pos.copy_(saved[1]); self.mask.copy_(saved[2])
-				s.synchronize()
-				# The activations of a step live in the graph's private memory pool.  Where that pool lands (which physical
-				# 2 MB page) decides how fast the few lines that every CTA reads right after a kernel boundary arrive: the same
-				# graph replays 7 % faster or slower from one capture to the next (two modes, measured).  So the step is captured several
-				# times, every candidate is timed on a few replays, and the fastest one is kept.  The replays write cache rows
-				# at the current position onwards, which the real steps write again; token and position are restored.
-				n_cand = max(1, self.graph_candidates)          # tensor parallel: every rank replays the same number of times, the choice is per rank
-				alive = []          # every candidate keeps its pool until the choice is made: a freed pool would be handed to the next capture
-				for _ in range(n_cand):
-					g = torch.cuda.CUDAGraph()
-					with torch.cuda.graph(g, stream=s):
-						self._step_body()
-					alive.append(g)
-					cand_logits = self.logits          # the capture's own output tensor (it lives in that graph's pool)
-					if n_cand == 1:
-						best, best_logits = g, cand_logits
-						break
-					reps = max(1, min(8, self.max_seq - 1 - int(saved[1].max().item())))
-					e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-					g.replay()
-					e0.record(s)
-					for _ in range(reps):
-						self.tok.copy_(saved[0]); self.pos.copy_(saved[1])
-						g.replay()
-					e1.record(s)
-					s.synchronize()
-					ms = e0.elapsed_time(e1) / reps
-					if best_ms is None or ms < best_ms:
-						best, best_ms, best_logits = g, ms, cand_logits
-				del alive
-			torch.cuda.current_stream().wait_stream(s)
-			# capture does not execute (and the timed replays started from the saved state): restore it
-			self.tok.copy_(saved[0]); self.pos.copy_(saved[1]); self.mask.copy_(saved[2])
-			self.graph = best
-			self.logits = best_logits
-		self.graph.replay()
-		return self.tok
-
-	@torch.no_grad()
-	def generate(self, input_ids: torch.Tensor, steps: int) -> torch.Tensor:
-		"""Greedy generation: returns [b, steps] token ids (the first comes from the prefill)."""
-		from . import _lib
-		out = [self.prefill(input_ids)]
-		for _ in range(steps - 1):
-			out.append(self.step().clone())
-		toks = torch.cat(out, dim=1)
-		# the kernels' bounded waits report through a status word instead of hanging: a non-zero word means
-		# that some result of this run cannot be trusted
-		status = _lib.kernel_status(self.device)
-		if status != 0:
-			raise _lib.GptqB200Error(f'a decode kernel reported status {status} (see _lib.kernel_status)')
-		return toks
+	def _before_capture(self):
+		if self.ar_o is not None:
+			# the fused exchange waits at most two seconds for a peer: start the ranks together
+			import torch.distributed as dist
+			torch.cuda.synchronize()
+			dist.barrier(group=self.tp_group)
 
 	def close(self):
 		"""Releases the tensor-parallel exchange buffers (mapped by the peers: call it on every rank, after the
 		last step has completed everywhere) and the captured graph."""
-		self.graph = None
+		super().close()
 		for name in ('ar_o', 'ar_down'):
 			ex = getattr(self, name, None)
 			if ex is not None:

@@ -1,0 +1,132 @@
+/*
+ * dense_b200.h — C ABI of libdense_b200.so: decoder layers with dense bf16 (or fp32) weights on NVIDIA B200 (sm_100a).
+ * Projections with fused row preparation and epilogues, and latent attention (keys and values in one low-rank row per token).
+ *
+ * Every pointer inside the argument blocks is a DEVICE pointer.  Entry points are asynchronous on `stream`, never
+ * synchronise, allocate or free, and return 0 or a negative GPTQ_ERR_* code (gptq_b200.h).
+ *
+ * dtype: 0 = bf16 weights and activations with fp32 accumulation, 1 = fp32 throughout (no reduced-precision products).
+ * Weights are [N, K] with K contiguous.  Feature sizes (K, head parts, latent rank) are multiples of 16: the caller pads
+ * weights and rows with zeros; sizes that enter a mean are passed as true sizes beside the padded ones.
+ */
+#ifndef DENSE_B200_H
+#define DENSE_B200_H
+
+#include <stddef.h>
+#include <stdint.h>
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+#define DENSE_CONTROL_BYTES 16384      /* control buffer of an engine: zeroed once; its last word is the status word */
+
+/* epilogues of dense_matmul */
+#define DENSE_EPI_F32     0            /* out fp32 [M, ldo] = scale * result */
+#define DENSE_EPI_T       1            /* out in the activation dtype */
+#define DENSE_EPI_SILU    2            /* weight rows in groups of 16: 8 gate rows, 8 up rows; out[8 g + j] = silu(gate_j) * up_j */
+#define DENSE_EPI_QKV     3            /* rotary queries | raw fp32 latent rows | sigmoid gates */
+#define DENSE_EPI_LOGITS  4            /* F32, and with `best` set the greedy choice per row (decode rows only) */
+
+/* Row preparation: x = table[token], or x_in (+ LayerNorm(y) * gain + shift when y is set, mean and variance over `width`
+ * of the `ld` columns); x_out (optional, never the same as x_in) receives it; the prepared row is x, or LayerNorm(x) * fin_w
+ * + fin_b when fin_w is set. */
+typedef struct {
+	const float *x_in;
+	float *x_out;
+	const float *y;
+	const float *gain, *shift;
+	const float *fin_w, *fin_b;
+	const void *table;
+	const int64_t *token;
+	int64_t vocab;
+	int width, ld;
+	float eps;
+	int *status;
+} dense_rows_t;
+
+typedef struct {
+	int mode;
+	void *out;
+	int64_t ldo;
+	float scale;
+	/* QKV: n_q query columns, heads of head_dim; in each head the pairs (2i, 2i+1) of [rot_at, rot_at + rot_dims) are rotated by
+	 * the table row of pos[m]; n_kv raw columns; n_gate gate columns */
+	int n_q, head_dim, rot_at, rot_dims, n_kv, n_gate;
+	const float *cos_t, *sin_t;        /* [max_pos, rot_dims / 2] */
+	const int32_t *pos;                /* [M] */
+	int max_pos;
+	void *q_out;
+	int q_f32;
+	float *kv_out;
+	float *gate_out;
+	int *status;
+	/* LOGITS */
+	unsigned long long *best;          /* [M], zero before and after every launch */
+	unsigned *ticket;
+	int64_t *tok;                      /* receives the arg-max (lowest index on ties) */
+	int32_t *pos_inout;                /* incremented */
+} dense_epilogue_t;
+
+/* Latent attention, absorbed form.  A cache row is [latent (kv_rank) | rotated key part (rot_dim)]. */
+typedef struct {
+	int M, rows_per_seq;               /* query rows, rows_per_seq consecutive rows per sequence */
+	int heads, dim, rot_dim, vdim, kv_rank, kv_width, rot_dims, max_seq, splits;
+	float scale, eps;
+	const int32_t *pos;                /* [M] */
+	const float *q;                    /* [M, heads * (dim + rot_dim)] fp32, rotated */
+	const void *w_uk, *w_uv;           /* [heads * dim, kv_rank], [heads * vdim, kv_rank] */
+	const float *kv_raw;               /* [M, kv_rank + rot_dim], or NULL: another layer has written the cache rows */
+	const float *kv_norm;              /* [kv_rank] */
+	const float *cos_t, *sin_t;
+	void *cache;                       /* [sequences, max_seq, kv_rank + rot_dim] */
+	void *qa_hi, *qa_lo;               /* bf16 [M, heads, kv_rank + rot_dim] */
+	float *qa_f32;                     /* dtype 1 */
+	float *part_ml;                    /* [M, heads, splits, 2] */
+	float *part_acc;                   /* [M, heads, splits, kv_rank] */
+	const float *gate;                 /* [M, gate_ld], or NULL */
+	int gate_ld;
+	void *out;                         /* [M, out_ld] */
+	int64_t out_ld;
+	int *status;
+} dense_latent_t;
+
+/* Latent attention of a prompt portion of one sequence, expanded form, bf16. */
+typedef struct {
+	int t, start, S;                   /* t query rows at positions start ..; S = start + t keys */
+	int heads, dim, rot_dim, vdim, kv_rank;
+	float scale;
+	const void *q;                     /* bf16 [t, heads * (dim + rot_dim)], rotated */
+	const void *k;                     /* bf16 [S, heads * dim] */
+	const void *vt;                    /* bf16 [heads * vdim, ldv]: values transposed, ldv a multiple of 8 */
+	int64_t ldv;
+	const void *cache;                 /* bf16 [S, kv_rank + rot_dim] */
+	const float *gate;
+	int gate_ld;
+	void *out;                         /* bf16 [t, out_ld] */
+	int64_t out_ld;
+	int *status;
+} dense_latent_prefill_t;
+
+int dense_version(void);
+int dense_last_cuda_error(void);
+
+/* y = epilogue(rows x W^T).  With `rows` the kernel prepares its input rows itself (few rows only, see dense_decode_rows_ok),
+ * else x is [M, ldx].  w is [N, ldw].  Chooses the decode kernel, the tensor-core kernel or the fp32 kernel by shape. */
+int dense_matmul(const void *x, int64_t ldx, const void *w, int64_t ldw, int M, int K, int N, int dtype, const dense_rows_t *rows, const dense_epilogue_t *epi,
+				 int *status, void *stream);
+int dense_decode_rows_ok(int M, int K, int dtype);      /* the decode kernel (and row preparation inside it) covers M rows of K */
+int dense_prepare_rows(const dense_rows_t *rows, int M, void *h, int64_t ldh, int dtype, void *stream);
+
+int dense_latent_splits(int M, int heads, int max_seq, int dtype);
+int dense_latent_append(const dense_latent_t *args, int dtype, void *stream);       /* cache rows only */
+int dense_latent_absorb(const dense_latent_t *args, int dtype, void *stream);       /* absorbed queries and, with kv_raw, cache rows */
+int dense_latent_attend(const dense_latent_t *args, int dtype, void *stream);
+int dense_latent_value(const dense_latent_t *args, int dtype, void *stream);
+int dense_latent_prefill_ok(int dim, int rot_dim, int vdim);
+int dense_latent_prefill(const dense_latent_prefill_t *args, void *stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif
