@@ -850,6 +850,281 @@ def kernel_case(args):
 	print(json.dumps({'kernel_case': args.kernel_case, 'M': M, 'launches': 8}))
 
 
+# ------------------------------------------------------------------------------------------
+# --workload befalix: prefill and decode of a latent-attention design beside the LLaMA path at equal size
+# ------------------------------------------------------------------------------------------
+BEFALIX_CASES = (
+	# name, layers, hidden, intermediate, heads, head dim (unrotated), rotated, value, latent
+	('2048', 8, 2048, 5504, 16, 128, 64, 128, 512),
+	('4096', 4, 4096, 11008, 32, 128, 64, 128, 512),
+	('8192', 2, 8192, 22016, 64, 128, 64, 128, 512),
+)
+
+
+def graph_us(calls, reps: int = 10) -> float:
+	"""Microseconds per call: `calls` (each on its own data, together larger than L2) captured in one CUDA graph, replayed."""
+	import torch
+	s = torch.cuda.Stream()
+	with torch.cuda.stream(s):
+		for c in calls:
+			c()
+		s.synchronize()
+		g = torch.cuda.CUDAGraph()
+		with torch.cuda.graph(g, stream=s):
+			for c in calls:
+				c()
+		for _ in range(3):
+			g.replay()
+		e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+		e0.record(s)
+		for _ in range(reps):
+			g.replay()
+		e1.record(s)
+		s.synchronize()
+	return e0.elapsed_time(e1) * 1e3 / reps / len(calls)
+
+
+def event_us(calls, reps: int = 3) -> float:
+	"""The same without a graph, for calls that may not be captured."""
+	import torch
+	for c in calls:
+		c()
+	torch.cuda.synchronize()
+	e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+	e0.record()
+	for _ in range(reps):
+		for c in calls:
+			c()
+	e1.record()
+	torch.cuda.synchronize()
+	return e0.elapsed_time(e1) * 1e3 / reps / len(calls)
+
+
+def engine_rates(engine, vocab: int, steps: int, prompt_len: int = PROMPT):
+	"""(prompt tokens/s, decode ms per step after the prompt) of any engine, device-timed."""
+	import torch
+	prompt = torch.randint(0, vocab, (engine.batch, prompt_len), generator=torch.Generator().manual_seed(3)).to(engine.device)
+	for _ in range(3):
+		engine.prefill(prompt)
+	e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+	torch.cuda.synchronize()
+	e0.record()
+	for _ in range(3):
+		engine.prefill(prompt)
+	e1.record()
+	torch.cuda.synchronize()
+	rate = 3 * prompt.numel() / e0.elapsed_time(e1) * 1e3
+	for _ in range(4):
+		engine.step()
+	torch.cuda.synchronize()
+	e0.record()
+	for _ in range(steps):
+		engine.step()
+	e1.record()
+	torch.cuda.synchronize()
+	return rate, e0.elapsed_time(e1) / steps
+
+
+def befalix_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: int = PROMPT):
+	"""Every kernel of the design alone, on rotating copies of its operands: microseconds, and the fraction of the measured
+	copy bandwidth (decode) or of the measured cuBLAS bf16 rate (prompts) that its algorithmic bytes or operations amount to."""
+	import ctypes
+	import torch
+	from gptq_triton_b200 import _dense
+	from gptq_triton_b200._lib import stream_ptr
+	from gptq_triton_b200.dense import Stream, epilogue, linear, matmul, prepare_rows, project_stream
+	m, cfg, dev, ctl = engine.model, engine.cfg, engine.device, engine.control
+	lib, sp = _dense.lib(), lambda: stream_ptr(dev)
+	layer = m.layers[0]
+	mx, spec, W = layer.mixer, layer.mixer.spec, m.embed.shape[1]
+	H, D, R, V, C = spec.heads, mx.D, mx.R, mx.V, mx.C
+	out = {}
+
+	def copies(w, limit=320e6):
+		return [w] + [w.clone() for _ in range(max(3, min(80, int(limit / (w.numel() * w.element_size())))))]
+
+	def record(name, us, nbytes=None, flops=None):
+		r = {'us': round(us, 2)}
+		if nbytes is not None:
+			r['frac_hbm'] = round(nbytes / us / 1e3 / hbm, 3)
+		if flops is not None:
+			r['frac_tensor'] = round(flops / us / 1e6 / tflops, 3)
+		out[name] = r
+
+	x1 = torch.randn((1, W), device=dev)
+	s1 = Stream(cfg.width, W, cfg.norm_eps, x=x1, y=torch.randn((1, W), device=dev), gain=layer.mixer_norm.gain, shift=layer.mixer_norm.shift)
+	pos = torch.full((1,), ctx, dtype=torch.int32, device=dev)
+	q = torch.randn((1, H * (D + R)), device=dev)
+	gate = torch.rand((1, mx.G), device=dev)
+	kv = torch.randn((1, spec.row), device=dev)
+	attn = torch.empty((1, H * V), dtype=m.dtype, device=dev)
+
+	def qkv_epi(M, posv, q_out, kv_out, gate_out, f32):
+		e = _dense.Epilogue()
+		e.mode, e.n_q, e.head_dim, e.rot_at, e.rot_dims, e.n_kv, e.n_gate = _dense.EPI_QKV, H * (D + R), D + R, D, spec.rot_dims, spec.row, mx.G
+		e.cos_t, e.sin_t, e.pos, e.max_pos = engine.tables[0][0].data_ptr(), engine.tables[0][1].data_ptr(), posv.data_ptr(), engine.max_seq
+		e.q_out, e.q_f32, e.kv_out, e.gate_out, e.status = q_out.data_ptr(), int(f32), kv_out.data_ptr(), gate_out.data_ptr(), _dense.status_ptr(ctl).value
+		return e
+	esz = lambda w: w.numel() * w.element_size()
+	e = qkv_epi(1, pos, q, kv, gate, True)
+	record('decode in-projection', graph_us([lambda w=w: project_stream(s1, w, e, ctl) for w in copies(mx.w_in)]), esz(mx.w_in))
+	S = ctx + 1
+	caches = [torch.randn((1, engine.max_seq, spec.row), device=dev).to(m.dtype) for _ in range(max(4, min(120, int(320e6 / (S * spec.row * 2)))))]
+	args = []
+	keep = []
+	for w_uk, w_uv, c in zip(copies(mx.w_uk), copies(mx.w_uv), caches):
+		a = mx.arguments(c, pos, 1, engine.tables[0], cfg.norm_eps, ctl, kv)
+		keep.append((mx.absorbed_buffers(a, q, gate, attn, engine.max_seq), w_uk, w_uv))
+		a.w_uk, a.w_uv = w_uk.data_ptr(), w_uv.data_ptr()
+		args.append(a)
+	call = lambda fn, a: _dense.check(fn(ctypes.byref(a), 0, sp()), 'bench')
+	call(lib.dense_latent_absorb, args[0])
+	record('decode absorb + cache row', graph_us([lambda a=a: call(lib.dense_latent_absorb, a) for a in args]), esz(mx.w_uk))
+	acc_bytes = H * args[0].splits * (C + 2) * 4
+	cargs = []
+	for c in caches:
+		a = mx.arguments(c, pos, 1, engine.tables[0], cfg.norm_eps, ctl, kv)
+		keep.append(mx.absorbed_buffers(a, q, gate, attn, engine.max_seq))
+		cargs.append(a)
+	record('decode attention', graph_us([lambda a=a: call(lib.dense_latent_attend, a) for a in cargs]), S * spec.row * 2)
+	record('decode merge + value', graph_us([lambda a=a: call(lib.dense_latent_value, a) for a in args]), esz(mx.w_uv) + acc_bytes)
+	record('decode out-projection', graph_us([lambda w=w: linear(attn, w, ctl) for w in copies(mx.w_o)]), esz(mx.w_o))
+	gu, down = layer.mlp.gate_up, layer.mlp.down
+	act = torch.empty((1, down.shape[1]), dtype=m.dtype, device=dev)
+	record('decode gate/up', graph_us([lambda w=w: project_stream(s1, w, epilogue(_dense.EPI_SILU, act), ctl) for w in copies(gu)]), esz(gu))
+	record('decode down', graph_us([lambda w=w: linear(act, w, ctl) for w in copies(down)]), esz(down))
+	logits = torch.empty((1, (cfg.vocab_size + 15) // 16 * 16), device=dev)
+	record('decode logits', graph_us([lambda w=w: project_stream(s1, w, epilogue(_dense.EPI_LOGITS, logits), ctl, keep=False, final=m.norm) for w in copies(m.embed)]), esz(m.embed))
+	# ---- prompt of t tokens ----
+	xs = torch.randn((t, W), device=dev)
+	st = Stream(cfg.width, W, cfg.norm_eps, x=xs, y=torch.randn((t, W), device=dev), gain=layer.mixer_norm.gain, shift=layer.mixer_norm.shift)
+	record('prompt rows (norm, residual)', graph_us([lambda: prepare_rows(st, ctl, m.dtype, True)] * 4), t * W * (4 + 4 + 4 + 2))
+	h = torch.randn((t, W), device=dev).to(m.dtype)
+	posp = torch.arange(t, dtype=torch.int32, device=dev)
+	qp = torch.empty((t, H * (D + R)), dtype=m.dtype, device=dev)
+	kvp, gp = torch.randn((t, spec.row), device=dev), torch.rand((t, mx.G), device=dev)
+	ep = qkv_epi(t, posp, qp, kvp, gp, False)
+	gemm = lambda name, fn, w, M=t: record(name, graph_us(fn), flops=2.0 * M * w.shape[0] * w.shape[1])
+	gemm('prompt in-projection', [lambda w=w: matmul(h, w, ep, ctl) for w in copies(mx.w_in)], mx.w_in)
+	ap = mx.arguments(caches[0], posp, t, engine.tables[0], cfg.norm_eps, ctl, kvp)
+	record('prompt cache rows', graph_us([lambda: call(lib.dense_latent_append, ap)] * 4), t * spec.row * 6)
+	lat = caches[0][0, :t, :C]
+	k, vt = torch.empty((t, H * D), dtype=m.dtype, device=dev), torch.empty((H * V, (t + 15) // 16 * 16), dtype=m.dtype, device=dev)
+	gemm('prompt expand keys', [lambda w=w: matmul(lat, w, epilogue(_dense.EPI_T, k), ctl) for w in copies(mx.w_uk)], mx.w_uk)
+	gemm('prompt expand values', [lambda w=w: matmul(w, lat, epilogue(_dense.EPI_T, vt), ctl) for w in copies(mx.w_uv)], mx.w_uv)
+	op = torch.empty((t, H * V), dtype=m.dtype, device=dev)
+	p = _dense.LatentPrefill()
+	p.t, p.start, p.S, p.heads, p.dim, p.rot_dim, p.vdim, p.kv_rank, p.scale = t, 0, t, H, D, R, V, C, spec.scale
+	p.q, p.k, p.vt, p.ldv, p.cache, p.gate, p.gate_ld = qp.data_ptr(), k.data_ptr(), vt.data_ptr(), vt.stride(0), caches[0].data_ptr(), gp.data_ptr(), gp.stride(0)
+	p.out, p.out_ld, p.status = op.data_ptr(), op.stride(0), _dense.status_ptr(ctl).value
+	us = graph_us([lambda: _dense.check(lib.dense_latent_prefill(ctypes.byref(p), sp()), 'bench')] * 4)
+	record('prompt attention', us, flops=float(t) * (t + 1) * H * (D + R + V))
+	gemm('prompt out-projection', [lambda w=w: linear(op, w, ctl) for w in copies(mx.w_o)], mx.w_o)
+	actp = torch.empty((t, down.shape[1]), dtype=m.dtype, device=dev)
+	gemm('prompt gate/up', [lambda w=w: matmul(h, w, epilogue(_dense.EPI_SILU, actp), ctl) for w in copies(gu)], gu)
+	gemm('prompt down', [lambda w=w: linear(actp, w, ctl) for w in copies(down)], down)
+	return out
+
+
+def llama_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: int = PROMPT):
+	"""The like kernels of the 4-bit LLaMA engine, the same way (weights rotate over the layers)."""
+	import torch
+	import torch.nn.functional as F
+	from gptq_triton_b200.fused_attention import qkv_attn_oproj_decode, qkv_attn_oproj_scratch
+	from gptq_triton_b200.llama import causal_mask
+	cfg, dev = engine.cfg, engine.device
+	L = engine.model.model.layers
+	hid, inter, H = cfg.hidden_size, cfg.intermediate_size, cfg.num_attention_heads
+	out = {}
+
+	def record(name, us, nbytes=None, flops=None):
+		out[name] = {'us': round(us, 2), **({'frac_hbm': round(nbytes / us / 1e3 / hbm, 3)} if nbytes is not None else {'frac_tensor': round(flops / us / 1e6 / tflops, 3)})}
+	x1 = torch.randn((1, 1, hid), device=dev).half()
+	ss = x1.float().pow(2).view(1, hid // 32, 32).sum(-1).contiguous()
+	pos = torch.full((1,), ctx, dtype=torch.int32, device=dev)
+	rot = [l for _ in range(max(1, 16 // len(L))) for l in L]
+	layers = list(enumerate(L))
+	if engine._one_kernel_attention(L[0].self_attn):
+		cos, sin = L[0].self_attn.tables(dev, engine.max_seq)
+		scratch = qkv_attn_oproj_scratch(H, hid, dev)
+		def block(i, l):
+			a, o = l.self_attn, l.self_attn.o_proj
+			qw, _, _ = a.qkv_proj.kernel_operands()
+			return qkv_attn_oproj_decode(a.qkv_proj.groupsize, x1, qw, a.qkv_proj.scales, a.qkv_proj.qzeros, cos, sin, pos, engine.kcache[i], engine.vcache[i], H,
+										 o.groupsize, o.qweight, o.scales, o.qzeros, scratch, residual=x1, sumsq_out=engine.ss_attn, rms_weight=l.input_layernorm.weight,
+										 rms_eps=1e-6, sumsq_in=ss)
+		record('decode attention block (qkv, attention, o)', graph_us([lambda i=i, l=l: block(i, l) for i, l in layers]),
+			   quantised_bytes(hid, 3 * hid) + quantised_bytes(hid, hid) + 2 * H * (ctx + 1) * 256)
+	y1 = torch.randn((1, 1, inter), device=dev).half()
+	record('decode gate/up', graph_us([lambda l=l: l.mlp.intermediate(x1, rms_weight=l.post_attention_layernorm.weight, rms_eps=1e-6, sumsq_in=ss) for l in rot]), quantised_bytes(hid, 2 * inter))
+	record('decode down', graph_us([lambda l=l: l.mlp.down_proj(y1, residual=x1, sumsq_out=engine.ss_mlp) for l in rot]), quantised_bytes(inter, hid))
+	record('decode o', graph_us([lambda l=l: l.self_attn.o_proj(x1, residual=x1, sumsq_out=engine.ss_attn) for l in rot]), quantised_bytes(hid, hid))
+	from gptq_triton_b200.fused_attention import attn_decode
+	q1 = torch.randn((1, H, 1, 128), device=dev).half()
+	kcs = [(torch.randn_like(engine.kcache[0]), torch.randn_like(engine.vcache[0])) for _ in range(max(4, int(320e6 / (2 * H * ctx * 256))))]
+	record('decode attention', graph_us([lambda k=k, v=v: attn_decode(q1, k, v, pos, ctx + 1) for k, v in kcs]), 2 * H * (ctx + 1) * 256)
+	xp = (torch.randn((1, t, hid), device=dev) * 0.5).half()
+	yp = (torch.randn((1, t, inter), device=dev) * 0.5).half()
+	pp = torch.arange(t, device=dev, dtype=torch.int32)[None]
+	record('prompt qkv', event_us([lambda i=i, l=l: l.self_attn.project_qkv(xp, pp, kv_cache=(engine.kcache[i], engine.vcache[i])) for i, l in layers]), flops=2.0 * t * hid * 3 * hid)
+	record('prompt o', event_us([lambda l=l: l.self_attn.o_proj(xp) for l in rot]), flops=2.0 * t * hid * hid)
+	record('prompt gate/up', event_us([lambda l=l: l.mlp.intermediate(xp) for l in rot]), flops=4.0 * t * hid * inter)
+	record('prompt down', event_us([lambda l=l: l.mlp.down_proj(yp) for l in rot]), flops=2.0 * t * hid * inter)
+	q, k, v = (torch.randn((1, H, t, 128), device=dev).half() for _ in range(3))
+	mask = causal_mask(t, 0, dev)
+	record('prompt attention', event_us([lambda: F.scaled_dot_product_attention(q, k, v, attn_mask=mask)] * 4), flops=float(t) * (t + 1) * H * 256)
+	return out
+
+
+def befalix_arm(args):
+	"""Prints one JSON line: per size, prompt tokens/s and decode ms per step of a Befalix model (bf16 weights, random) and of a
+	4-bit LLaMA with the same hidden size, MLP, heads and number of layers, and every kernel's fraction of its roofline."""
+	import torch
+	import gptq_triton_b200 as G
+	from gptq_triton_b200 import _lib
+	from gptq_triton_b200.llama import LlamaConfig
+	torch.cuda.set_device(0)
+	dev = torch.device('cuda', 0)
+	hbm, source = measured_peaks()
+	peaks = ROOT / 'MEASURED_PEAKS.json'
+	tflops = float(json.load(open(peaks))['bf16_tflops']) if peaks.exists() else 1590.0
+	sampler = ClockSampler(0, None)
+	sampler.start()
+	cases = {}
+	for name, layers, hid, inter, H, D, R, V, C in BEFALIX_CASES:
+		if args.case and name not in args.case.split(','):
+			continue
+		max_seq = PROMPT + args.steps + 64
+		cfg = G.BefalixConfig.from_dict({'vocab': 32000, 'width': hid, 'norm': {'eps': 1e-6}, 'residual_mult': 1.0, 'logit_scale': 1.0, 'layers': [
+			{'type': 'latent_attention', 'mlp': {'kind': 'dense', 'ff': inter},
+			 'mixer': {'heads': H, 'dim': D, 'rot_dim': R, 'vdim': V, 'kv_rank': C, 'scale': (D + R) ** -0.5, 'rot': {'base': 10000.0, 'dims': R}}}] * layers})
+		model = G.synthetic_befalix(cfg, seed=1, device=dev)
+		engine = G.BefalixEngine(model, batch=1, max_seq=max_seq)
+		rate, ms = engine_rates(engine, cfg.vocab_size, args.steps)
+		nbytes = sum(b.numel() * b.element_size() for b in model.buffers()) + layers * (PROMPT + args.steps // 2) * model.layers[0].mixer.spec.row * 2
+		flops = PROMPT * 2.0 * sum(b.numel() for l in model.layers for n, b in l.named_buffers() if b.dim() == 2) + layers * float(PROMPT) * (PROMPT + 1) * H * (D + R + V)
+		rec = {'hidden': hid, 'intermediate': inter, 'heads': H, 'layers': layers,
+			   'befalix': {'prefill_tokens_s': round(rate), 'decode_ms_per_step': round(ms, 4), 'decode_tokens_s': round(1e3 / ms, 1), 'decode_frac_hbm': round(nbytes / ms / 1e6 / hbm, 3),
+						   'prefill_frac_tensor': round(flops * rate / PROMPT / 1e12 / tflops, 3), 'kernels': befalix_kernels(G, engine, hbm, tflops)}}
+		engine.close()
+		del engine, model
+		torch.cuda.empty_cache()
+		lcfg = LlamaConfig(hidden_size=hid, intermediate_size=inter, num_hidden_layers=layers, num_attention_heads=H, max_position_embeddings=max_seq)
+		model = G.synthetic_quantized_llama(lcfg, groupsize=GROUPSIZE, seed=1, device=dev)
+		engine = G.DecodeEngine(model, batch=1, max_seq=max_seq)
+		rate, ms = engine_rates(engine, lcfg.vocab_size, args.steps)
+		nbytes = layers * (quantised_bytes(hid, 4 * hid) + quantised_bytes(hid, 2 * inter) + quantised_bytes(inter, hid) + 2 * H * (PROMPT + args.steps // 2) * 256) + hid * 32000 * 2
+		flops = PROMPT * 2.0 * layers * (4 * hid * hid + 3 * hid * inter) + layers * float(PROMPT) * (PROMPT + 1) * H * 256
+		rec['llama_4bit'] = {'prefill_tokens_s': round(rate), 'decode_ms_per_step': round(ms, 4), 'decode_tokens_s': round(1e3 / ms, 1), 'decode_frac_hbm': round(nbytes / ms / 1e6 / hbm, 3),
+							 'prefill_frac_tensor': round(flops * rate / PROMPT / 1e12 / tflops, 3), 'kernels': llama_kernels(G, engine, hbm, tflops)}
+		engine.close()
+		del engine, model
+		torch.cuda.empty_cache()
+		cases[name] = rec
+	print(json.dumps({'workload': 'befalix', 'prompt': PROMPT, 'batch': 1, 'data': 'synthetic', 'weights': 'befalix bf16, llama 4-bit g128 (random)', 'hbm_gbs': hbm, 'bf16_tflops': tflops,
+					  'peak_source': source, 'kernel_status': _lib.kernel_status(dev), 'clocks': sampler.stop(), 'cases': cases}))
+
+
 def main():
 	ap = argparse.ArgumentParser()
 	ap.add_argument('--gpus', type=int, default=1)
@@ -861,7 +1136,9 @@ def main():
 	ap.add_argument('--no-parity', action='store_true', help='skip the greedy-decoding parity check before the timed region')
 	ap.add_argument('--no-prefill', action='store_true', help='skip the prefill-kernel record')
 	ap.add_argument('--config4', default='auto', choices=['auto', 'on', 'off'], help='also measure the 65B-architecture batch-16 configuration as a sub-record (auto: with 2 or more GPUs)')
-	ap.add_argument('--workload', default='llama7b', choices=['llama7b', 'llama65b-b16'], help='llama65b-b16: 65B architecture, batch 16 (tensor-parallel runs)')
+	ap.add_argument('--workload', default='llama7b', choices=['llama7b', 'llama65b-b16', 'befalix'],
+					help='llama65b-b16: 65B architecture, batch 16 (tensor-parallel runs); befalix: latent-attention models beside LLaMA at equal sizes')
+	ap.add_argument('--case', default='', help='befalix: sizes to run (2048, 4096, 8192), separated by commas')
 	ap.add_argument('--no-graph', action='store_true', help='do not capture the decode step in a CUDA graph')
 	ap.add_argument('--kernel-case', default=None, choices=['gateup', 'qkv', 'o', 'down', 'prefill', 'attn', 'lmhead', 'chain', 'qkvattn'], help='profiling aid: run a few launches of one kernel and exit')
 	ap.add_argument('--m', type=int, default=1, help='batch rows for --kernel-case')
@@ -869,6 +1146,8 @@ def main():
 	args = ap.parse_args()
 	if args.kernel_case:
 		kernel_case(args)
+	elif args.workload == 'befalix':
+		befalix_arm(args)
 	elif args.impl == 'reference':
 		reference_arm(args)
 	else:

@@ -6,6 +6,7 @@ Configuration, weight names and the engine; the mechanisms are in latent_attenti
 from __future__ import annotations
 
 import json
+import warnings
 from dataclasses import dataclass
 from pathlib import Path
 from typing import Dict, List, Optional, Sequence
@@ -44,7 +45,7 @@ class BefalixConfig:
 		for i, layer in enumerate(d['layers']):
 			if layer['type'] != 'latent_attention':
 				raise ValueError(f"layer {i}: mixer '{layer['type']}' is not part of this design")
-			m, mlp = layer['mixer'], layer['mlp']
+			m, mlp = layer['mixer'], layer.get('mlp')
 			if mlp is not None and mlp['kind'] != 'dense':
 				raise ValueError(f"layer {i}: feed-forward '{mlp['kind']}' is not part of this design")
 			spec = LatentAttentionSpec(heads=m['heads'], dim=m['dim'], rot_dim=m['rot_dim'], vdim=m['vdim'], kv_rank=m['kv_rank'], rot_base=m['rot']['base'],
@@ -108,8 +109,10 @@ class BefalixForCausalLM(nn.Module):
 		self.config, self.dtype = config, dtype
 		shapes = config.tensor_shapes()
 		missing, extra = sorted(set(shapes) - set(tensors)), sorted(set(tensors) - set(shapes))
-		if missing or extra:
-			raise ValueError(f'checkpoint tensors do not fit the configuration: missing {missing[:5]}, unexpected {extra[:5]}')
+		if missing:
+			raise ValueError(f'checkpoint tensors do not fit the configuration: missing {missing[:5]}')
+		if extra:
+			warnings.warn(f'checkpoint tensors that the configuration does not use: {extra[:5]}')
 
 		def get(name):
 			if tuple(tensors[name].shape) != shapes[name]:

@@ -50,7 +50,7 @@ static bool rows_bad(const RowPrep &r, int dtype) {
 static bool latent_bad(const LatentArgs &a, int dtype, bool attend) {
 	if (a.M < 1 || a.rows_per_seq < 1 || a.M % a.rows_per_seq || a.heads < 1 || a.dim < 16 || a.rot_dim < 16 || a.vdim < 16 || a.kv_rank < 16) return true;
 	if (a.dim % 16 || a.rot_dim % 16 || a.vdim % 16 || a.kv_rank % 16 || a.rot_dims % 2 || a.rot_dims < 0 || a.rot_dims > a.rot_dim) return true;
-	if (a.kv_width < 1 || a.kv_width > a.kv_rank || a.max_seq < 1 || a.splits < 1 || a.splits > 32 || (dtype != 0 && dtype != 1)) return true;
+	if (a.kv_width < 1 || a.kv_width > a.kv_rank || a.max_seq < 1 || a.splits < 1 || a.splits > 64 || (dtype != 0 && dtype != 1)) return true;
 	if (!a.pos || !a.cache || !a.status) return true;
 	if (a.kv_raw && (!a.kv_norm || !a.cos_t || !a.sin_t)) return true;
 	if (attend && (dtype ? !a.qa_f32 : !a.qa_hi || !a.qa_lo)) return true;

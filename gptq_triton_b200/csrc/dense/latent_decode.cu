@@ -21,6 +21,7 @@ namespace {
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int AB_R = 64;                 // latent columns per CTA of the absorb kernel
 constexpr int AB_M = 8;                  // query rows per pass
+constexpr int AB_V = 8;                  // float4 units of a latent per lane: kv_rank <= 1024
 constexpr int AB_G = DN_THREADS / 16;    // groups of 16 threads: each takes every 16th row of W_uk
 
 template <typename T>
@@ -31,40 +32,48 @@ __global__ void __launch_bounds__(DN_THREADS) latent_absorb_kernel(const LatentA
 	const int chunks = (p.kv_rank + AB_R - 1) / AB_R, R = p.kv_rank + p.rot_dim, hd = p.dim + p.rot_dim;
 	const int work = p.heads * chunks;
 	if ((int)blockIdx.x >= work) {
-		// ---- cache rows: RMS norm of the latent, rotation of the shared key part, both fp32 --------------------------
-		float *s_norm = &s_red[0][0][0];
-		const int m = (blockIdx.x - work) + blockIdx.y * (gridDim.x - work);
-		if (m >= p.M) {
-			pdl_wait();
-			pdl_trigger();
-			return;
-		}
+		// ---- cache rows: RMS norm of the latent, rotation of the shared key part, both fp32; a warp per row ----------
+		const int m = (((int)blockIdx.x - work) + blockIdx.y * ((int)gridDim.x - work)) * DN_WARPS + warp;
 		pdl_wait();
 		pdl_trigger();
+		if (m >= p.M) return;
 		const int pos = __ldcg(p.pos + m), seq = m / p.rows_per_seq;
 		if (pos < 0 || pos >= p.max_seq) {            // a position outside the cache is dropped
-			if (tid == 0) atomicExch(p.status, DN_BAD_POSITION);
+			if (lane == 0) atomicExch(p.status, DN_BAD_POSITION);
 			return;
 		}
 		const float *src = p.kv_raw + (size_t)m * R;
 		T *dst = reinterpret_cast<T *>(p.cache) + ((size_t)seq * p.max_seq + pos) * R;
+		float4 v[AB_V];
 		float s = 0.f;
-		for (int i = tid; i < p.kv_rank; i += DN_THREADS) {
-			const float v = __ldcg(src + i);
-			s = fmaf(v, v, s);
+#pragma unroll
+		for (int i = 0; i < AB_V; ++i) {
+			const int c = (i * 32 + lane) * 4;
+			if (i * 128 < p.kv_rank) {
+				v[i] = c < p.kv_rank ? __ldcg(reinterpret_cast<const float4 *>(src + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+				s = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, s))));
+			}
 		}
-		const float inv = 1.f / sqrtf(block_sum(s, s_norm) / (float)p.kv_width + p.eps);
-		for (int i = tid; i < p.kv_rank; i += DN_THREADS) Elem<T>::store(dst + i, __ldcg(src + i) * inv * __ldg(p.kv_norm + i));
-		for (int i = tid; i < p.rot_dim / 2; i += DN_THREADS) {
-			float u = __ldcg(src + p.kv_rank + 2 * i), v = __ldcg(src + p.kv_rank + 2 * i + 1);
+		const float inv = 1.f / sqrtf(warp_sum(s) / (float)p.kv_width + p.eps);
+#pragma unroll
+		for (int i = 0; i < AB_V; ++i) {
+			const int c = (i * 32 + lane) * 4;
+			if (c < p.kv_rank) {
+				const float4 w = __ldg(reinterpret_cast<const float4 *>(p.kv_norm + c));
+				Elem<T>::store4(dst + c, make_float4(v[i].x * inv * w.x, v[i].y * inv * w.y, v[i].z * inv * w.z, v[i].w * inv * w.w));
+			}
+		}
+		for (int i = lane; i < p.rot_dim / 2; i += 32) {
+			const float2 x = __ldcg(reinterpret_cast<const float2 *>(src + p.kv_rank) + i);
+			float u = x.x, w = x.y;
 			if (2 * i < p.rot_dims) {
 				const size_t t = (size_t)pos * (p.rot_dims / 2) + i;
-				const float c = __ldg(p.cos_t + t), sn = __ldg(p.sin_t + t), a = u * c - v * sn;
-				v = v * c + u * sn;
+				const float c = __ldg(p.cos_t + t), sn = __ldg(p.sin_t + t), a = u * c - w * sn;
+				w = w * c + u * sn;
 				u = a;
 			}
 			Elem<T>::store(dst + p.kv_rank + 2 * i, u);
-			Elem<T>::store(dst + p.kv_rank + 2 * i + 1, v);
+			Elem<T>::store(dst + p.kv_rank + 2 * i + 1, w);
 		}
 		return;
 	}
@@ -168,11 +177,12 @@ __global__ void __launch_bounds__(DN_THREADS) latent_attend_kernel(const LatentA
 	const int stages = at_stages(R);
 	const int m = blockIdx.z, h0 = blockIdx.y * AT_HEADS, split = blockIdx.x, seq = m / p.rows_per_seq;
 	const uint32_t sq = smem_u32(at_smem), sk = sq + 2 * AT_HEADS * row;
-	// positions are older than the previous launch (see the note on dependent launch), the newest cache rows are not
-	const int len = max(1, min(__ldcg(p.pos + m) + 1, p.max_seq));
-	int per = (len + p.splits - 1) / p.splits;
-	per = (per + AT_KEYS - 1) / AT_KEYS * AT_KEYS;
-	const int k_lo = min(split * per, len), k_hi = min(k_lo + per, len), ntiles = (k_hi - k_lo + AT_KEYS - 1) / AT_KEYS;
+	// positions are older than the previous launch (see the note on dependent launch), and so are the cache rows before the
+	// first position of this call
+	const int len = max(1, min(__ldcg(p.pos + m) + 1, p.max_seq)), fresh = __ldcg(p.pos + seq * p.rows_per_seq);
+	const int tiles = (len + AT_KEYS - 1) / AT_KEYS;
+	const int t_lo = (int)((long long)split * tiles / p.splits), ntiles = (int)((long long)(split + 1) * tiles / p.splits) - t_lo;
+	const int k_lo = t_lo * AT_KEYS, k_hi = min(k_lo + ntiles * AT_KEYS, len);
 	const bf16 *cache = reinterpret_cast<const bf16 *>(p.cache) + (size_t)seq * p.max_seq * R;
 	auto fetch = [&](int t) {            // keys beyond the range repeat the last one (their scores are masked)
 		const uint32_t dst = sk + (uint32_t)(t % stages) * AT_KEYS * row;
@@ -182,6 +192,8 @@ __global__ void __launch_bounds__(DN_THREADS) latent_attend_kernel(const LatentA
 			asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + k * row + c * 16), "l"(cache + (size_t)key * R + c * 8) : "memory");
 		}
 	};
+	int old = 0;                          // leading tiles that may be fetched ahead of the wait
+	while (old < min(ntiles, stages - 1) && k_lo + (old + 1) * AT_KEYS <= fresh) fetch(old++);
 	pdl_wait();
 	pdl_trigger();
 	for (int i = tid; i < 2 * AT_HEADS * chunks; i += DN_THREADS) {
@@ -190,7 +202,7 @@ __global__ void __launch_bounds__(DN_THREADS) latent_attend_kernel(const LatentA
 		asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(sq + (part * AT_HEADS + hh) * row + c * 16), "l"(src) : "memory");
 	}
 	for (int t = 0; t < stages - 1; ++t) {
-		if (t < ntiles) fetch(t);
+		if (t >= old && t < ntiles) fetch(t);
 		cp_async_commit();
 	}
 
@@ -212,16 +224,18 @@ __global__ void __launch_bounds__(DN_THREADS) latent_attend_kernel(const LatentA
 		__syncthreads();
 		const uint32_t kt = sk + (uint32_t)(t % stages) * AT_KEYS * row;
 		// scores of 16 heads x 8 keys; the two warps of a key group share the k range
-		float s[4] = {0.f, 0.f, 0.f, 0.f};
+		float s[4] = {0.f, 0.f, 0.f, 0.f}, sl[4] = {0.f, 0.f, 0.f, 0.f};      // high and remainder parts: two independent chains
 #pragma unroll 4
 		for (int k = kh; k < ks; k += 2) {
-			uint32_t a[4], b[2];
+			uint32_t a[4], al[4], b[2];
 			ldmatrix_x2(b, kt + b_off + k * 32);
 			ldmatrix_x4(a, sq + a_off + k * 32);
+			ldmatrix_x4(al, sq + AT_HEADS * row + a_off + k * 32);
 			mma16816_bf16(s, a[0], a[1], a[2], a[3], b[0], b[1]);
-			ldmatrix_x4(a, sq + AT_HEADS * row + a_off + k * 32);
-			mma16816_bf16(s, a[0], a[1], a[2], a[3], b[0], b[1]);
+			mma16816_bf16(sl, al[0], al[1], al[2], al[3], b[0], b[1]);
 		}
+#pragma unroll
+		for (int i = 0; i < 4; ++i) s[i] += sl[i];
 		const int c = kg * 8 + 2 * tig;
 		s_s[kh][gid][c] = s[0];
 		s_s[kh][gid][c + 1] = s[1];
@@ -383,24 +397,39 @@ constexpr int VA_ROWS = 32;              // value rows per CTA: four per warp
 constexpr int VA_SPLITS = 64;
 
 template <typename T>
-__global__ void __launch_bounds__(DN_THREADS) latent_value_kernel(const LatentArgs p) {
-	extern __shared__ __align__(16) float va_lat[];      // [kv_rank]
+__global__ void __launch_bounds__(DN_THREADS, 1) latent_value_kernel(const LatentArgs p) {
+	extern __shared__ __align__(16) float va_lat[];      // [2][kv_rank]
 	__shared__ float s_w[VA_SPLITS];
-	constexpr int PF = 2, RW = VA_ROWS / DN_WARPS;
+	constexpr int E = 16 / sizeof(T), PF = 2 * sizeof(T) / 2, RW = VA_ROWS / DN_WARPS, SB = 16;
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, head = blockIdx.y, m = blockIdx.z, v0 = blockIdx.x * VA_ROWS + warp * RW;
 	const T *uv = reinterpret_cast<const T *>(p.w_uv) + (size_t)head * p.vdim * p.kv_rank;
-	const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-	float4 w[RW][PF];
+	const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
+	uint4 w[RW][PF];                     // this warp's rows of W_uv, up to 512 columns
+	auto load_w = [&](int r, int i) {
+		const int c = (i * 32 + lane) * E;
+		return v0 + r < p.vdim && c < p.kv_rank ? ld_nc_v4(uv + (size_t)(v0 + r) * p.kv_rank + c) : zero4;
+	};
 #pragma unroll
 	for (int r = 0; r < RW; ++r)
 #pragma unroll
-		for (int i = 0; i < PF; ++i) {
-			const int c = (i * 32 + lane) * 4;
-			w[r][i] = (v0 + r < p.vdim && c < p.kv_rank) ? Elem<T>::load4(uv + (size_t)(v0 + r) * p.kv_rank + c) : zero;
-		}
+		for (int i = 0; i < PF; ++i) w[r][i] = load_w(r, i);
 	pdl_wait();
 	pdl_trigger();
 	const size_t base = ((size_t)m * p.heads + head) * p.splits;
+	const float gate = p.gate ? __ldcg(p.gate + (size_t)m * p.gate_ld + head) : 1.f;
+	// weighted sum over the ranges: half the threads take the even ranges, half the odd ones; the partials are requested before
+	// their weights are known
+	const int half = tid >> 7, nc = p.kv_rank >> 2;
+	const float4 *acc = reinterpret_cast<const float4 *>(p.part_acc + base * p.kv_rank);
+	float4 pre[SB];
+	auto load_acc = [&](int s0, int c) {
+#pragma unroll
+		for (int j = 0; j < SB; ++j) {
+			const int s = s0 + 2 * j + half;
+			pre[j] = s < p.splits && c < nc ? __ldcg(acc + (size_t)s * nc + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+		}
+	};
+	load_acc(0, tid & 127);
 	if (warp == 0) {
 		float2 ml[VA_SPLITS / 32];
 		float M = -INFINITY;
@@ -419,39 +448,56 @@ __global__ void __launch_bounds__(DN_THREADS) latent_value_kernel(const LatentAr
 		}
 		L = warp_sum(L);
 #pragma unroll
-		for (int i = 0; i < VA_SPLITS / 32; ++i)
-			if (i * 32 + lane < p.splits) s_w[i * 32 + lane] = ml[i].x / L;
+		for (int i = 0; i < VA_SPLITS / 32; ++i) s_w[i * 32 + lane] = ml[i].x / L;
 	}
 	__syncthreads();
-	for (int c = tid * 4; c < p.kv_rank; c += DN_THREADS * 4) {
-		float4 v = zero;
-		const float4 *src = reinterpret_cast<const float4 *>(p.part_acc + base * p.kv_rank + c);
-#pragma unroll 8
-		for (int s = 0; s < p.splits; ++s) {
-			const float4 a = __ldcg(src + (size_t)s * (p.kv_rank >> 2));
-			const float ws = s_w[s];
-			v.x = fmaf(a.x, ws, v.x);
-			v.y = fmaf(a.y, ws, v.y);
-			v.z = fmaf(a.z, ws, v.z);
-			v.w = fmaf(a.w, ws, v.w);
-		}
-		*reinterpret_cast<float4 *>(va_lat + c) = v;
-	}
-	__syncthreads();
-	const float gate = p.gate ? __ldcg(p.gate + (size_t)m * p.gate_ld + head) : 1.f;
+	for (int c = tid & 127; c < nc; c += 128) {
+		float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+		for (int s0 = 0; s0 < p.splits; s0 += 2 * SB) {
+			if (s0 || c >= 128) load_acc(s0, c);
 #pragma unroll
-	for (int r = 0; r < RW; ++r) {
-		float s = 0.f;
-		for (int i = 0; i * 128 < p.kv_rank; ++i) {
-			const int c = (i * 32 + lane) * 4;
-			if (c < p.kv_rank && v0 + r < p.vdim) {
-				const float4 a = i == 0 ? w[r][0] : i == 1 ? w[r][1] : Elem<T>::load4(uv + (size_t)(v0 + r) * p.kv_rank + c);
-				const float4 b = *reinterpret_cast<const float4 *>(va_lat + c);
-				s = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, s))));
+			for (int j = 0; j < SB; ++j) {
+				const float ws = s_w[min(s0 + 2 * j + half, VA_SPLITS - 1)];
+				v.x = fmaf(pre[j].x, ws, v.x);
+				v.y = fmaf(pre[j].y, ws, v.y);
+				v.z = fmaf(pre[j].z, ws, v.z);
+				v.w = fmaf(pre[j].w, ws, v.w);
 			}
 		}
-		s = warp_sum(s);
-		if (lane == 0 && v0 + r < p.vdim) Elem<T>::store(reinterpret_cast<T *>(p.out) + (size_t)m * p.out_ld + head * p.vdim + v0 + r, s * gate);
+		*reinterpret_cast<float4 *>(va_lat + half * p.kv_rank + 4 * c) = v;
+	}
+	__syncthreads();
+	float sum[RW] = {};
+	auto dot = [&](int r, int c, uint4 a) {
+		const float4 l0 = *reinterpret_cast<const float4 *>(va_lat + c), l1 = *reinterpret_cast<const float4 *>(va_lat + p.kv_rank + c);
+		if (sizeof(T) == 4) {
+			sum[r] = fmaf(__uint_as_float(a.x), l0.x + l1.x, fmaf(__uint_as_float(a.y), l0.y + l1.y, fmaf(__uint_as_float(a.z), l0.z + l1.z, fmaf(__uint_as_float(a.w), l0.w + l1.w, sum[r]))));
+		} else {
+			const float4 k0 = *reinterpret_cast<const float4 *>(va_lat + c + 4), k1 = *reinterpret_cast<const float4 *>(va_lat + p.kv_rank + c + 4);
+			const float4 f = Elem<bf16>::unpack(make_uint2(a.x, a.y)), g = Elem<bf16>::unpack(make_uint2(a.z, a.w));
+			sum[r] = fmaf(f.x, l0.x + l1.x, fmaf(f.y, l0.y + l1.y, fmaf(f.z, l0.z + l1.z, fmaf(f.w, l0.w + l1.w, sum[r]))));
+			sum[r] = fmaf(g.x, k0.x + k1.x, fmaf(g.y, k0.y + k1.y, fmaf(g.z, k0.z + k1.z, fmaf(g.w, k0.w + k1.w, sum[r]))));
+		}
+	};
+#pragma unroll
+	for (int i = 0; i < PF; ++i) {
+		const int c = (i * 32 + lane) * E;
+		if (c < p.kv_rank) {
+#pragma unroll
+			for (int r = 0; r < RW; ++r) dot(r, c, w[r][i]);
+		}
+	}
+	for (int i = PF; i * 32 * E < p.kv_rank; ++i) {
+		const int c = (i * 32 + lane) * E;
+		if (c < p.kv_rank) {
+#pragma unroll
+			for (int r = 0; r < RW; ++r) dot(r, c, load_w(r, i));
+		}
+	}
+#pragma unroll
+	for (int r = 0; r < RW; ++r) {
+		const float v = warp_sum(sum[r]);
+		if (lane == 0 && v0 + r < p.vdim) Elem<T>::store(reinterpret_cast<T *>(p.out) + (size_t)m * p.out_ld + head * p.vdim + v0 + r, v * gate);
 	}
 }
 
@@ -461,7 +507,7 @@ int latent_absorb_launch(const LatentArgs &p, bool queries, int dtype, cudaStrea
 	LatentArgs a = p;
 	if (!queries) a.heads = 0;                         // cache rows only
 	const int work = a.heads * ((a.kv_rank + AB_R - 1) / AB_R), gy = queries ? std::max(1, std::min(1024, (a.M + AB_M - 1) / AB_M)) : 1;
-	const int append = a.kv_raw ? (a.M + gy - 1) / gy : 0;
+	const int append = a.kv_raw ? (a.M + gy * DN_WARPS - 1) / (gy * DN_WARPS) : 0;
 	if (work + append == 0) return GPTQ_OK;
 	const size_t smem = (size_t)AB_M * a.dim * sizeof(float);
 	return dtype ? dn_launch(latent_absorb_kernel<float>, dim3(work + append, gy), dim3(DN_THREADS), smem, stream, a)
@@ -473,7 +519,7 @@ bool latent_attend_ok(int kv_rank, int rot_dim) { return kv_rank <= 1024 && rot_
 int latent_splits(int M, int heads, int max_seq, int dtype) {
 	const int per_row = dtype ? heads : (heads + AT_HEADS - 1) / AT_HEADS;
 	const int want = dn_sm_count() / std::max(1, M * per_row);
-	return std::max(1, std::min(std::min(32, want), (max_seq + AT_KEYS - 1) / AT_KEYS));
+	return std::max(1, std::min(std::min(VA_SPLITS, want), (max_seq + AT_KEYS - 1) / AT_KEYS));
 }
 
 int latent_attend_launch(const LatentArgs &p, int dtype, cudaStream_t stream) {
@@ -490,7 +536,7 @@ int latent_attend_launch(const LatentArgs &p, int dtype, cudaStream_t stream) {
 
 int latent_value_launch(const LatentArgs &p, int dtype, cudaStream_t stream) {
 	const dim3 grid((p.vdim + VA_ROWS - 1) / VA_ROWS, p.heads, p.M), block(DN_THREADS);
-	const size_t smem = (size_t)p.kv_rank * sizeof(float);
+	const size_t smem = 2 * (size_t)p.kv_rank * sizeof(float);
 	return dtype ? dn_launch(latent_value_kernel<float>, grid, block, smem, stream, p) : dn_launch(latent_value_kernel<bf16>, grid, block, smem, stream, p);
 }
 

@@ -144,10 +144,16 @@ __global__ void __launch_bounds__(NQ * 128 + 64, 1) latent_prefill_kernel(const 
 				const int a = j % pl.sk;
 				if (!wait(bar_fk + 8 * a, j / pl.sk)) return false;
 				uint32_t acc = 0;
-				for (int c = 0; c < nch; ++c) {
-					const int steps = min(64, c < pl.nd ? p.dim - 64 * c : p.rot_dim - 64 * (c - pl.nd)) >> 4;
-					const uint32_t qa = sq + i * k_bytes + c * LP_CHUNK, ka = sk + a * k_bytes + c * LP_CHUNK;
-					for (int k = 0; k < steps; ++k, acc = 1) umma_f16(tmem + i * LP_T, smem_desc_sw128(qa + k * 32), smem_desc_sw128(ka + k * 32), id_qk, acc);
+				// a descriptor advances by 2 (32 bytes) per K step; one thread issues everything, so the loop must stay short
+				uint64_t qd = smem_desc_sw128(sq + i * k_bytes), kd = smem_desc_sw128(sk + a * k_bytes);
+				for (int c = 0; c < nch; ++c, qd += LP_CHUNK / 16, kd += LP_CHUNK / 16) {
+					const int steps = (c < pl.nd ? p.dim - 64 * c : p.rot_dim - 64 * (c - pl.nd)) >> 4;
+#pragma unroll
+					for (int k = 0; k < 4; ++k)
+						if (k < steps) {
+							umma_f16(tmem + i * LP_T, qd + 2 * k, kd + 2 * k, id_qk, acc);
+							acc = 1;
+						}
 				}
 				umma_commit(bar_s + 8 * i);
 				return true;
@@ -155,10 +161,16 @@ __global__ void __launch_bounds__(NQ * 128 + 64, 1) latent_prefill_kernel(const 
 			auto pv = [&](int i, int j) {
 				const int b = j % pl.sv;
 				if (!wait(bar_p + 8 * i, j) || !wait(bar_fv + 8 * b, j / pl.sv)) return false;
-				const uint32_t d = tmem + NQ * LP_T + i * p.vdim, va = sv + b * v_bytes;
+				const uint32_t d = tmem + NQ * LP_T + i * p.vdim, pa = tmem + i * LP_T;
+				const uint64_t vd = smem_desc_sw128(sv + b * v_bytes), vd1 = vd + (v_bytes >> 5);
+				uint32_t acc = j ? 1u : 0u;
+#pragma unroll
 				for (int part = 0; part < 2; ++part)
-					for (int k = 0; k < 8; ++k)
-						umma_f16_ts(d, tmem + i * LP_T + part * 64 + k * 8, smem_desc_sw128(va + (k >> 2) * (v_bytes / 2) + (k & 3) * 32), id_pv, (j | part | k) ? 1u : 0u);
+#pragma unroll
+					for (int k = 0; k < 8; ++k) {
+						umma_f16_ts(d, pa + part * 64 + k * 8, (k < 4 ? vd : vd1) + 2 * (k & 3), id_pv, acc);
+						acc = 1;
+					}
 				umma_commit(bar_o + 8 * i);
 				return true;
 			};
@@ -284,7 +296,7 @@ bool lp_plan(int nq, int dim, int rot_dim, int vdim, LpPlan *out) {
 	pl.nr = (rot_dim + 63) / 64;
 	if (vdim > 256 || nq * (LP_T + vdim) > 512) return false;
 	const size_t k = (size_t)(pl.nd + pl.nr) * LP_CHUNK, v = (size_t)vdim * 256;
-	const int opts[3][2] = {{2, 2}, {2, 1}, {1, 1}};
+	const int opts[4][2] = {{2, 2}, {1, 2}, {2, 1}, {1, 1}};      // V is needed sooner after its release than K
 	for (auto &o : opts) {
 		pl.sk = o[0];
 		pl.sv = o[1];

@@ -98,11 +98,7 @@ class LatentAttention(nn.Module):
 		e.q_out, e.q_f32, e.kv_out, e.gate_out, e.status = ptr(q), int(not expanded), ptr(kv), ptr(gate), _dense.status_ptr(control)
 		x = project_stream(stream, self.w_in, e, control)
 
-		a = _dense.Latent()
-		a.M, a.rows_per_seq, a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, a.kv_width = M, rows_per_seq, H, self.D, self.R, self.V, self.C, s.kv_rank
-		a.rot_dims, a.max_seq, a.splits, a.scale, a.eps = s.rot_dims, max_seq, 1, s.scale, eps
-		a.pos, a.cos_t, a.sin_t, a.cache, a.status = ptr(pos), ptr(cos), ptr(sin), ptr(cache), _dense.status_ptr(control)
-		a.kv_raw, a.kv_norm = ptr(kv), ptr(self.kv_norm)
+		a = self.arguments(cache, pos, rows_per_seq, tables, eps, control, kv)
 		lib, code, st = _dense.lib(), _dense.DTYPE_CODE[dt], stream_ptr(dev)
 		out = torch.empty((M, H * self.V), dtype=dt, device=dev)
 		if expanded:
@@ -113,20 +109,35 @@ class LatentAttention(nn.Module):
 				lo = b * rows_per_seq
 				self._expanded(q[lo:lo + rows_per_seq], cache[b, :S], gate[lo:lo + rows_per_seq], out[lo:lo + rows_per_seq], start, control)
 		else:
-			splits = lib.dense_latent_splits(M, H, max_seq if start is None else start + rows_per_seq, code)
-			qa = torch.empty((1 if f32 else 2, M, H, s.row), dtype=dt, device=dev)
-			ml = torch.empty((M, H, splits, 2), dtype=torch.float32, device=dev)
-			acc = torch.empty((M, H, splits, self.C), dtype=torch.float32, device=dev)
-			a.splits, a.q, a.w_uk, a.w_uv, a.part_ml, a.part_acc = splits, ptr(q), ptr(self.w_uk), ptr(self.w_uv), ptr(ml), ptr(acc)
-			if f32:
-				a.qa_f32 = ptr(qa)
-			else:
-				a.qa_hi, a.qa_lo = ptr(qa[0]), ptr(qa[1])
-			a.gate, a.gate_ld, a.out, a.out_ld = ptr(gate), self.G, ptr(out), out.stride(0)
+			scratch = self.absorbed_buffers(a, q, gate, out, max_seq if start is None else start + rows_per_seq)      # noqa: F841 (alive until the launches)
 			_dense.check(lib.dense_latent_absorb(ctypes.byref(a), code, st), 'dense_latent_absorb')
 			_dense.check(lib.dense_latent_attend(ctypes.byref(a), code, st), 'dense_latent_attend')
 			_dense.check(lib.dense_latent_value(ctypes.byref(a), code, st), 'dense_latent_value')
 		return x, linear(out, self.w_o, control)
+
+	def arguments(self, cache, pos, rows_per_seq: int, tables, eps: float, control, kv) -> '_dense.Latent':
+		"""Sizes, positions, tables and cache of a call; kv: raw rows to append, or None."""
+		s, a = self.spec, _dense.Latent()
+		a.M, a.rows_per_seq, a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, a.kv_width = pos.numel(), rows_per_seq, s.heads, self.D, self.R, self.V, self.C, s.kv_rank
+		a.rot_dims, a.max_seq, a.splits, a.scale, a.eps = s.rot_dims, cache.shape[1], 1, s.scale, eps
+		a.pos, a.cos_t, a.sin_t, a.cache, a.status = ptr(pos), ptr(tables[0]), ptr(tables[1]), ptr(cache), _dense.status_ptr(control)
+		a.kv_raw, a.kv_norm = ptr(kv), ptr(self.kv_norm)
+		return a
+
+	def absorbed_buffers(self, a: '_dense.Latent', q, gate, out, keys: int):
+		"""Scratch of the absorbed form for up to `keys` visible positions, entered into `a`; returns what must stay alive."""
+		dev, f32 = q.device, out.dtype == torch.float32
+		a.splits = _dense.lib().dense_latent_splits(a.M, a.heads, keys, _dense.DTYPE_CODE[out.dtype])
+		qa = torch.empty((1 if f32 else 2, a.M, a.heads, self.spec.row), dtype=out.dtype, device=dev)
+		ml = torch.empty((a.M, a.heads, a.splits, 2), dtype=torch.float32, device=dev)
+		acc = torch.empty((a.M, a.heads, a.splits, self.C), dtype=torch.float32, device=dev)
+		a.q, a.w_uk, a.w_uv, a.part_ml, a.part_acc = ptr(q), ptr(self.w_uk), ptr(self.w_uv), ptr(ml), ptr(acc)
+		if f32:
+			a.qa_f32 = ptr(qa)
+		else:
+			a.qa_hi, a.qa_lo = ptr(qa[0]), ptr(qa[1])
+		a.gate, a.gate_ld, a.out, a.out_ld = ptr(gate), self.G, ptr(out), out.stride(0)
+		return qa, ml, acc
 
 	def _expanded(self, q, rows, gate, out, start: int, control):
 		"""One sequence: keys and (transposed) values of the cached rows [S, row], then the tensor-core attention kernel."""

@@ -5,6 +5,7 @@ from pathlib import Path
 import pytest
 
 ROOT = Path(__file__).resolve().parent.parent
+sys.path.insert(0, str(Path(__file__).resolve().parent))          # helper modules beside the tests
 if str(ROOT) not in sys.path:
 	sys.path.insert(0, str(ROOT))
 
