@@ -5,7 +5,7 @@ from gptq_triton_b200.befalix import BefalixConfig, BefalixEngine, BefalixForCau
 from oracle import latent_oracle as O
 
 # error of the logits (mean taken off, rms over the vocabulary, relative to the logits' spread) that rounding causes
-LIMIT = {torch.float32: 1e-5, torch.bfloat16: 2.5e-2}
+LIMIT = {torch.float32: 1e-5, torch.bfloat16: 4.5e-2}
 
 
 def layer(heads, dim, rot_dim, vdim, kv_rank, ff, base=10000.0, scale=None, kv_from=None, rot_dims=None):

@@ -424,6 +424,6 @@ def test_mistakes_that_the_comparisons_must_see():
 		'gate': changed(edit_w=lambda w: w.update({'l0.mix.g': -w['l0.mix.g']})),
 		'latent norm': changed(edit_w=lambda w: w.update({'l1.mix.dkv.norm': torch.ones_like(w['l1.mix.dkv.norm'])})),
 		'layer scale': changed(edit_w=lambda w: w.update({'l2.ls2': torch.ones_like(w['l2.ls2'])})),
-		'norm bias': changed(edit_w=lambda w: w.update({'l3.norm1.b': torch.zeros_like(w['l3.norm1.b'])})),
+		'norm bias': changed(edit_w=lambda w: w.update({'l3.norm1.b': -w['l3.norm1.b']})),
 	}
 	assert all(v > 1.5 * LM.LIMIT[B16] for v in cases.values()), cases
