@@ -686,6 +686,30 @@ def kernel_case(args):
 		torch.cuda.synchronize()
 		print(json.dumps({'kernel_case': 'prefill', 'M': int(x.shape[0]), 'launches': 3}))
 		return
+	if args.kernel_case in ('latent-prefill', 'latent-decode'):
+		# latent attention, 2048 tokens: the tensor-core prompt kernel alone / decode steps of two layers (about 2 GB on the device)
+		import ctypes
+		from gptq_triton_b200 import _dense
+		if args.kernel_case == 'latent-prefill':
+			ctl = _dense.control_buffer(dev)
+			t, H, D, R, V, C = PROMPT, args.heads, 128, 64, 128, 512
+			bf = lambda *shape: torch.randn(shape, device=dev).bfloat16()
+			q, k, vt, c, g, o = bf(t, H * (D + R)), bf(t, H * D), bf(H * V, t), bf(t, C + R), torch.rand((t, H), device=dev), bf(t, H * V)
+			p = _dense.LatentPrefill()
+			p.t, p.start, p.S, p.heads, p.dim, p.rot_dim, p.vdim, p.kv_rank, p.scale = t, 0, t, H, D, R, V, C, (D + R) ** -0.5
+			p.q, p.k, p.vt, p.ldv, p.cache, p.gate, p.gate_ld = q.data_ptr(), k.data_ptr(), vt.data_ptr(), t, c.data_ptr(), g.data_ptr(), H
+			p.out, p.out_ld, p.status = o.data_ptr(), H * V, _dense.status_ptr(ctl).value
+			for _ in range(3):
+				_dense.check(_dense.lib().dense_latent_prefill(ctypes.byref(p), None), 'dense_latent_prefill')
+		else:
+			cfg = befalix_config(G, 2, 4096, 11008, 32, 128, 64, 128, 512, vocab=2048)
+			e = G.BefalixEngine(G.synthetic_befalix(cfg, device=dev), 1, PROMPT + 16, use_graph=False)
+			e.feed(torch.randint(0, cfg.vocab_size, (1, PROMPT), generator=torch.Generator().manual_seed(3)))
+			for _ in range(3):
+				e.step()
+		torch.cuda.synchronize()
+		print(json.dumps({'kernel_case': args.kernel_case}))
+		return
 	if args.kernel_case == 'chain':
 		# the persistent decode-step kernel on four layers of the 7B architecture after a 2048-token prompt (about 1 GB on
 		# the device): a few steps, nothing else; also prints the step time of both engines
@@ -995,6 +1019,9 @@ def befalix_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: 
 	record('decode down', graph_us([lambda w=w: linear(act, w, ctl) for w in copies(down)]), esz(down))
 	logits = torch.empty((1, (cfg.vocab_size + 15) // 16 * 16), device=dev)
 	record('decode logits', graph_us([lambda w=w: project_stream(s1, w, epilogue(_dense.EPI_LOGITS, logits), ctl, keep=False, final=m.norm) for w in copies(m.embed)]), esz(m.embed))
+	# the attention block as a whole (LLaMA runs it as one kernel)
+	parts = ['decode in-projection', 'decode absorb + cache row', 'decode attention', 'decode merge + value', 'decode out-projection']
+	record('decode attention block (sum)', sum(out[n]['us'] for n in parts), esz(mx.w_in) + esz(mx.w_uk) + esz(mx.w_uv) + esz(mx.w_o) + S * spec.row * 2)
 	# ---- prompt of t tokens ----
 	xs = torch.randn((t, W), device=dev)
 	st = Stream(cfg.width, W, cfg.norm_eps, x=xs, y=torch.randn((t, W), device=dev), gain=layer.mixer_norm.gain, shift=layer.mixer_norm.shift)
@@ -1076,6 +1103,12 @@ def llama_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: in
 	return out
 
 
+def befalix_config(G, layers, hid, inter, H, D, R, V, C, vocab=32000):
+	layer = {'type': 'latent_attention', 'mlp': {'kind': 'dense', 'ff': inter},
+			 'mixer': {'heads': H, 'dim': D, 'rot_dim': R, 'vdim': V, 'kv_rank': C, 'scale': (D + R) ** -0.5, 'rot': {'base': 10000.0, 'dims': R}}}
+	return G.BefalixConfig.from_dict({'vocab': vocab, 'width': hid, 'norm': {'eps': 1e-6}, 'residual_mult': 1.0, 'logit_scale': 1.0, 'layers': [layer] * layers})
+
+
 def befalix_arm(args):
 	"""Prints one JSON line: per size, prompt tokens/s and decode ms per step of a Befalix model (bf16 weights, random) and of a
 	4-bit LLaMA with the same hidden size, MLP, heads and number of layers, and every kernel's fraction of its roofline."""
@@ -1095,9 +1128,7 @@ def befalix_arm(args):
 		if args.case and name not in args.case.split(','):
 			continue
 		max_seq = PROMPT + args.steps + 64
-		cfg = G.BefalixConfig.from_dict({'vocab': 32000, 'width': hid, 'norm': {'eps': 1e-6}, 'residual_mult': 1.0, 'logit_scale': 1.0, 'layers': [
-			{'type': 'latent_attention', 'mlp': {'kind': 'dense', 'ff': inter},
-			 'mixer': {'heads': H, 'dim': D, 'rot_dim': R, 'vdim': V, 'kv_rank': C, 'scale': (D + R) ** -0.5, 'rot': {'base': 10000.0, 'dims': R}}}] * layers})
+		cfg = befalix_config(G, layers, hid, inter, H, D, R, V, C)
 		model = G.synthetic_befalix(cfg, seed=1, device=dev)
 		engine = G.BefalixEngine(model, batch=1, max_seq=max_seq)
 		rate, ms = engine_rates(engine, cfg.vocab_size, args.steps)
@@ -1140,9 +1171,9 @@ def main():
 					help='llama65b-b16: 65B architecture, batch 16 (tensor-parallel runs); befalix: latent-attention models beside LLaMA at equal sizes')
 	ap.add_argument('--case', default='', help='befalix: sizes to run (2048, 4096, 8192), separated by commas')
 	ap.add_argument('--no-graph', action='store_true', help='do not capture the decode step in a CUDA graph')
-	ap.add_argument('--kernel-case', default=None, choices=['gateup', 'qkv', 'o', 'down', 'prefill', 'attn', 'lmhead', 'chain', 'qkvattn'], help='profiling aid: run a few launches of one kernel and exit')
+	ap.add_argument('--kernel-case', default=None, choices=['gateup', 'qkv', 'o', 'down', 'prefill', 'attn', 'lmhead', 'chain', 'qkvattn', 'latent-prefill', 'latent-decode'], help='profiling aid: run a few launches of one kernel and exit')
 	ap.add_argument('--m', type=int, default=1, help='batch rows for --kernel-case')
-	ap.add_argument('--heads', type=int, default=32, help='heads for --kernel-case attn')
+	ap.add_argument('--heads', type=int, default=32, help='heads for --kernel-case attn and latent-prefill')
 	args = ap.parse_args()
 	if args.kernel_case:
 		kernel_case(args)

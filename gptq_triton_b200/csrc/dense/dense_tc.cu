@@ -4,7 +4,8 @@
 // Persistent, one CTA per SM, output tiles of 128 rows x BN columns, K in blocks of 64:
 //   warp 0      TMA producer (one thread): X tile and W tile of a K-block into a ring of stages, 128-byte swizzle
 //   warp 1      tensor-memory owner and MMA issuer (one thread): four tcgen05.mma of K = 16 per block
-//   warps 2-5   epilogue: tcgen05.ld of the accumulators, then the fused epilogue of the projection
+//   warps 2-9   epilogue, two warps per lane quarter and half the columns each: tcgen05.ld of the accumulators, then the fused
+//               epilogue of the projection
 // The accumulators are double-buffered in tensor memory, so the epilogue of a tile runs under the MMAs of the next one.
 // Every wait is bounded; one that runs out sets the status word and the kernel unwinds.
 #include <algorithm>
@@ -19,7 +20,7 @@ int dense_tensor_map(const void *base, long long rows, long long cols, long long
 
 namespace {
 
-constexpr int TD_BM = 128, TD_BK = 64, TD_THREADS = 192;
+constexpr int TD_BM = 128, TD_BK = 64, TD_EPI = 256, TD_THREADS = 64 + TD_EPI;
 constexpr int TD_A_BYTES = TD_BM * TD_BK * 2;
 constexpr uint32_t TD_SPIN = 1u << 24;
 constexpr size_t TD_SMEM = 226 * 1024;
@@ -53,7 +54,7 @@ __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_co
 		}
 		for (int s = 0; s < 2; ++s) {
 			mbar_init(bar_acc + 8 * s, 1);
-			mbar_init(bar_free + 8 * s, 128);
+			mbar_init(bar_free + 8 * s, TD_EPI);
 		}
 		*s_abort = 0;
 		fence_mbar_init();
@@ -116,7 +117,7 @@ __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_co
 		}
 		__syncwarp();
 	} else {
-		const int q = warp & 3;
+		const int q = warp & 3, half = (warp - 2) >> 2;
 		int lt = 0;
 		bool ok = true;
 		for (int t = blockIdx.x; t < ntiles && ok; t += gridDim.x, ++lt) {
@@ -130,7 +131,7 @@ __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_co
 			tc_fence_after();
 			const uint32_t t0 = tmem + b * BN + ((uint32_t)(q * 32) << 16);
 #pragma unroll 1
-			for (int c = 0; c < BN; c += 32) {
+			for (int c = 32 * half; c < BN; c += 64) {
 				float v[2][16];
 				tmem_ld16(t0 + c, v[0]);
 				tmem_ld16(t0 + c + 16, v[1]);
