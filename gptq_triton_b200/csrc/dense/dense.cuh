@@ -39,6 +39,16 @@ template <> struct Elem<bf16> {
 		o.y = *reinterpret_cast<uint32_t *>(&b);
 		*reinterpret_cast<uint2 *>(p) = o;
 	}
+	static __device__ __forceinline__ void store8(bf16 *p, const float *v) {
+		uint4 o;
+		uint32_t *w = reinterpret_cast<uint32_t *>(&o);
+#pragma unroll
+		for (int i = 0; i < 4; ++i) {
+			__nv_bfloat162 a = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+			w[i] = *reinterpret_cast<uint32_t *>(&a);
+		}
+		*reinterpret_cast<uint4 *>(p) = o;
+	}
 	static __device__ __forceinline__ float ldcg(const bf16 *p) {
 		return __uint_as_float((uint32_t)__ldcg(reinterpret_cast<const unsigned short *>(p)) << 16);
 	}
@@ -47,6 +57,10 @@ template <> struct Elem<bf16> {
 template <> struct Elem<float> {
 	static __device__ __forceinline__ float4 load4(const float *p) { return __ldg(reinterpret_cast<const float4 *>(p)); }
 	static __device__ __forceinline__ void store4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+	static __device__ __forceinline__ void store8(float *p, const float *v) {
+		store4(p, make_float4(v[0], v[1], v[2], v[3]));
+		store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
+	}
 	static __device__ __forceinline__ float ldcg(const float *p) { return __ldcg(p); }
 	static __device__ __forceinline__ void store(float *p, float v) { *p = v; }
 };
@@ -286,13 +300,13 @@ __device__ __forceinline__ void epi_16(const DenseEpi &e, int m, int n, const fl
 	} else if (e.mode == DENSE_EPI_T) {
 		T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
 #pragma unroll
-		for (int i = 0; i < 4; ++i) Elem<T>::store4(o + 4 * i, make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]));
+		for (int i = 0; i < 2; ++i) Elem<T>::store8(o + 8 * i, v + 8 * i);
 	} else if (e.mode == DENSE_EPI_SILU) {          // eight gate columns, then the eight up columns of the same outputs
 		T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + (n >> 1);
+		float r[8];
 #pragma unroll
-		for (int i = 0; i < 2; ++i)
-			Elem<T>::store4(o + 4 * i, make_float4(silu_exact(v[4 * i]) * v[8 + 4 * i], silu_exact(v[4 * i + 1]) * v[9 + 4 * i],
-												   silu_exact(v[4 * i + 2]) * v[10 + 4 * i], silu_exact(v[4 * i + 3]) * v[11 + 4 * i]));
+		for (int i = 0; i < 8; ++i) r[i] = silu_exact(v[i]) * v[8 + i];
+		Elem<T>::store8(o, r);
 	} else {          // QKV: a group of 16 columns lies in one head, on one side of rot_at, in one section
 		if (n < e.n_q) {
 			const int off = n % e.head_dim - e.rot_at;
