@@ -173,7 +173,7 @@ def register_status_buffer(buf: torch.Tensor):
 def kernel_status(device=None) -> int:
 	"""OR of the status words that the decode kernels keep in their workspaces (0 = healthy;
 	1 = a TMA / bulk load never completed within the bounded wait; 2 = shared memory misaligned;
-	3 = a wait inside the tensor-core kernel ran out; 4 = position outside the rotary table / cache;
+	3 = a wait inside the tensor-core kernel ran out; 4 = position outside the rotary table / cache, or token outside the vocabulary;
 	5 = a peer never arrived in the fused tensor-parallel all-reduce; 6 = a split-K partial sum never arrived;
 	7 = a grid barrier of the persistent decode-step kernel timed out)."""
 	st = 0
