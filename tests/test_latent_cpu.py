@@ -60,7 +60,7 @@ def test_arguments_are_refused_on_the_host(lib):
 	assert lib.dense_latent_prefill(None, None) == -1
 	assert lib.dense_decode_rows_ok(8, 4096, 0) == 1 and lib.dense_decode_rows_ok(9, 4096, 0) == 0
 	assert lib.dense_decode_rows_ok(8, 22016, 0) == 0 and lib.dense_decode_rows_ok(1, 22016, 1) == 1
-	assert lib.dense_latent_prefill_ok(128, 64, 128) == 1 and lib.dense_latent_prefill_ok(256, 64, 256) == 1 and lib.dense_latent_prefill_ok(1024, 64, 128) == 0
+	assert lib.dense_latent_prefill_ok(128, 64, 128) == 1 and lib.dense_latent_prefill_ok(192, 64, 256) == 1 and lib.dense_latent_prefill_ok(1024, 64, 128) == 0
 
 
 def test_config_reads_every_constant_and_checks_shared_caches():
