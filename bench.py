@@ -976,7 +976,7 @@ def befalix_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: 
 		out[name] = r
 
 	x1 = torch.randn((1, W), device=dev)
-	s1 = Stream(cfg.width, W, cfg.norm_eps, x=x1, y=torch.randn((1, W), device=dev), gain=layer.mixer_norm.gain, shift=layer.mixer_norm.shift)
+	s1 = layer.mixer_norm.join(Stream(cfg.width, W, cfg.norm_eps), x1, torch.randn((1, W), device=dev))
 	pos = torch.full((1,), ctx, dtype=torch.int32, device=dev)
 	q = torch.randn((1, H * (D + R)), device=dev)
 	gate = torch.rand((1, mx.G), device=dev)
@@ -1015,7 +1015,7 @@ def befalix_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: 
 	record('decode out-projection', graph_us([lambda w=w: linear(attn, w, ctl) for w in copies(mx.w_o)]), esz(mx.w_o))
 	gu, down = layer.mlp.gate_up, layer.mlp.down
 	act = torch.empty((1, down.shape[1]), dtype=m.dtype, device=dev)
-	record('decode gate/up', graph_us([lambda w=w: project_stream(s1, w, epilogue(_dense.EPI_SILU, act), ctl) for w in copies(gu)]), esz(gu))
+	record('decode gate/up', graph_us([lambda w=w: project_stream(s1, w, layer.mlp.gated(act), ctl) for w in copies(gu)]), esz(gu))
 	record('decode down', graph_us([lambda w=w: linear(act, w, ctl) for w in copies(down)]), esz(down))
 	logits = torch.empty((1, (cfg.vocab_size + 15) // 16 * 16), device=dev)
 	record('decode logits', graph_us([lambda w=w: project_stream(s1, w, epilogue(_dense.EPI_LOGITS, logits), ctl, keep=False, final=m.norm) for w in copies(m.embed)]), esz(m.embed))
@@ -1024,7 +1024,7 @@ def befalix_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: 
 	record('decode attention block (sum)', sum(out[n]['us'] for n in parts), esz(mx.w_in) + esz(mx.w_uk) + esz(mx.w_uv) + esz(mx.w_o) + S * spec.row * 2)
 	# ---- prompt of t tokens ----
 	xs = torch.randn((t, W), device=dev)
-	st = Stream(cfg.width, W, cfg.norm_eps, x=xs, y=torch.randn((t, W), device=dev), gain=layer.mixer_norm.gain, shift=layer.mixer_norm.shift)
+	st = layer.mixer_norm.join(Stream(cfg.width, W, cfg.norm_eps), xs, torch.randn((t, W), device=dev))
 	record('prompt rows (norm, residual)', graph_us([lambda: prepare_rows(st, ctl, m.dtype, True)] * 4), t * W * (4 + 4 + 4 + 2))
 	h = torch.randn((t, W), device=dev).to(m.dtype)
 	posp = torch.arange(t, dtype=torch.int32, device=dev)
@@ -1048,7 +1048,7 @@ def befalix_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: 
 	record('prompt attention', us, flops=float(t) * (t + 1) * H * (D + R + V))
 	gemm('prompt out-projection', [lambda w=w: linear(op, w, ctl) for w in copies(mx.w_o)], mx.w_o)
 	actp = torch.empty((t, down.shape[1]), dtype=m.dtype, device=dev)
-	gemm('prompt gate/up', [lambda w=w: matmul(h, w, epilogue(_dense.EPI_SILU, actp), ctl) for w in copies(gu)], gu)
+	gemm('prompt gate/up', [lambda w=w: matmul(h, w, layer.mlp.gated(actp), ctl) for w in copies(gu)], gu)
 	gemm('prompt down', [lambda w=w: linear(actp, w, ctl) for w in copies(down)], down)
 	return out
 

@@ -7,6 +7,7 @@ from . import fused_mlp, quant_linear
 from .fused_attention import QuantLlamaAttention, make_quant_attn, qkv_rope
 from .fused_mlp import QuantLlamaMLP, gateup_silu, make_fused_mlp, triton_llama_mlp_4
 from .befalix import BefalixConfig, BefalixEngine, BefalixForCausalLM, load_befalix, synthetic_befalix
+from .lifinex import LifinexConfig, LifinexEngine, LifinexForCausalLM, load_lifinex, synthetic_lifinex
 from .llama import DecodeEngine, LlamaConfig, LlamaForCausalLM
 from .loader import autotune_warmup, load_quant, save_quant, synthetic_quantized_llama
 from .registry import ARCHITECTURES, load_model, make_engine
@@ -19,6 +20,7 @@ __all__ = [
 	'QuantLlamaMLP', 'make_fused_mlp', 'triton_llama_mlp_4', 'gateup_silu',
 	'load_model', 'make_engine', 'ARCHITECTURES',
 	'BefalixConfig', 'BefalixEngine', 'BefalixForCausalLM', 'load_befalix', 'synthetic_befalix',
+	'LifinexConfig', 'LifinexEngine', 'LifinexForCausalLM', 'load_lifinex', 'synthetic_lifinex',
 	'dequantize', 'unpack_qweight', 'unpack_qzeros',
 	'quant_linear', 'fused_mlp',
 ]

@@ -14,7 +14,10 @@ from ._lib import GptqB200Error, ptr, register_status_buffer, require_cuda, stre
 LIB_PATH = Path(__file__).resolve().parent / 'libdense_b200.so'
 CONTROL_BYTES = 16384
 
-EPI_F32, EPI_T, EPI_SILU, EPI_QKV, EPI_LOGITS = range(5)
+EPI_F32, EPI_T, EPI_GATED, EPI_QKV, EPI_LOGITS, EPI_TABLE = range(6)
+ACT_CODE = {'silu': 0, 'gelu_tanh': 1}
+NORM_NONE, NORM_LAYER, NORM_RMS = range(3)
+MAX_NORM_GROUPS = 256
 DTYPE_CODE = {torch.bfloat16: 0, torch.float32: 1}
 
 _P, _I = c_void_p, c_int
@@ -22,14 +25,15 @@ _P, _I = c_void_p, c_int
 
 class Rows(ctypes.Structure):
 	_fields_ = [('x_in', _P), ('x_out', _P), ('y', _P), ('gain', _P), ('shift', _P), ('fin_w', _P), ('fin_b', _P), ('table', _P), ('token', _P),
-				('vocab', c_int64), ('width', _I), ('ld', _I), ('eps', c_float), ('status', _P)]
+				('vocab', c_int64), ('pos_table', _P), ('pos', _P), ('max_pos', _I), ('y_norm', _I), ('fin_norm', _I), ('fin_groups', _I), ('width', _I), ('ld', _I), ('eps', c_float), ('status', _P)]
 
 
 class Epilogue(ctypes.Structure):
 	_fields_ = [('mode', _I), ('out', _P), ('ldo', c_int64), ('scale', c_float),
 				('n_q', _I), ('head_dim', _I), ('rot_at', _I), ('rot_dims', _I), ('n_kv', _I), ('n_gate', _I),
 				('cos_t', _P), ('sin_t', _P), ('pos', _P), ('max_pos', _I), ('q_out', _P), ('q_f32', _I), ('kv_out', _P), ('gate_out', _P), ('status', _P),
-				('best', _P), ('ticket', _P), ('tok', _P), ('pos_inout', _P)]
+				('best', _P), ('ticket', _P), ('tok', _P), ('pos_inout', _P), ('act', _I), ('tab', _P), ('tab_ld', c_int64), ('tab_rows', c_int64), ('tab_col', _I),
+				('tab_token', _P)]
 
 
 class Latent(ctypes.Structure):
@@ -42,6 +46,18 @@ class Latent(ctypes.Structure):
 class LatentPrefill(ctypes.Structure):
 	_fields_ = [(n, _I) for n in ('t', 'start', 'S', 'heads', 'dim', 'rot_dim', 'vdim', 'kv_rank')] + [
 		('scale', c_float), ('q', _P), ('k', _P), ('vt', _P), ('ldv', c_int64), ('cache', _P), ('gate', _P), ('gate_ld', _I), ('out', _P), ('out_ld', c_int64), ('status', _P)]
+
+
+class Gqa(ctypes.Structure):
+	_fields_ = [(n, _I) for n in ('M', 'rows_per_seq', 'heads', 'kv_heads', 'maps', 'dim', 'vdim', 'dim_true', 'vdim_true', 'max_seq', 'splits')] + [
+		(n, c_float) for n in ('scale', 'cap', 'eps', 'lambda_', 'out_mul')] + [
+		('out_norm', _I), ('pos', _P), ('raw', _P), ('raw_ld', c_int64), ('q_norm', _P), ('k_norm', _P), ('k_cache', _P), ('v_cache', _P), ('q_hi', _P), ('q_lo', _P),
+		('q_f32', _P), ('part_ml', _P), ('part_acc', _P), ('out', _P), ('out_ld', c_int64), ('status', _P)]
+
+
+class Ssm(ctypes.Structure):
+	_fields_ = [(n, _I) for n in ('M', 'rows_per_seq', 'heads', 'vdim', 'state', 'groups', 'taps', 'z_at', 'conv_at', 'dt_at', 'conv_ld')] + [
+		('raw_ld', c_int64)] + [(n, _P) for n in ('raw', 'pos', 'conv_w', 'conv_b', 'dt_bias', 'a', 'd', 'ring', 's', 'u', 'out')] + [('out_ld', c_int64), ('status', _P)]
 
 
 _SIGNATURES = {
@@ -57,6 +73,13 @@ _SIGNATURES = {
 	'dense_latent_value': (c_int, [_P, _I, _P]),
 	'dense_latent_prefill_ok': (c_int, [_I, _I, _I]),
 	'dense_latent_prefill': (c_int, [_P, _P]),
+	'dense_gqa_splits': (c_int, [_I, _I, _I, _I, _I, _I]),
+	'dense_gqa_append': (c_int, [_P, _I, _P]),
+	'dense_gqa_attend': (c_int, [_P, _I, _P]),
+	'dense_gqa_merge': (c_int, [_P, _I, _P]),
+	'dense_ssm_step': (c_int, [_P, _P]),
+	'dense_ssm_conv': (c_int, [_P, _P]),
+	'dense_ssm_scan': (c_int, [_P, _P]),
 }
 
 _lib: Optional[ctypes.CDLL] = None

@@ -1,24 +1,20 @@
 """Befalix: decoder-only language models with latent attention (per-head output gates, layers that may share an earlier
 layer's cached rows), SiLU-gated MLPs, post-norm residual sublayers with LayerNorm and layer scale, tied output embedding.
 
-Configuration, weight names and the engine; the mechanisms are in latent_attention.py and dense.py.
+Configuration, weight names and the engine; the mechanisms are in latent_attention.py and dense.py,
+what designs with dense weights share in dense_model.py.
 """
 from __future__ import annotations
 
 import json
-import warnings
 from dataclasses import dataclass
-from pathlib import Path
-from typing import Dict, List, Optional, Sequence
+from typing import Dict, List, Optional
 
 import torch
 import torch.nn as nn
 
-from . import _dense
-from ._lib import ptr
-from .cache import StaticCache
-from .dense import DenseMLP, LayerNorm, PostNorm, Stream, epilogue, pad_to, padded, project_stream
-from .engine import StaticEngine
+from .dense import DenseMLP, LayerNorm, PostNorm, Stream
+from .dense_model import DenseCausalLM, DenseEngine, load_checkpoint
 from .latent_attention import LatentAttention, LatentAttentionSpec, interleaved_rope_tables
 
 ARCHITECTURE = 'Befalix'
@@ -98,36 +94,25 @@ class BefalixLayer(nn.Module):
 			self.mlp_norm = PostNorm(get('norm2'), get('norm2.b'), get('ls2'), config.residual_mult)
 
 
-class BefalixForCausalLM(nn.Module):
+class BefalixForCausalLM(DenseCausalLM):
 	"""Inference weights in the kernels' layout, built from a checkpoint's tensors."""
 	architecture = ARCHITECTURE
 
 	def __init__(self, config: BefalixConfig, tensors: Dict[str, torch.Tensor], dtype: torch.dtype = torch.bfloat16, device='cuda'):
-		super().__init__()
-		if dtype not in _dense.DTYPE_CODE:
-			raise ValueError(f'{ARCHITECTURE} runs in bfloat16 or float32, not {dtype}')
-		self.config, self.dtype = config, dtype
-		shapes = config.tensor_shapes()
-		missing, extra = sorted(set(shapes) - set(tensors)), sorted(set(tensors) - set(shapes))
-		if missing:
-			raise ValueError(f'checkpoint tensors do not fit the configuration: missing {missing[:5]}')
-		if extra:
-			warnings.warn(f'checkpoint tensors that the configuration does not use: {extra[:5]}')
-
-		def get(name):
-			if tuple(tensors[name].shape) != shapes[name]:
-				raise ValueError(f'{name} has shape {tuple(tensors[name].shape)}, the configuration needs {shapes[name]}')
-			return tensors[name].to(device=device, dtype=dtype)
-		self.register_buffer('embed', pad_to(get('embed'), config.vocab_size, padded(config.width)).contiguous())
-		self.layers = nn.ModuleList([BefalixLayer(layer, config, lambda n, i=i: get(f'l{i}.{n}')) for i, layer in enumerate(config.layers)])
+		super().__init__(config, tensors, dtype, device)
+		get = self.reader(tensors, device)
+		self.register_buffer('embed', self.table(get('embed')))
+		self.layers = nn.ModuleList([BefalixLayer(layer, config, self.reader(tensors, device, f'l{i}.')) for i, layer in enumerate(config.layers)])
 		self.norm = LayerNorm(get('final.norm'), get('final.norm.b'))
+
+	@property
+	def head(self) -> torch.Tensor:
+		return self.embed
 
 
 def load_befalix(checkpoint, device='cuda', dtype: Optional[torch.dtype] = None) -> BefalixForCausalLM:
 	"""Checkpoint directory with config.json and model.safetensors."""
-	from safetensors.torch import load_file
-	ck = Path(checkpoint)
-	return BefalixForCausalLM(BefalixConfig.from_json(ck / 'config.json'), load_file(str(ck / 'model.safetensors')), dtype or torch.bfloat16, device)
+	return load_checkpoint(BefalixForCausalLM, BefalixConfig, checkpoint, device, dtype)
 
 
 @torch.no_grad()
@@ -147,27 +132,18 @@ def synthetic_befalix(config: BefalixConfig, seed: int = 0, device='cuda', dtype
 	return BefalixForCausalLM(config, tensors, dtype, device)
 
 
-class BefalixEngine(StaticEngine):
+class BefalixEngine(DenseEngine):
 	"""Static cache of latent rows; a layer that shares another's reads that layer's rows.  A decode step of one sequence is
 	seven kernels per layer plus one for the logits and the greedy choice."""
-	max_portion = 8192
 
 	def __init__(self, model: BefalixForCausalLM, batch: int, max_seq: int, use_graph: bool = True):
-		super().__init__(model, batch, max_seq, model.embed.device, use_graph)
-		cfg = model.config
-		self.cfg = cfg
-		mixers = [layer.mixer for layer in cfg.layers]
-		self.cache = StaticCache([m.kv_from if m.kv_from is not None else {'rows': (max_seq, m.row)} for m in mixers], batch, model.dtype, self.device)
+		mixers = [layer.mixer for layer in model.config.layers]
+		super().__init__(model, batch, max_seq, [m.kv_from if m.kv_from is not None else {'rows': (max_seq, m.row)} for m in mixers], use_graph)
 		tables = {}
 		for m in mixers:
 			if (m.rot_base, m.rot_dims) not in tables:
 				tables[m.rot_base, m.rot_dims] = interleaved_rope_tables(m.rot_base, m.rot_dims, max_seq, self.device)
 		self.tables = [tables[m.rot_base, m.rot_dims] for m in mixers]
-		# arrival counter and candidates of the greedy choice (8 bytes per row from byte 256), status word at the end
-		self.control = _dense.control_buffer(self.device)
-		if 256 + 8 * batch > _dense.CONTROL_BYTES - 8:
-			raise ValueError(f'batch {batch} is larger than the control buffer provides for')
-		self._taps = None          # tests: a list that receives the residual stream after every layer
 
 	def _layers(self, token: torch.Tensor, pos: torch.Tensor, rows_per_seq: int, start: Optional[int]) -> Stream:
 		m, cfg = self.model, self.cfg
@@ -178,35 +154,5 @@ class BefalixEngine(StaticEngine):
 			if layer.mlp is not None:
 				x, y = layer.mlp(stream, self.control)
 				stream = layer.mlp_norm.join(stream, x, y)
-			if self._taps is not None:
-				from .dense import prepare_rows
-				self._taps.append(prepare_rows(stream, self.control, m.dtype, True)[1][:, :cfg.width].clone())
+			self._tap(stream)
 		return stream
-
-	def _head(self, stream: Stream, greedy: bool = False) -> torch.Tensor:
-		"""Final norm and tied output projection: fp32 logits [M, vocab] (a view of padded rows).  greedy: the same kernel
-		also writes self.tok and advances self.pos."""
-		m, cfg = self.model, self.cfg
-		logits = torch.empty((stream.rows, padded(cfg.vocab_size)), dtype=torch.float32, device=self.device)
-		e = epilogue(_dense.EPI_LOGITS, logits, cfg.logit_scale)
-		if greedy:
-			e.ticket, e.best, e.tok, e.pos_inout = self.control.data_ptr(), self.control.data_ptr() + 256, ptr(self.tok), ptr(self.pos)
-		project_stream(stream, m.embed, e, self.control, keep=False, final=m.norm)
-		return logits[:, :cfg.vocab_size]
-
-	def _portion(self, input_ids: torch.Tensor, start: int, want: Sequence[int]) -> Optional[torch.Tensor]:
-		b, t = input_ids.shape
-		pos = torch.arange(start, start + t, device=self.device, dtype=torch.int32).repeat(b)
-		stream = self._layers(input_ids.reshape(-1).contiguous(), pos, t, start)
-		if not want:
-			return None
-		index = (torch.arange(b, device=self.device)[:, None] * t + torch.tensor(list(want), device=self.device)[None, :]).reshape(-1)
-		return self._head(stream.take(index)).reshape(b, len(want), -1)
-
-	def _step_body(self):
-		stream = self._layers(self.tok.view(-1), self.pos.view(-1), 1, None)
-		greedy = bool(_dense.lib().dense_decode_rows_ok(self.batch, stream.ld, _dense.DTYPE_CODE[self.model.dtype]))
-		self.logits = self._head(stream, greedy).view(self.batch, 1, -1)
-		if not greedy:
-			self.tok.copy_(self.logits.argmax(-1))
-			self.pos.add_(1)

@@ -52,6 +52,7 @@ template <> struct Elem<bf16> {
 	static __device__ __forceinline__ float ldcg(const bf16 *p) {
 		return __uint_as_float((uint32_t)__ldcg(reinterpret_cast<const unsigned short *>(p)) << 16);
 	}
+	static __device__ __forceinline__ float ldg(const bf16 *p) { return __uint_as_float((uint32_t)__ldg(reinterpret_cast<const unsigned short *>(p)) << 16); }
 	static __device__ __forceinline__ void store(bf16 *p, float v) { *p = __float2bfloat16_rn(v); }
 };
 template <> struct Elem<float> {
@@ -62,6 +63,7 @@ template <> struct Elem<float> {
 		store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
 	}
 	static __device__ __forceinline__ float ldcg(const float *p) { return __ldcg(p); }
+	static __device__ __forceinline__ float ldg(const float *p) { return __ldg(p); }
 	static __device__ __forceinline__ void store(float *p, float v) { *p = v; }
 };
 
@@ -111,23 +113,23 @@ __device__ __forceinline__ float block_sum(float v, float *slot) {
 
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
+// 0.5 z (1 + tanh u) with 1 + tanh u = 2 / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh(float z) { return z / (1.f + expf(-1.5957691216057308f * fmaf(0.044715f * z, z * z, z))); }
+__device__ __forceinline__ float activation(int act, float z) { return act == DENSE_ACT_GELU ? gelu_tanh(z) : silu_exact(z); }
 
 // ---- row preparation ------------------------------------------------------------------------------------------------
-// Forms row m of the residual stream and the normalised or plain row that the next projection reads, all in fp32:
-//   x = table[token]                                      (start of a step), or
-//   x = x_in + (y - mean(y)) / sqrt(var(y) + eps) * gain + shift      (post-norm residual; gain and shift carry the
-//                                                          norm's affine part, the layer scale and the residual multiplier)
-//   out = x, or LayerNorm(x) * fin_w + fin_b               (final norm)
+// Forms row m of the residual stream and the row that the next projection reads, all in fp32:
+//   x = table[token] (+ pos_table[pos])                   (start of a step), or
+//   x = x_in + norm(y) * gain + shift                     (residual; norm: none, LayerNorm or RMS norm; gain and shift carry
+//                                                          the norm's affine part, layer scales and residual multipliers)
+//   out = x, or norm(x) * fin_w + fin_b                   (LayerNorm, RMS norm, RMS norm of equal parts)
 // Rows are padded with zeros from `width` to `ld` columns.
 using RowPrep = dense_rows_t;
 
 constexpr int RP_REGS = 4;              // float4 units of a row that a thread keeps in registers
+constexpr int RP_SMEM = 4 * DN_WARPS + DENSE_MAX_NORM_GROUPS;      // floats of shared memory that a preparation uses
 
-template <typename T>
-__device__ __forceinline__ float4 rp_x(const RowPrep &p, size_t base, int u) {
-	if (p.table) return Elem<T>::load4(reinterpret_cast<const T *>(p.table) + base + 4 * u);
-	return __ldcg(reinterpret_cast<const float4 *>(p.x_in + base) + u);
-}
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 __device__ __forceinline__ float rp_sqdev(float4 v, float mean, int c, int width) {
 	float s = 0.f;
 	const float a = v.x - mean, b = v.y - mean, d = v.z - mean, e = v.w - mean;
@@ -137,18 +139,66 @@ __device__ __forceinline__ float rp_sqdev(float4 v, float mean, int c, int width
 	if (c + 3 < width) s = fmaf(e, e, s);
 	return s;
 }
-__device__ __forceinline__ float4 rp_affine(float4 x, float4 y, float mean, float inv, float4 g, float4 s) {
-	return make_float4(x.x + fmaf((y.x - mean) * inv, g.x, s.x), x.y + fmaf((y.y - mean) * inv, g.y, s.y), x.z + fmaf((y.z - mean) * inv, g.z, s.z),
-					   x.w + fmaf((y.w - mean) * inv, g.w, s.w));
+// (v - mean) * inv * gain + shift, gain and shift optional
+__device__ __forceinline__ float4 rp_affine(float4 v, float mean, float inv, const float *gain, const float *shift, int u) {
+	const float4 g = gain ? __ldg(reinterpret_cast<const float4 *>(gain) + u) : make_float4(1.f, 1.f, 1.f, 1.f);
+	const float4 s = shift ? __ldg(reinterpret_cast<const float4 *>(shift) + u) : make_float4(0.f, 0.f, 0.f, 0.f);
+	return make_float4(fmaf((v.x - mean) * inv, g.x, s.x), fmaf((v.y - mean) * inv, g.y, s.y), fmaf((v.z - mean) * inv, g.z, s.z), fmaf((v.w - mean) * inv, g.w, s.w));
+}
+
+// The RMS norm of equal parts of row x (global memory, `width` columns): a warp sums a share of a part, the shares of a part
+// are added in order.  inv: fin_groups (or DN_WARPS, if that is more) floats of shared memory.
+template <typename T>
+__device__ void norm_parts(const RowPrep &p, const float *x, T *dst, float *inv) {
+	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n = p.width / p.fin_groups;
+	const int shares = p.fin_groups >= DN_WARPS ? 1 : DN_WARPS / p.fin_groups, per = (n + shares - 1) / shares;
+	for (int i = warp; i < p.fin_groups * shares; i += DN_WARPS) {
+		const int g = i / shares, c0 = (i - g * shares) * per, c1 = min(c0 + per, n);
+		float s = 0.f;
+#pragma unroll 8
+		for (int c = c0 + lane; c < c1; c += 32) {
+			const float v = __ldcg(x + (size_t)g * n + c);
+			s = fmaf(v, v, s);
+		}
+		s = warp_sum(s);
+		if (lane == 0) inv[i] = s;
+	}
+	__syncthreads();
+	float f = 0.f;
+	if (tid < p.fin_groups) {
+		float s = 0.f;
+		for (int i = 0; i < shares; ++i) s += inv[tid * shares + i];
+		f = 1.f / sqrtf(s / (float)n + p.eps);
+	}
+	__syncthreads();
+	if (tid < p.fin_groups) inv[tid] = f;
+	__syncthreads();
+	for (int u = tid; u < p.ld >> 2; u += DN_THREADS) {
+		const float4 v = __ldcg(reinterpret_cast<const float4 *>(x) + u);
+		const int c = 4 * u, g = min(c / n, p.fin_groups - 1), edge = (g + 1) * n;
+		const float f0 = inv[g];
+		float4 w = p.fin_w ? __ldg(reinterpret_cast<const float4 *>(p.fin_w) + u) : make_float4(1.f, 1.f, 1.f, 1.f);
+		if (edge >= c + 4 || g == p.fin_groups - 1) {
+			w.x *= f0; w.y *= f0; w.z *= f0; w.w *= f0;
+		} else {                          // parts that end inside the unit (they may be shorter than one)
+			auto at = [&](int i) { return inv[min((c + i) / n, p.fin_groups - 1)]; };
+			w.x *= f0; w.y *= at(1); w.z *= at(2); w.w *= at(3);
+		}
+		Elem<T>::store4(dst + c, make_float4(v.x * w.x, v.y * w.y, v.z * w.z, v.w * w.w));
+	}
 }
 
 // The whole CTA (256 threads) prepares one row.  dst: where the T row goes (global or shared memory); write_x: also store
-// the new residual row.  red: 4 * DN_WARPS floats of shared memory, reused across rows (callers synchronise between rows).
+// the new residual row.  red: RP_SMEM floats of shared memory, reused across rows (callers synchronise between rows).
 template <typename T>
 __device__ void prepare_row(const RowPrep &p, int m, T *dst, bool write_x, float *red) {
 	const int tid = threadIdx.x, nu = p.ld >> 2;
-	size_t xb = (size_t)m * p.ld;
+	size_t xb = (size_t)m * p.ld, pb = 0;
 	const size_t yb = xb;
+	if (p.fin_groups > 1) {
+		norm_parts<T>(p, p.x_in + xb, dst, red + 4 * DN_WARPS);
+		return;
+	}
 	if (p.table) {
 		long long t = __ldcg(reinterpret_cast<const long long *>(p.token) + m);
 		if (t < 0 || t >= p.vocab) {          // never index the table out of range
@@ -156,50 +206,63 @@ __device__ void prepare_row(const RowPrep &p, int m, T *dst, bool write_x, float
 			t = 0;
 		}
 		xb = (size_t)t * p.ld;
+		if (p.pos_table) {
+			int q = __ldcg(p.pos + m);
+			if (q < 0 || q >= p.max_pos) {
+				if (tid == 0) atomicExch(p.status, DN_BAD_POSITION);
+				q = 0;
+			}
+			pb = (size_t)q * p.ld;
+		}
 	}
+	auto read_x = [&](int u) {
+		if (!p.table) return __ldcg(reinterpret_cast<const float4 *>(p.x_in + xb) + u);
+		const float4 v = Elem<T>::load4(reinterpret_cast<const T *>(p.table) + xb + 4 * u);
+		return p.pos_table ? add4(v, Elem<T>::load4(reinterpret_cast<const T *>(p.pos_table) + pb + 4 * u)) : v;
+	};
 	float4 x[RP_REGS], y[RP_REGS];
 	const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
 	for (int i = 0; i < RP_REGS; ++i) {
 		const int u = tid + i * DN_THREADS;
-		x[i] = u < nu ? rp_x<T>(p, xb, u) : zero;
+		x[i] = u < nu ? read_x(u) : zero;
 		y[i] = (p.y && u < nu) ? __ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u) : zero;
 	}
 	const float inv_n = 1.f / (float)p.width;
-	float mean = 0.f, inv = 0.f;
-	if (p.y) {
+	float mean = 0.f, inv = 1.f;
+	if (p.y && p.y_norm != DENSE_NORM_NONE) {
 		float s = 0.f;
+		if (p.y_norm == DENSE_NORM_LAYER) {
 #pragma unroll
-		for (int i = 0; i < RP_REGS; ++i) s += (y[i].x + y[i].y) + (y[i].z + y[i].w);
-		for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) {
-			const float4 v = __ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u);
-			s += (v.x + v.y) + (v.z + v.w);
+			for (int i = 0; i < RP_REGS; ++i) s += (y[i].x + y[i].y) + (y[i].z + y[i].w);
+			for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) {
+				const float4 v = __ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u);
+				s += (v.x + v.y) + (v.z + v.w);
+			}
+			mean = block_sum(s, red) * inv_n;
+			s = 0.f;
 		}
-		mean = block_sum(s, red) * inv_n;
-		s = 0.f;
 #pragma unroll
 		for (int i = 0; i < RP_REGS; ++i) s += rp_sqdev(y[i], mean, 4 * (tid + i * DN_THREADS), p.width);
 		for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS)
 			s += rp_sqdev(__ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u), mean, 4 * u, p.width);
 		inv = 1.f / sqrtf(block_sum(s, red + DN_WARPS) * inv_n + p.eps);
 	}
-	auto next_x = [&](float4 xv, float4 yv, int u) {
-		if (!p.y) return xv;
-		return rp_affine(xv, yv, mean, inv, __ldg(reinterpret_cast<const float4 *>(p.gain) + u), __ldg(reinterpret_cast<const float4 *>(p.shift) + u));
-	};
+	auto next_x = [&](float4 xv, float4 yv, int u) { return p.y ? add4(xv, rp_affine(yv, mean, inv, p.gain, p.shift, u)) : xv; };
+	const bool norm = p.fin_norm != DENSE_NORM_NONE;
 #pragma unroll
 	for (int i = 0; i < RP_REGS; ++i) {
 		const int u = tid + i * DN_THREADS;
 		if (u < nu) {
 			x[i] = next_x(x[i], y[i], u);
 			if (write_x) reinterpret_cast<float4 *>(p.x_out + yb)[u] = x[i];
-			if (!p.fin_w) Elem<T>::store4(dst + 4 * u, x[i]);
+			if (!norm) Elem<T>::store4(dst + 4 * u, x[i]);
 		}
 	}
 	auto far_x = [&](int u) {          // units beyond the registers are formed again where they are needed
-		return next_x(rp_x<T>(p, xb, u), p.y ? __ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u) : zero, u);
+		return next_x(read_x(u), p.y ? __ldcg(reinterpret_cast<const float4 *>(p.y + yb) + u) : zero, u);
 	};
-	if (!p.fin_w) {
+	if (!norm) {
 		for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) {
 			const float4 v = far_x(u);
 			if (write_x) reinterpret_cast<float4 *>(p.x_out + yb)[u] = v;
@@ -207,16 +270,18 @@ __device__ void prepare_row(const RowPrep &p, int m, T *dst, bool write_x, float
 		}
 		return;
 	}
-	// final norm over the new row (x_out must not be x_in when rows are longer than the registers hold: the row is read again)
-	float s = 0.f;
+	// norm of the new row (x_out must not be x_in when rows are longer than the registers hold: the row is read again)
+	float s = 0.f, fm = 0.f;
+	if (p.fin_norm == DENSE_NORM_LAYER) {
 #pragma unroll
-	for (int i = 0; i < RP_REGS; ++i) s += (x[i].x + x[i].y) + (x[i].z + x[i].w);
-	for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) {
-		const float4 v = far_x(u);
-		s += (v.x + v.y) + (v.z + v.w);
+		for (int i = 0; i < RP_REGS; ++i) s += (x[i].x + x[i].y) + (x[i].z + x[i].w);
+		for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) {
+			const float4 v = far_x(u);
+			s += (v.x + v.y) + (v.z + v.w);
+		}
+		fm = block_sum(s, red + 2 * DN_WARPS) * inv_n;
+		s = 0.f;
 	}
-	const float fm = block_sum(s, red + 2 * DN_WARPS) * inv_n;
-	s = 0.f;
 #pragma unroll
 	for (int i = 0; i < RP_REGS; ++i) s += rp_sqdev(x[i], fm, 4 * (tid + i * DN_THREADS), p.width);
 	for (int u = tid + RP_REGS * DN_THREADS; u < nu; u += DN_THREADS) s += rp_sqdev(far_x(u), fm, 4 * u, p.width);
@@ -229,14 +294,13 @@ __device__ void prepare_row(const RowPrep &p, int m, T *dst, bool write_x, float
 			v = far_x(u);
 			if (write_x) reinterpret_cast<float4 *>(p.x_out + yb)[u] = v;
 		}
-		const float4 w = __ldg(reinterpret_cast<const float4 *>(p.fin_w) + u), b = __ldg(reinterpret_cast<const float4 *>(p.fin_b) + u);
-		Elem<T>::store4(dst + 4 * u, make_float4(fmaf((v.x - fm) * fi, w.x, b.x), fmaf((v.y - fm) * fi, w.y, b.y), fmaf((v.z - fm) * fi, w.z, b.z),
-												 fmaf((v.w - fm) * fi, w.w, b.w)));
+		v = rp_affine(v, fm, fi, p.fin_w, p.fin_b, u);
+		Elem<T>::store4(dst + 4 * u, v);
 	}
 }
 
 // ---- epilogues ------------------------------------------------------------------------------------------------------
-// Every fp32 result of a projection belongs to a pair of columns (n, n + 1), n even (SILU: gate column and up column).
+// Every fp32 result of a projection belongs to a pair of columns (n, n + 1), n even (GATED: gate column and up column).
 using DenseEpi = dense_epilogue_t;
 
 __device__ __forceinline__ int epi_pos(const DenseEpi &e, int m) {
@@ -246,6 +310,12 @@ __device__ __forceinline__ int epi_pos(const DenseEpi &e, int m) {
 		pos = 0;
 	}
 	return pos;
+}
+
+// row of the per-token table; a token outside it has been reported when the embedding was looked up
+__device__ __forceinline__ long long epi_tab_row(const DenseEpi &e, int m) {
+	const long long t = __ldcg(reinterpret_cast<const long long *>(e.tab_token) + m);
+	return t < 0 || t >= e.tab_rows ? 0 : t;
 }
 
 // One pair of results of row m.  T is the activation type.
@@ -260,6 +330,13 @@ __device__ __forceinline__ void epi_pair(const DenseEpi &e, int m, int n, float 
 			T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
 			Elem<T>::store(o, a);
 			Elem<T>::store(o + 1, b);
+			break;
+		}
+		case DENSE_EPI_TABLE: {
+			T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
+			const T *t = reinterpret_cast<const T *>(e.tab) + epi_tab_row(e, m) * e.tab_ld + e.tab_col + n;
+			Elem<T>::store(o, activation(e.act, a) * Elem<T>::ldg(t));
+			Elem<T>::store(o + 1, activation(e.act, b) * Elem<T>::ldg(t + 1));
 			break;
 		}
 		case DENSE_EPI_QKV: {
@@ -301,11 +378,25 @@ __device__ __forceinline__ void epi_16(const DenseEpi &e, int m, int n, const fl
 		T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
 #pragma unroll
 		for (int i = 0; i < 2; ++i) Elem<T>::store8(o + 8 * i, v + 8 * i);
-	} else if (e.mode == DENSE_EPI_SILU) {          // eight gate columns, then the eight up columns of the same outputs
+	} else if (e.mode == DENSE_EPI_TABLE) {
+		T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
+		const T *t = reinterpret_cast<const T *>(e.tab) + epi_tab_row(e, m) * e.tab_ld + e.tab_col + n;
+		float r[16];
+#pragma unroll
+		for (int i = 0; i < 4; ++i) {
+			const float4 f = Elem<T>::load4(t + 4 * i);
+			r[4 * i] = activation(e.act, v[4 * i]) * f.x;
+			r[4 * i + 1] = activation(e.act, v[4 * i + 1]) * f.y;
+			r[4 * i + 2] = activation(e.act, v[4 * i + 2]) * f.z;
+			r[4 * i + 3] = activation(e.act, v[4 * i + 3]) * f.w;
+		}
+#pragma unroll
+		for (int i = 0; i < 2; ++i) Elem<T>::store8(o + 8 * i, r + 8 * i);
+	} else if (e.mode == DENSE_EPI_GATED) {         // eight gate columns, then the eight up columns of the same outputs
 		T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + (n >> 1);
 		float r[8];
 #pragma unroll
-		for (int i = 0; i < 8; ++i) r[i] = silu_exact(v[i]) * v[8 + i];
+		for (int i = 0; i < 8; ++i) r[i] = activation(e.act, v[i]) * v[8 + i];
 		Elem<T>::store8(o, r);
 	} else {          // QKV: a group of 16 columns lies in one head, on one side of rot_at, in one section
 		if (n < e.n_q) {

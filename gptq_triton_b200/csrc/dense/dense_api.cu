@@ -3,7 +3,9 @@
 #include <set>
 #include <utility>
 
+#include "gqa.cuh"
 #include "latent.cuh"
+#include "ssm.cuh"
 
 namespace gptq {
 
@@ -41,10 +43,13 @@ int dn_smem_opt_in(const void *kernel, size_t bytes) {
 static bool rows_bad(const RowPrep &r, int dtype) {
 	if (r.width < 1 || r.ld < r.width || r.ld % 16 != 0 || !(r.eps >= 0.f) || !r.status) return true;
 	if (r.table ? !r.token || r.vocab < 1 : !r.x_in) return true;
-	if (r.y && (!r.gain || !r.shift)) return true;
-	if (r.fin_w && !r.fin_b) return true;
+	if (r.pos_table && (!r.table || !r.pos || r.max_pos < 1)) return true;
+	if (r.y_norm < DENSE_NORM_NONE || r.y_norm > DENSE_NORM_RMS || r.fin_norm < DENSE_NORM_NONE || r.fin_norm > DENSE_NORM_RMS) return true;
+	if ((r.fin_w || r.fin_b) && r.fin_norm == DENSE_NORM_NONE) return true;
+	if (r.fin_groups < 1 || r.fin_groups > DENSE_MAX_NORM_GROUPS) return true;
+	if (r.fin_groups > 1 && (r.fin_norm != DENSE_NORM_RMS || r.width % r.fin_groups || r.table || r.y || r.x_out || r.fin_b)) return true;
 	if (r.x_out && r.x_out == r.x_in) return true;
-	return !aligned16(r.x_in) || !aligned16(r.x_out) || !aligned16(r.y) || !aligned16(r.gain) || !aligned16(r.shift) || !aligned16(r.fin_w) || !aligned16(r.fin_b) || !aligned16(r.table);
+	return !aligned16(r.pos_table) || !aligned16(r.x_in) || !aligned16(r.x_out) || !aligned16(r.y) || !aligned16(r.gain) || !aligned16(r.shift) || !aligned16(r.fin_w) || !aligned16(r.fin_b) || !aligned16(r.table);
 }
 
 static bool latent_bad(const LatentArgs &a, int dtype, bool attend) {
@@ -55,6 +60,21 @@ static bool latent_bad(const LatentArgs &a, int dtype, bool attend) {
 	if (a.kv_raw && (!a.kv_norm || !a.cos_t || !a.sin_t)) return true;
 	if (attend && (dtype ? !a.qa_f32 : !a.qa_hi || !a.qa_lo)) return true;
 	return false;
+}
+
+static bool gqa_bad(const GqaArgs &a, int dtype) {
+	if (a.M < 1 || a.rows_per_seq < 1 || a.M % a.rows_per_seq || a.heads < 1 || a.kv_heads < 1 || a.heads % a.kv_heads || a.maps < 1 || a.maps > 2) return true;
+	if (a.dim < 16 || a.vdim < 16 || a.dim % 16 || a.vdim % 16 || a.dim_true < 1 || a.dim_true > a.dim || a.vdim_true < 1 || a.vdim_true > a.vdim) return true;
+	if (a.max_seq < 1 || a.splits < 1 || a.splits > 64 || !(a.cap >= 0.f) || !(a.eps >= 0.f) || (dtype != 0 && dtype != 1)) return true;
+	return !a.pos || !a.k_cache || !a.v_cache || !a.status || (dtype ? !a.q_f32 : !a.q_hi);
+}
+
+static bool ssm_bad(const SsmArgs &a) {
+	if (a.M < 1 || a.rows_per_seq < 1 || a.M % a.rows_per_seq || a.heads < 1 || a.vdim < 1 || a.state < 1 || a.state > SS_MAX_STATE) return true;
+	if (a.groups < 1 || a.heads % a.groups || a.taps < 1 || a.taps > SS_MAX_TAPS) return true;
+	const int inner = a.heads * a.vdim, channels = inner + 2 * a.groups * a.state;
+	if (a.z_at < 0 || a.conv_at < 0 || a.dt_at < 0 || a.conv_ld < channels || a.z_at + inner > a.raw_ld || a.conv_at + channels > a.raw_ld || a.dt_at + a.heads > a.raw_ld) return true;
+	return !a.raw || !a.pos || !a.conv_w || !a.conv_b || !a.dt_bias || !a.a || !a.d || !a.ring || !a.s || !a.status;
 }
 
 }   // namespace gptq
@@ -80,7 +100,11 @@ int dense_matmul(const void *x, int64_t ldx, const void *w, int64_t ldw, int M, 
 		case DENSE_EPI_LOGITS:
 			if (!epi->out || epi->ldo < n16 || epi->ldo % 8) return GPTQ_ERR_INVALID;
 			break;
-		case DENSE_EPI_SILU:
+		case DENSE_EPI_TABLE:
+			if (!epi->out || epi->ldo < n16 || epi->ldo % 8 || !epi->tab || !epi->tab_token || epi->tab_rows < 1) return GPTQ_ERR_INVALID;
+			if (epi->tab_col < 0 || epi->tab_col % 8 || epi->tab_ld % 8 || epi->tab_ld < epi->tab_col + n16 || !aligned16(epi->tab)) return GPTQ_ERR_ALIGN;
+			break;
+		case DENSE_EPI_GATED:
 			if (!epi->out || N % 16 || epi->ldo < N / 2 || epi->ldo % 8) return GPTQ_ERR_INVALID;
 			break;
 		case DENSE_EPI_QKV:
@@ -93,6 +117,7 @@ int dense_matmul(const void *x, int64_t ldx, const void *w, int64_t ldw, int M, 
 		default:
 			return GPTQ_ERR_INVALID;
 	}
+	if (epi->act != DENSE_ACT_SILU && epi->act != DENSE_ACT_GELU) return GPTQ_ERR_INVALID;
 	if (epi->mode == DENSE_EPI_LOGITS && epi->best && (!epi->ticket || !epi->tok || !epi->pos_inout)) return GPTQ_ERR_INVALID;
 	DenseArgs a = {};
 	a.x = x;
@@ -150,6 +175,41 @@ int dense_latent_prefill(const dense_latent_prefill_t *a, void *stream) {
 	if (a->ldv % 8 || a->ldv < a->S || a->out_ld % 8 || a->out_ld < (int64_t)a->heads * a->vdim) return GPTQ_ERR_ALIGN;
 	if (!latent_prefill_ok(a->dim, a->rot_dim, a->vdim)) return GPTQ_ERR_UNSUPPORTED;
 	return latent_prefill_launch(*a, reinterpret_cast<cudaStream_t>(stream));
+}
+
+
+int dense_gqa_splits(int M, int heads, int kv_heads, int maps, int max_seq, int dtype) {
+	return M < 1 || heads < 1 || kv_heads < 1 || maps < 1 || max_seq < 1 ? 1 : gqa_splits(M, heads, kv_heads, maps, max_seq, dtype);
+}
+
+int dense_gqa_append(const dense_gqa_t *a, int dtype, void *stream) {
+	if (!a || gqa_bad(*a, dtype) || !a->raw) return GPTQ_ERR_INVALID;
+	if (a->dim > 512 || a->vdim > 512) return GPTQ_ERR_UNSUPPORTED;
+	if (!aligned16(a->raw) || a->raw_ld % 4 || a->raw_ld < (int64_t)(a->heads + a->kv_heads) * a->maps * a->dim + (int64_t)a->kv_heads * a->vdim) return GPTQ_ERR_ALIGN;
+	return gqa_append_launch(*a, dtype, reinterpret_cast<cudaStream_t>(stream));
+}
+int dense_gqa_attend(const dense_gqa_t *a, int dtype, void *stream) {
+	if (!a || gqa_bad(*a, dtype) || !a->part_ml || !a->part_acc || (!dtype && !a->q_lo)) return GPTQ_ERR_INVALID;
+	if (!gqa_attend_ok(a->maps, a->dim, a->vdim) || a->M > 65535) return GPTQ_ERR_UNSUPPORTED;
+	return gqa_attend_launch(*a, dtype, reinterpret_cast<cudaStream_t>(stream));
+}
+int dense_gqa_merge(const dense_gqa_t *a, int dtype, void *stream) {
+	if (!a || gqa_bad(*a, dtype) || !a->part_ml || !a->part_acc || !a->out || a->out_ld % 8 || a->out_ld < (int64_t)a->heads * a->vdim) return GPTQ_ERR_INVALID;
+	if (a->vdim > 512 || a->M > 65535) return GPTQ_ERR_UNSUPPORTED;
+	return gqa_merge_launch(*a, dtype, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int dense_ssm_step(const dense_ssm_t *a, void *stream) {
+	if (!a || ssm_bad(*a) || a->rows_per_seq != 1 || !a->out || a->out_ld < (int64_t)a->heads * a->vdim || a->M > 65535) return GPTQ_ERR_INVALID;
+	return ssm_step_launch(*a, reinterpret_cast<cudaStream_t>(stream));
+}
+int dense_ssm_conv(const dense_ssm_t *a, void *stream) {
+	if (!a || ssm_bad(*a) || !a->u) return GPTQ_ERR_INVALID;
+	return ssm_conv_launch(*a, reinterpret_cast<cudaStream_t>(stream));
+}
+int dense_ssm_scan(const dense_ssm_t *a, void *stream) {
+	if (!a || ssm_bad(*a) || !a->u || !a->out || a->out_ld < (int64_t)a->heads * a->vdim) return GPTQ_ERR_INVALID;
+	return ssm_scan_launch(*a, reinterpret_cast<cudaStream_t>(stream));
 }
 
 }   // extern "C"

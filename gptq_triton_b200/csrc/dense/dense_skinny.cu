@@ -5,8 +5,8 @@
 // are the A operand of mma.m16n8k16 and the activations the B operand.  A dot product does not care about the order of k, so
 // lane (gid, tig) feeds the eight consecutive k that its 16-byte loads deliver for rows gid and gid + 8 and the same eight k
 // of activation row gid: two MMAs per pair of loads, no shuffle.  fp32: the same layout on the FMA units.
-// The prologue optionally prepares the rows itself (embedding lookup, post-norm residual, final norm), the epilogue applies
-// what follows the projection (rotary queries / raw latent / gates, SiLU(gate) * up, scaled logits with the greedy choice).
+// The prologue optionally prepares the rows itself (embedding lookup, residual, norm), the epilogue applies what
+// follows the projection (rotary queries / raw latent / gates, act(gate) * up, scaled logits with the greedy choice).
 #include <algorithm>
 
 #include "dense.cuh"
@@ -16,7 +16,7 @@ namespace gptq {
 namespace {
 
 constexpr int SK_M = 8, SK_U = 4, SK_REDLD = 17;
-constexpr size_t SK_STATIC = (2 * DN_WARPS * SK_M * SK_REDLD + 4 * DN_WARPS) * sizeof(float) + 64;
+constexpr size_t SK_STATIC = (2 * DN_WARPS * SK_M * SK_REDLD + RP_SMEM) * sizeof(float) + 64;
 constexpr size_t SK_SMEM_MAX = 227 * 1024 - SK_STATIC - 1024;
 
 template <typename T>
@@ -25,7 +25,7 @@ __global__ void __launch_bounds__(DN_THREADS, 2) dense_skinny_kernel(const Dense
 	constexpr int STEP = 4 * E;                  // k per step of a warp
 	extern __shared__ __align__(16) unsigned char sk_smem[];
 	__shared__ float s_red[2][DN_WARPS][SK_M][SK_REDLD];
-	__shared__ float s_norm[4 * DN_WARPS];
+	__shared__ float s_norm[RP_SMEM];
 	__shared__ int s_last;
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
 	const int xs = p.K * (int)sizeof(T) + 16;    // bytes per staged row
@@ -134,16 +134,16 @@ __global__ void __launch_bounds__(DN_THREADS, 2) dense_skinny_kernel(const Dense
 		__syncthreads();                         // the buffer is written again two tiles later, behind the next tile's barrier
 		if (tid < 8 * p.M) {
 			const int m = tid >> 3, j = tid & 7, tile = (int)blockIdx.x + ti * (int)gridDim.x;
-			const bool silu = p.e.mode == DENSE_EPI_SILU;
-			const int ra = silu ? j : 2 * j, rb = silu ? j + 8 : 2 * j + 1;
+			const bool gated = p.e.mode == DENSE_EPI_GATED;
+			const int ra = gated ? j : 2 * j, rb = gated ? j + 8 : 2 * j + 1;
 			float va = 0.f, vb = 0.f;
 #pragma unroll
 			for (int i = 0; i < DN_WARPS; ++i) {
 				va += red[i][m][ra];
 				vb += red[i][m][rb];
 			}
-			if (silu) {
-				Elem<T>::store(reinterpret_cast<T *>(p.e.out) + (size_t)m * p.e.ldo + tile * 8 + j, silu_exact(va) * vb);
+			if (gated) {
+				Elem<T>::store(reinterpret_cast<T *>(p.e.out) + (size_t)m * p.e.ldo + tile * 8 + j, activation(p.e.act, va) * vb);
 			} else {
 				const int n = tile * 16 + 2 * j;
 				epi_pair<T>(p.e, m, n, va, vb);
@@ -203,7 +203,7 @@ int dense_skinny_launch(const DenseArgs &a, int dtype, cudaStream_t stream) {
 // ---- the same row preparation as a kernel of its own (prompts, and many rows) -------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(DN_THREADS) dense_rows_kernel(const RowPrep p, T *h, long long ldh) {
-	__shared__ float s_norm[4 * DN_WARPS];
+	__shared__ float s_norm[RP_SMEM];
 	pdl_wait();
 	pdl_trigger();
 	prepare_row<T>(p, blockIdx.x, h + (size_t)blockIdx.x * ldh, p.x_out != nullptr, s_norm);

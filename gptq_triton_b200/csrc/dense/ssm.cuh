@@ -1,0 +1,16 @@
+// Launchers of the state-space recurrence kernels.
+#pragma once
+
+#include "dense.cuh"
+
+namespace gptq {
+
+using SsmArgs = dense_ssm_t;
+
+constexpr int SS_MAX_STATE = 256, SS_MAX_TAPS = 16;
+
+int ssm_step_launch(const SsmArgs &p, cudaStream_t stream);
+int ssm_conv_launch(const SsmArgs &p, cudaStream_t stream);
+int ssm_scan_launch(const SsmArgs &p, cudaStream_t stream);
+
+}   // namespace gptq

@@ -1,5 +1,5 @@
-"""Decoder building blocks with dense bf16 or fp32 weights: projections with fused input and output steps, a SiLU-gated MLP,
-post-norm residual sublayers with LayerNorm and layer scale.
+"""Decoder building blocks with dense bf16 or fp32 weights: projections with fused input and output steps, gated MLPs, norms
+ahead of a projection (LayerNorm, RMS norm, RMS norm of equal parts), post-norm residual sublayers, a per-token side input.
 
 The residual stream is fp32 throughout.  Feature sizes are padded with zeros to multiples of 16 when weights are loaded, so
 the kernels need no edge cases inside a row; sizes that enter a mean stay the true ones.
@@ -7,7 +7,7 @@ the kernels need no edge cases inside a row; sizes that enter a mean stay the tr
 from __future__ import annotations
 
 import ctypes
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Optional
 
 import torch
@@ -36,15 +36,18 @@ def pad_to(t: torch.Tensor, *shape: int) -> torch.Tensor:
 
 @dataclass
 class Stream:
-	"""The residual stream between two sublayers, not yet formed: rows of `table` by token, or
-	x (+ LayerNorm(y) * gain + shift).  The next projection (or the row kernel) forms it."""
+	"""The residual stream between two sublayers, not yet formed: rows of `table` by token (plus rows of `pos_table` by
+	position), or x (+ norm(y) * gain + shift).  The next projection (or the row kernel) forms it."""
 	width: int
 	ld: int
 	eps: float
 	table: Optional[torch.Tensor] = None
 	token: Optional[torch.Tensor] = None
+	pos_table: Optional[torch.Tensor] = None
+	pos: Optional[torch.Tensor] = None
 	x: Optional[torch.Tensor] = None
 	y: Optional[torch.Tensor] = None
+	y_norm: int = _dense.NORM_NONE
 	gain: Optional[torch.Tensor] = None
 	shift: Optional[torch.Tensor] = None
 
@@ -55,18 +58,25 @@ class Stream:
 	def take(self, index: torch.Tensor) -> 'Stream':
 		"""The stream of some rows only."""
 		pick = lambda t: None if t is None else t.index_select(0, index)
-		return Stream(self.width, self.ld, self.eps, self.table, None if self.token is None else self.token.reshape(-1).index_select(0, index), pick(self.x), pick(self.y),
-					  self.gain, self.shift)
+		flat = lambda t: None if t is None else t.reshape(-1).index_select(0, index)
+		return replace(self, token=flat(self.token), pos=flat(self.pos), x=pick(self.x), y=pick(self.y))
 
-	def spec(self, control: torch.Tensor, x_out: Optional[torch.Tensor], final) -> '_dense.Rows':
+	def then(self, x: torch.Tensor, y: torch.Tensor, y_norm: int = _dense.NORM_NONE, gain: Optional[torch.Tensor] = None, shift: Optional[torch.Tensor] = None) -> 'Stream':
+		"""The stream x + norm(y) * gain + shift."""
+		return Stream(self.width, self.ld, self.eps, x=x, y=y, y_norm=y_norm, gain=gain, shift=shift)
+
+	def spec(self, control: torch.Tensor, x_out: Optional[torch.Tensor], final: Optional['Norm']) -> '_dense.Rows':
 		r = _dense.Rows()
 		if self.x is None:
 			r.table, r.token, r.vocab = ptr(self.table), ptr(self.token), self.table.shape[0]
+			if self.pos_table is not None:
+				r.pos_table, r.pos, r.max_pos = ptr(self.pos_table), ptr(self.pos), self.pos_table.shape[0]
 		else:
 			r.x_in = ptr(self.x)
-		r.x_out, r.y, r.gain, r.shift = ptr(x_out), ptr(self.y), ptr(self.gain), ptr(self.shift)
+		r.x_out, r.y, r.y_norm, r.gain, r.shift = ptr(x_out), ptr(self.y), self.y_norm, ptr(self.gain), ptr(self.shift)
+		r.fin_groups = 1
 		if final is not None:
-			r.fin_w, r.fin_b = ptr(final.weight), ptr(final.bias)
+			r.fin_norm, r.fin_w, r.fin_b, r.fin_groups = final.kind, ptr(final.weight), ptr(final.bias), final.parts
 		r.width, r.ld, r.eps, r.status = self.width, self.ld, self.eps, _dense.status_ptr(control)
 		return r
 
@@ -118,14 +128,31 @@ def linear(x: torch.Tensor, w: torch.Tensor, control: torch.Tensor, out_dtype: O
 	return out
 
 
-class LayerNorm(nn.Module):
-	"""Weight and bias (fp32, padded) of a LayerNorm that a projection applies to the stream it reads."""
+class Norm(nn.Module):
+	"""A norm that a projection applies to the stream it reads; weight and bias fp32, padded."""
+	kind = _dense.NORM_NONE
+	parts = 1
 
-	def __init__(self, weight: torch.Tensor, bias: torch.Tensor):
+	def __init__(self, weight: torch.Tensor, bias: Optional[torch.Tensor] = None):
 		super().__init__()
 		n = padded(weight.numel())
 		self.register_buffer('weight', pad_to(weight.float(), n))
-		self.register_buffer('bias', pad_to(bias.float(), n))
+		self.register_buffer('bias', None if bias is None else pad_to(bias.float(), n))
+
+
+class LayerNorm(Norm):
+	kind = _dense.NORM_LAYER
+
+
+class RMSNorm(Norm):
+	"""x / rms(x) * (offset + weight), by the mean square of the row or of each of `parts` equal parts."""
+	kind = _dense.NORM_RMS
+
+	def __init__(self, weight: torch.Tensor, offset: float = 0.0, parts: int = 1):
+		if not 1 <= parts <= _dense.MAX_NORM_GROUPS or weight.numel() % parts:
+			raise ValueError(f'an RMS norm of {weight.numel()} entries in {parts} parts')
+		super().__init__(weight.float() + offset)
+		self.parts = parts
 
 
 class PostNorm(nn.Module):
@@ -140,23 +167,53 @@ class PostNorm(nn.Module):
 		self.register_buffer('shift', pad_to((bias.double() * f).float(), n))
 
 	def join(self, stream: Stream, x: torch.Tensor, y: torch.Tensor) -> Stream:
-		return Stream(stream.width, stream.ld, stream.eps, x=x, y=y, gain=self.gain, shift=self.shift)
+		return stream.then(x, y, _dense.NORM_LAYER, self.gain, self.shift)
 
 
 class DenseMLP(nn.Module):
-	"""down(silu(gate h) * (up h)).  Gate and up rows alternate in groups of eight in one matrix, so that one pass over it
+	"""down(act(gate h) * (up h)).  Gate and up rows alternate in groups of eight in one matrix, so that one pass over it
 	leaves both factors of an output in the same thread."""
 
-	def __init__(self, gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor):
+	def __init__(self, gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor, act: str = 'silu'):
 		super().__init__()
 		ff, width = gate.shape
 		f, w = padded(ff), padded(width)
 		g, u = pad_to(gate, f, w), pad_to(up, f, w)
+		self.act = _dense.ACT_CODE[act]
 		self.register_buffer('gate_up', torch.stack([g.view(f // 8, 8, w), u.view(f // 8, 8, w)], dim=1).reshape(2 * f, w).contiguous())
 		self.register_buffer('down', pad_to(down, w, f).contiguous())
 
-	def forward(self, stream: Stream, control: torch.Tensor):
+	def gated(self, out: torch.Tensor) -> '_dense.Epilogue':
+		e = epilogue(_dense.EPI_GATED, out)
+		e.act = self.act
+		return e
+
+	def forward(self, stream: Stream, control: torch.Tensor, norm: Optional[Norm] = None):
 		"""Returns (residual stream x, sublayer output y), both fp32."""
 		a = torch.empty((stream.rows, self.down.shape[1]), dtype=self.down.dtype, device=self.down.device)
-		x = project_stream(stream, self.gate_up, epilogue(_dense.EPI_SILU, a), control)
+		x = project_stream(stream, self.gate_up, self.gated(a), control, final=norm)
 		return x, linear(a, self.down, control)
+
+
+class TokenSide(nn.Module):
+	"""A layer's per-token input: x + RMSNorm(proj(act(gate x) * e)) with e the columns [column, column + dim) of the token's row
+	of `table` (all sizes padded)."""
+
+	def __init__(self, gate: torch.Tensor, proj: torch.Tensor, norm_weight: torch.Tensor, column: int, act: str = 'gelu_tanh'):
+		super().__init__()
+		dim, width = gate.shape
+		d, w = padded(dim), padded(width)
+		self.column, self.act = column, _dense.ACT_CODE[act]
+		self.register_buffer('gate', pad_to(gate, d, w).contiguous())
+		self.register_buffer('proj', pad_to(proj, w, d).contiguous())
+		self.register_buffer('gain', pad_to(norm_weight.float(), w))
+
+	def gated(self, out: torch.Tensor, table: torch.Tensor, token: torch.Tensor) -> '_dense.Epilogue':
+		e = epilogue(_dense.EPI_TABLE, out)
+		e.act, e.tab, e.tab_ld, e.tab_rows, e.tab_col, e.tab_token = self.act, ptr(table), table.stride(0), table.shape[0], self.column, ptr(token)
+		return e
+
+	def forward(self, stream: Stream, table: torch.Tensor, token: torch.Tensor, control: torch.Tensor) -> Stream:
+		a = torch.empty((stream.rows, self.gate.shape[0]), dtype=self.gate.dtype, device=self.gate.device)
+		x = project_stream(stream, self.gate, self.gated(a, table, token), control)
+		return stream.then(x, linear(a, self.proj, control), _dense.NORM_RMS, self.gain)

@@ -7,7 +7,7 @@ A model's engine subclasses StaticEngine and supplies the cache layout, `_portio
 from __future__ import annotations
 
 import os
-from typing import Optional, Sequence
+from typing import List, Optional, Sequence
 
 import torch
 
@@ -44,6 +44,10 @@ class StaticEngine:
 	def _before_capture(self):
 		pass
 
+	def _carried(self) -> List[torch.Tensor]:
+		"""Recurrent state that a step overwrites: put back after the trial runs of a capture."""
+		return []
+
 	def _restore(self, tok: torch.Tensor, pos: torch.Tensor):
 		self.tok.copy_(tok)
 		self.pos.copy_(pos)
@@ -51,7 +55,7 @@ class StaticEngine:
 	# -- the loop ----------------------------------------------------------------------------------
 	def reset(self):
 		"""Gives the cache rows back: the next tokens start new sequences at position 0.  Rows of earlier sequences are never
-		read again, because a query sees positions up to its own only."""
+		read again, because a query sees positions up to its own only, and recurrent state counts as zero at position 0."""
 		self.next_pos = 0
 		self.pos.zero_()
 
@@ -109,6 +113,7 @@ class StaticEngine:
 			self._before_capture()
 			# warm up on a side stream (allocations, workspaces), then capture
 			saved = (self.tok.clone(), self.pos.clone())
+			carried = [t.clone() for t in self._carried()]
 			s = torch.cuda.Stream()
 			s.wait_stream(torch.cuda.current_stream())
 			best, best_ms, best_logits = None, None, None
@@ -149,6 +154,8 @@ class StaticEngine:
 			torch.cuda.current_stream().wait_stream(s)
 			# capture does not execute (and the timed replays started from the saved state): restore it
 			self._restore(*saved)
+			for t, old in zip(self._carried(), carried):
+				t.copy_(old)
 			self.graph = best
 			self.graph_logits = best_logits
 		self.graph.replay()

@@ -8,7 +8,7 @@ from typing import Callable, Dict, Optional, Tuple
 
 import torch
 
-from . import befalix, llama, loader
+from . import befalix, lifinex, llama, loader
 
 
 @dataclass(frozen=True)
@@ -29,6 +29,7 @@ def register(arch: Architecture):
 
 register(Architecture('LlamaForCausalLM', lambda ck, device, dtype: loader.load_quant(str(ck), device=device), llama.DecodeEngine, (torch.float16,), ('gptq',)))
 register(Architecture(befalix.ARCHITECTURE, befalix.load_befalix, befalix.BefalixEngine, (torch.bfloat16, torch.float32), ('dense',)))
+register(Architecture(lifinex.ARCHITECTURE, lifinex.load_lifinex, lifinex.LifinexEngine, (torch.bfloat16, torch.float32), ('dense',)))
 
 
 def architecture_of(checkpoint) -> Architecture:

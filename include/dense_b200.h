@@ -1,6 +1,7 @@
 /*
  * dense_b200.h — C ABI of libdense_b200.so: decoder layers with dense bf16 (or fp32) weights on NVIDIA B200 (sm_100a).
- * Projections with fused row preparation and epilogues, and latent attention (keys and values in one low-rank row per token).
+ * Projections with fused row preparation and epilogues, latent attention (keys and values in one low-rank row per token),
+ * grouped-query attention with one or two softmax maps per head, and a selective state-space recurrence.
  *
  * Every pointer inside the argument blocks is a DEVICE pointer.  Entry points are asynchronous on `stream`, never
  * synchronise, allocate or free, and return 0 or a negative GPTQ_ERR_* code (gptq_b200.h).
@@ -24,13 +25,24 @@ extern "C" {
 /* epilogues of dense_matmul */
 #define DENSE_EPI_F32     0            /* out fp32 [M, ldo] = scale * result */
 #define DENSE_EPI_T       1            /* out in the activation dtype */
-#define DENSE_EPI_SILU    2            /* weight rows in groups of 16: 8 gate rows, 8 up rows; out[8 g + j] = silu(gate_j) * up_j */
+#define DENSE_EPI_GATED   2            /* weight rows in groups of 16: 8 gate rows, 8 up rows; out[8 g + j] = act(gate_j) * up_j */
 #define DENSE_EPI_QKV     3            /* rotary queries | raw fp32 latent rows | sigmoid gates */
 #define DENSE_EPI_LOGITS  4            /* F32, and with `best` set the greedy choice per row (decode rows only) */
+#define DENSE_EPI_TABLE   5            /* out in the activation dtype = act(result) * tab[token, tab_col + n] */
 
-/* Row preparation: x = table[token], or x_in (+ LayerNorm(y) * gain + shift when y is set, mean and variance over `width`
- * of the `ld` columns); x_out (optional, never the same as x_in) receives it; the prepared row is x, or LayerNorm(x) * fin_w
- * + fin_b when fin_w is set. */
+/* activations of GATED and TABLE */
+#define DENSE_ACT_SILU 0
+#define DENSE_ACT_GELU 1               /* the tanh form */
+
+/* norms of a row (mean, variance and mean square over `width` of the `ld` columns) */
+#define DENSE_NORM_NONE  0
+#define DENSE_NORM_LAYER 1             /* (v - mean) / sqrt(var + eps) */
+#define DENSE_NORM_RMS   2             /* v / sqrt(mean(v^2) + eps) */
+#define DENSE_MAX_NORM_GROUPS 256
+
+/* Row preparation.  x = table[token] (+ pos_table[pos]), or x_in; with y set, x += y_norm(y) * gain + shift (gain absent: 1,
+ * shift absent: 0).  x_out (optional, never the same as x_in) receives x.  The prepared row is fin_norm(x) * fin_w + fin_b (each
+ * optional); an RMS norm may work on fin_groups equal parts of the row, each by its own mean square (then y must be absent). */
 typedef struct {
 	const float *x_in;
 	float *x_out;
@@ -40,6 +52,10 @@ typedef struct {
 	const void *table;
 	const int64_t *token;
 	int64_t vocab;
+	const void *pos_table;             /* [max_pos, ld] */
+	const int32_t *pos;                /* [M] */
+	int max_pos;
+	int y_norm, fin_norm, fin_groups;
 	int width, ld;
 	float eps;
 	int *status;
@@ -66,6 +82,12 @@ typedef struct {
 	unsigned *ticket;
 	int64_t *tok;                      /* receives the arg-max (lowest index on ties) */
 	int32_t *pos_inout;                /* incremented */
+	/* GATED, TABLE */
+	int act;
+	const void *tab;                   /* [tab_rows, tab_ld] in the activation dtype */
+	int64_t tab_ld, tab_rows;
+	int tab_col;
+	const int64_t *tab_token;          /* [M] */
 } dense_epilogue_t;
 
 /* Latent attention, absorbed form.  A cache row is [latent (kv_rank) | rotated key part (rot_dim)]. */
@@ -108,6 +130,55 @@ typedef struct {
 	int *status;
 } dense_latent_prefill_t;
 
+/* Grouped-query attention with `maps` (1 or 2) softmax maps per head over shared values.  Query head h reads key / value head
+ * h / (heads / kv_heads).  Per map: score = cap * tanh(q . k * scale / cap) (cap 0: q . k * scale), causal softmax, a_map = sum p v.
+ * Result per head: o = a_1, or a_1 - lambda * a_2; with out_norm o / sqrt(mean(o^2) + eps); times out_mul.
+ * A raw row is [queries: heads * maps * dim | keys: kv_heads * maps * dim | values: kv_heads * vdim]; queries and keys are
+ * RMS-normed per head and map when q_norm / k_norm are given. */
+typedef struct {
+	int M, rows_per_seq;               /* query rows, rows_per_seq consecutive rows per sequence */
+	int heads, kv_heads, maps, dim, vdim;      /* dim and vdim padded to multiples of 16 */
+	int dim_true, vdim_true;           /* what the norms average over */
+	int max_seq, splits;
+	float scale, cap, eps, lambda, out_mul;
+	int out_norm;
+	const int32_t *pos;                /* [M] */
+	const void *raw;                   /* [M, raw_ld] fp32 */
+	int64_t raw_ld;
+	const float *q_norm, *k_norm;      /* [dim] or NULL */
+	void *k_cache;                     /* [sequences, max_seq, kv_heads * maps * dim] */
+	void *v_cache;                     /* [sequences, max_seq, kv_heads * vdim] */
+	void *q_hi, *q_lo;                 /* bf16 [M, heads * maps * dim]: normed queries times scale (/ cap), high part and remainder */
+	float *q_f32;                      /* dtype 1 */
+	float *part_ml;                    /* [M, heads * maps, splits, 2] */
+	float *part_acc;                   /* [M, heads * maps, splits, vdim] */
+	void *out;                         /* [M, out_ld] */
+	int64_t out_ld;
+	int *status;
+} dense_gqa_t;
+
+/* Selective state-space recurrence with a short causal convolution in front (Mamba-2).  A raw row is fp32
+ * [z: inner | x: inner, B: groups * state, C: groups * state | dt: heads], inner = heads * vdim, sections at z_at, conv_at, dt_at.
+ *   u = silu(conv(x, B, C) + conv_b);  dt = softplus(dt + dt_bias);  S = exp(a * dt) S + dt x B^T;  y = S C + d * x;  out = y * silu(z)
+ * The last `taps` convolution inputs of a sequence are kept in a ring (slot = position mod taps).  At position 0 the state and
+ * the inputs before it are taken as zero, whatever the buffers hold. */
+typedef struct {
+	int M, rows_per_seq;
+	int heads, vdim, state, groups, taps;
+	int z_at, conv_at, dt_at, conv_ld; /* conv_ld: padded number of convolution channels */
+	int64_t raw_ld;
+	const float *raw;                  /* [M, raw_ld] */
+	const int32_t *pos;                /* [M] */
+	const float *conv_w, *conv_b;      /* [taps, conv_ld] (last tap: the current token), [conv_ld] */
+	const float *dt_bias, *a, *d;      /* [heads] */
+	float *ring;                       /* [sequences, taps, conv_ld] */
+	float *s;                          /* [sequences, heads, vdim, state] */
+	float *u;                          /* scratch of portions: [M, conv_ld] */
+	float *out;                        /* [M, out_ld] fp32 */
+	int64_t out_ld;
+	int *status;
+} dense_ssm_t;
+
 int dense_version(void);
 int dense_last_cuda_error(void);
 
@@ -125,6 +196,15 @@ int dense_latent_attend(const dense_latent_t *args, int dtype, void *stream);
 int dense_latent_value(const dense_latent_t *args, int dtype, void *stream);
 int dense_latent_prefill_ok(int dim, int rot_dim, int vdim);
 int dense_latent_prefill(const dense_latent_prefill_t *args, void *stream);
+
+int dense_gqa_splits(int M, int heads, int kv_heads, int maps, int max_seq, int dtype);
+int dense_gqa_append(const dense_gqa_t *args, int dtype, void *stream);      /* normed queries, cache rows */
+int dense_gqa_attend(const dense_gqa_t *args, int dtype, void *stream);      /* partial results per key range */
+int dense_gqa_merge(const dense_gqa_t *args, int dtype, void *stream);       /* key ranges and maps into the output */
+
+int dense_ssm_step(const dense_ssm_t *args, void *stream);                   /* rows_per_seq = 1 */
+int dense_ssm_conv(const dense_ssm_t *args, void *stream);                   /* portions: u */
+int dense_ssm_scan(const dense_ssm_t *args, void *stream);                   /* portions: out, state, ring */
 
 #ifdef __cplusplus
 }
