@@ -44,7 +44,7 @@ def softplus(z):
 
 
 def soft_cap(s, cap):
-	return cap * torch.tanh(s / cap)
+	return s if cap is None else cap * torch.tanh(s / cap)
 
 
 def causal_softmax(s):
@@ -58,25 +58,38 @@ def diff_lambda(w, mixer):
 	return torch.exp((w['lq1'] * w['lk1']).sum()) - torch.exp((w['lq2'] * w['lk2']).sum()) + mixer['diff']
 
 
-def attention_maps(h, w, mixer, eps):
-	"""Outputs of both maps [t, heads, 2, vdim]."""
-	t, H, G, D, V = h.shape[0], mixer['heads'], mixer['kv_heads'], mixer['dim'], mixer['vdim']
-	q = rms_norm((h @ w['q'].T).reshape(t, H, 2, D), w['q.norm'], eps)
-	k = rms_norm((h @ w['k'].T).reshape(t, G, 2, D), w['k.norm'], eps)
-	v = (h @ w['v'].T).reshape(t, G, V)
-	out = torch.empty((t, H, 2, V), dtype=h.dtype)
-	for n in range(H):
-		g = n // (H // G)
-		for m in range(2):
-			s = soft_cap(q[:, n, m] @ k[:, g, m].T * mixer['scale'], mixer['softcap'])
-			out[:, n, m] = causal_softmax(s) @ v[:, g]
+def attention_maps(q, k, v, scale, cap):
+	"""q [t, heads, maps, dim], k [t, kv_heads, maps, dim], v [t, kv_heads, vdim] -> every map's output [t, heads, maps, vdim]."""
+	t, H, n, _ = q.shape
+	G = k.shape[1]
+	out = torch.empty((t, H, n, v.shape[2]), dtype=q.dtype)
+	for h in range(H):
+		g = h // (H // G)
+		for m in range(n):
+			out[:, h, m] = causal_softmax(soft_cap(q[:, h, m] @ k[:, g, m].T * scale, cap)) @ v[:, g]
 	return out
 
 
+def normed_qkv(h, w, mixer, eps, maps=2):
+	t, H, G, D, V = h.shape[0], mixer['heads'], mixer['kv_heads'], mixer['dim'], mixer['vdim']
+	q = rms_norm((h @ w['q'].T).reshape(t, H, maps, D), w['q.norm'], eps)
+	k = rms_norm((h @ w['k'].T).reshape(t, G, maps, D), w['k.norm'], eps)
+	return q, k, (h @ w['v'].T).reshape(t, G, V)
+
+
+def combine_maps(a, lam, diff, eps):
+	"""a [t, heads, 2, vdim] -> [t, heads * vdim]."""
+	return (unit_rms(a[:, :, 0] - lam * a[:, :, 1], eps) * (1 - diff)).flatten(1)
+
+
 def differential_attention(h, w, mixer, eps):
-	a = attention_maps(h, w, mixer, eps)
-	o = unit_rms(a[:, :, 0] - diff_lambda(w, mixer) * a[:, :, 1], eps) * (1 - mixer['diff'])
-	return o.reshape(h.shape[0], -1) @ w['o'].T
+	a = attention_maps(*normed_qkv(h, w, mixer, eps), mixer['scale'], mixer['softcap'])
+	return combine_maps(a, diff_lambda(w, mixer), mixer['diff'], eps) @ w['o'].T
+
+
+def plain_attention(h, w, mixer, eps):
+	"""The same with a single map per head."""
+	return attention_maps(*normed_qkv(h, w, mixer, eps, 1), mixer['scale'], mixer['softcap']).flatten(1) @ w['o'].T
 
 
 def causal_conv(u, w, b):

@@ -36,8 +36,8 @@ def test_header_binding_and_library_agree(lib):
 def test_struct_layouts_match_the_header(tmp_path):
 	"""sizeof and the last member's offset of every argument block, as the C compiler lays them out."""
 	import subprocess
-	structs = {'dense_rows_t': (_dense.Rows, 'status'), 'dense_epilogue_t': (_dense.Epilogue, 'pos_inout'), 'dense_latent_t': (_dense.Latent, 'status'),
-			   'dense_latent_prefill_t': (_dense.LatentPrefill, 'status')}
+	structs = {'dense_rows_t': (_dense.Rows, 'status'), 'dense_epilogue_t': (_dense.Epilogue, 'tab_token'), 'dense_latent_t': (_dense.Latent, 'status'),
+			   'dense_latent_prefill_t': (_dense.LatentPrefill, 'status'), 'dense_gqa_t': (_dense.Gqa, 'status'), 'dense_ssm_t': (_dense.Ssm, 'status')}
 	src = '#include <stdio.h>\n#include "dense_b200.h"\nint main(void) {' + ''.join(
 		f'printf("%zu %zu\\n", sizeof({n}), offsetof({n}, {last}));' for n, (_, last) in structs.items()) + 'return 0; }'
 	(tmp_path / 's.c').write_text(src)
