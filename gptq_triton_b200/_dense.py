@@ -77,6 +77,8 @@ _SIGNATURES = {
 	'dense_gqa_append': (c_int, [_P, _I, _P]),
 	'dense_gqa_attend': (c_int, [_P, _I, _P]),
 	'dense_gqa_merge': (c_int, [_P, _I, _P]),
+	'dense_gqa_prefill_maps': (c_int, [_I, _I, _I]),
+	'dense_gqa_prefill': (c_int, [_P, _I, _P]),
 	'dense_ssm_step': (c_int, [_P, _P]),
 	'dense_ssm_conv': (c_int, [_P, _P]),
 	'dense_ssm_scan': (c_int, [_P, _P]),

@@ -199,6 +199,16 @@ int dense_gqa_merge(const dense_gqa_t *a, int dtype, void *stream) {
 	return gqa_merge_launch(*a, dtype, reinterpret_cast<cudaStream_t>(stream));
 }
 
+int dense_gqa_prefill_maps(int maps, int dim, int vdim) { return gqa_prefill_maps(maps, dim, vdim); }
+int dense_gqa_prefill(const dense_gqa_t *a, int start, void *stream) {
+	if (!a || gqa_bad(*a, 0) || start < 0 || start + a->M > a->max_seq || a->rows_per_seq != a->M) return GPTQ_ERR_INVALID;
+	const int maps = gqa_prefill_maps(a->maps, a->dim, a->vdim);
+	if (!maps) return GPTQ_ERR_UNSUPPORTED;
+	if (maps == 2 ? !a->out || a->out_ld % 8 || a->out_ld < (int64_t)a->heads * a->vdim || !aligned16(a->out) : !a->part_ml || !a->part_acc || a->splits != 1) return GPTQ_ERR_INVALID;
+	if (!aligned16(a->q_hi) || !aligned16(a->k_cache) || !aligned16(a->v_cache)) return GPTQ_ERR_ALIGN;
+	return gqa_prefill_launch(*a, start, reinterpret_cast<cudaStream_t>(stream));
+}
+
 int dense_ssm_step(const dense_ssm_t *a, void *stream) {
 	if (!a || ssm_bad(*a) || a->rows_per_seq != 1 || !a->out || a->out_ld < (int64_t)a->heads * a->vdim || a->M > 65535) return GPTQ_ERR_INVALID;
 	return ssm_step_launch(*a, reinterpret_cast<cudaStream_t>(stream));

@@ -19,6 +19,8 @@ int gqa_append_launch(const GqaArgs &p, int dtype, cudaStream_t stream);
 bool gqa_attend_ok(int maps, int dim, int vdim);
 int gqa_splits(int M, int heads, int kv_heads, int maps, int max_seq, int dtype);
 int gqa_attend_launch(const GqaArgs &p, int dtype, cudaStream_t stream);
+int gqa_prefill_maps(int maps, int dim, int vdim);      // maps per CTA of the prompt kernel: 2 (writes out), 1 (writes partials), 0: does not fit
+int gqa_prefill_launch(const GqaArgs &p, int start, cudaStream_t stream);
 int gqa_merge_launch(const GqaArgs &p, int dtype, cudaStream_t stream);
 
 }   // namespace gptq

@@ -18,45 +18,22 @@
 // With NQ = 2 the MMAs of one query tile run under the softmax of the other.  Every wait is bounded.
 #include <algorithm>
 
-#include "../tcgen05.cuh"
 #include "latent.cuh"
+#include "prefill_common.cuh"
 
 namespace gptq {
-
-int dense_tensor_map(const void *base, long long rows, long long cols, long long ld, int box_rows, int box_cols, CUtensorMap *out);
 
 namespace {
 
 constexpr int LP_T = 128;                               // query rows and keys per tile
 constexpr int LP_CHUNK = LP_T * 128;                    // bytes of a 128 x 64 bf16 operand chunk
 constexpr int LP_TILE_THREADS = 2 * LP_T;               // softmax threads per query tile
-constexpr uint32_t LP_SPIN = 1u << 24;
 constexpr size_t LP_SMEM = 227 * 1024 - 4 * 2 * LP_T * sizeof(float);      // what a CTA may have, less the exchanged maxima
 
 struct LpPlan {
 	int nd, nr, sk, sv;                                   // chunks of the unrotated / rotated part, stages of K and V
 	size_t smem;
 };
-
-__device__ __forceinline__ float ex2(float x) {
-	float r;
-	asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-	return r;
-}
-// One poll inline; the bounded loop (and the look at the abort flag) out of line, so that the code of a wait that is already
-// over stays short.
-__device__ __noinline__ bool wait_slow(uint32_t bar, uint32_t parity, volatile int *abort_flag) {
-	return !*abort_flag && mbar_wait_bounded(bar, parity, LP_SPIN);
-}
-__device__ __forceinline__ bool wait_fast(uint32_t bar, uint32_t parity, volatile int *abort_flag) {
-	return mbar_try_wait(bar, parity) || wait_slow(bar, parity, abort_flag);
-}
-// registers loaded by tcgen05.ld may be used only behind the wait: tie them to it
-template <int N>
-__device__ __forceinline__ void tmem_settle(float (&v)[N]) {
-#pragma unroll
-	for (int i = 0; i < N; ++i) asm volatile("" : "+f"(v[i]));
-}
 
 template <int NQ>
 __global__ void __launch_bounds__(NQ * (LP_TILE_THREADS + 32) + 32, 1) latent_prefill_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_constant__ CUtensorMap tmk,
@@ -125,7 +102,7 @@ __global__ void __launch_bounds__(NQ * (LP_TILE_THREADS + 32) + 32, 1) latent_pr
 			int jk = 0, jv = 0;
 			for (int j = 0; j < nmax; ++j) {
 				const int a = j % pl.sk, b = j % pl.sv;
-				if (*s_abort || !mbar_wait_bounded(bar_ek + 8 * a, ((j / pl.sk) & 1) ^ 1, LP_SPIN)) { fail(); break; }
+				if (*s_abort || !mbar_wait_bounded(bar_ek + 8 * a, ((j / pl.sk) & 1) ^ 1, ATTN_SPIN)) { fail(); break; }
 				mbar_arrive_expect_tx(bar_fk + 8 * a, k_bytes);
 				for (int c = 0; c < nch; ++c) {
 					const uint32_t dst = sk + a * k_bytes + c * LP_CHUNK;
@@ -133,15 +110,15 @@ __global__ void __launch_bounds__(NQ * (LP_TILE_THREADS + 32) + 32, 1) latent_pr
 					else tma_load_2d(dst, &tmr, p.kv_rank + 64 * (c - pl.nd), j * LP_T, bar_fk + 8 * a);
 				}
 				jk = j + 1;
-				if (*s_abort || !mbar_wait_bounded(bar_ev + 8 * b, ((j / pl.sv) & 1) ^ 1, LP_SPIN)) { fail(); break; }
+				if (*s_abort || !mbar_wait_bounded(bar_ev + 8 * b, ((j / pl.sv) & 1) ^ 1, ATTN_SPIN)) { fail(); break; }
 				mbar_arrive_expect_tx(bar_fv + 8 * b, v_bytes);
 				for (int c = 0; c < 2; ++c) tma_load_2d(sv + b * v_bytes + c * (v_bytes / 2), &tmv, j * LP_T + 64 * c, head * p.vdim, bar_fv + 8 * b);
 				jv = j + 1;
 			}
 			// no copy may be in flight when the CTA ends
-			mbar_wait_bounded(bar_q, 0, LP_SPIN);
-			for (int j = max(0, jk - pl.sk); j < jk; ++j) mbar_wait_bounded(bar_fk + 8 * (j % pl.sk), (j / pl.sk) & 1, LP_SPIN);
-			for (int j = max(0, jv - pl.sv); j < jv; ++j) mbar_wait_bounded(bar_fv + 8 * (j % pl.sv), (j / pl.sv) & 1, LP_SPIN);
+			mbar_wait_bounded(bar_q, 0, ATTN_SPIN);
+			for (int j = max(0, jk - pl.sk); j < jk; ++j) mbar_wait_bounded(bar_fk + 8 * (j % pl.sk), (j / pl.sk) & 1, ATTN_SPIN);
+			for (int j = max(0, jv - pl.sv); j < jv; ++j) mbar_wait_bounded(bar_fv + 8 * (j % pl.sv), (j / pl.sv) & 1, ATTN_SPIN);
 		}
 		__syncwarp();
 	} else if (warp >= W_MMA) {
@@ -201,7 +178,7 @@ __global__ void __launch_bounds__(NQ * (LP_TILE_THREADS + 32) + 32, 1) latent_pr
 				}
 			}
 			umma_commit(bar_drain + 8 * i);          // every MMA has completed before tensor memory goes back
-			mbar_wait_bounded(bar_drain + 8 * i, 0, LP_SPIN);
+			mbar_wait_bounded(bar_drain + 8 * i, 0, ATTN_SPIN);
 		}
 		__syncwarp();
 	} else {

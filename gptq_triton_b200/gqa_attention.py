@@ -17,6 +17,10 @@ from ._lib import ptr, stream_ptr
 from .dense import Norm, Stream, epilogue, linear, pad_to, padded, project_stream
 
 
+# portions of more rows than this per sequence run on the tensor-core prompt kernel (bf16)
+DECODE_MAX_ROWS = 8
+
+
 @dataclass(frozen=True)
 class GroupedAttentionSpec:
 	heads: int
@@ -65,10 +69,14 @@ class GroupedAttention(nn.Module):
 		a = self.arguments(raw, cache, pos, rows_per_seq, stream.eps, control)
 		lib, code, st = _dense.lib(), _dense.DTYPE_CODE[dt], stream_ptr(dev)
 		out = torch.empty((M, s.heads * self.V), dtype=dt, device=dev)
-		scratch = self.buffers(a, out, max_seq if start is None else start + rows_per_seq)      # noqa: F841 (alive until the launches)
-		_dense.check(lib.dense_gqa_append(ctypes.byref(a), code, st), 'dense_gqa_append')
-		_dense.check(lib.dense_gqa_attend(ctypes.byref(a), code, st), 'dense_gqa_attend')
-		_dense.check(lib.dense_gqa_merge(ctypes.byref(a), code, st), 'dense_gqa_merge')
+		maps = 0 if start is None or dt == torch.float32 or rows_per_seq <= DECODE_MAX_ROWS else lib.dense_gqa_prefill_maps(s.maps, self.D, self.V)
+		if maps:
+			self._prompt(a, out, rows_per_seq, start, maps, cache)
+		else:
+			scratch = self.buffers(a, out, max_seq if start is None else start + rows_per_seq)      # noqa: F841 (alive until the launches)
+			_dense.check(lib.dense_gqa_append(ctypes.byref(a), code, st), 'dense_gqa_append')
+			_dense.check(lib.dense_gqa_attend(ctypes.byref(a), code, st), 'dense_gqa_attend')
+			_dense.check(lib.dense_gqa_merge(ctypes.byref(a), code, st), 'dense_gqa_merge')
 		return x, linear(out, self.w_o, control)
 
 	def arguments(self, raw, cache, pos, rows_per_seq: int, eps: float, control) -> '_dense.Gqa':
@@ -94,6 +102,27 @@ class GroupedAttention(nn.Module):
 		else:
 			a.q_hi, a.q_lo = ptr(q[0]), ptr(q[1])
 		return q, ml, acc
+
+	def _prompt(self, a: '_dense.Gqa', out, t: int, start: int, maps: int, cache):
+		"""Normed queries and cache rows of all sequences, then the tensor-core attention kernel per sequence."""
+		s, dev, lib = self.spec, out.device, _dense.lib()
+		st = stream_ptr(dev)
+		q = torch.empty((a.M, s.heads * s.maps * self.D), dtype=out.dtype, device=dev)
+		a.q_hi, a.out, a.out_ld, a.splits = ptr(q), ptr(out), out.stride(0), 1
+		if maps < s.maps or s.maps == 1:
+			ml = torch.empty((a.M, s.heads * s.maps, 2), dtype=torch.float32, device=dev)
+			acc = torch.empty((a.M, s.heads * s.maps, self.V), dtype=torch.float32, device=dev)
+			a.part_ml, a.part_acc = ptr(ml), ptr(acc)
+		_dense.check(lib.dense_gqa_append(ctypes.byref(a), 0, st), 'dense_gqa_append')
+		for b in range(a.M // t):
+			one = _dense.Gqa.from_buffer_copy(a)
+			rows = slice(b * t, (b + 1) * t)
+			one.M, one.q_hi, one.out, one.k_cache, one.v_cache = t, ptr(q[rows]), ptr(out[rows]), ptr(cache['k'][b]), ptr(cache['v'][b])
+			if a.part_ml:
+				one.part_ml, one.part_acc = ptr(ml[rows]), ptr(acc[rows])
+			_dense.check(lib.dense_gqa_prefill(ctypes.byref(one), start, st), 'dense_gqa_prefill')
+		if a.part_ml:
+			_dense.check(lib.dense_gqa_merge(ctypes.byref(a), 0, st), 'dense_gqa_merge')
 
 
 def diff_lambda(lq1: torch.Tensor, lk1: torch.Tensor, lq2: torch.Tensor, lk2: torch.Tensor, diff: float) -> float:

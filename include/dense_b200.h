@@ -201,6 +201,11 @@ int dense_gqa_splits(int M, int heads, int kv_heads, int maps, int max_seq, int 
 int dense_gqa_append(const dense_gqa_t *args, int dtype, void *stream);      /* normed queries, cache rows */
 int dense_gqa_attend(const dense_gqa_t *args, int dtype, void *stream);      /* partial results per key range */
 int dense_gqa_merge(const dense_gqa_t *args, int dtype, void *stream);       /* key ranges and maps into the output */
+/* A prompt portion of one sequence at positions start .. start + M - 1 on the tensor cores, bf16: keys and values from the
+ * cache, queries from q_hi.  dense_gqa_prefill_maps: 2: both maps at once, writes out; 1: writes partials (splits = 1) for
+ * dense_gqa_merge; 0: sizes that do not fit. */
+int dense_gqa_prefill_maps(int maps, int dim, int vdim);
+int dense_gqa_prefill(const dense_gqa_t *args, int start, void *stream);
 
 int dense_ssm_step(const dense_ssm_t *args, void *stream);                   /* rows_per_seq = 1 */
 int dense_ssm_conv(const dense_ssm_t *args, void *stream);                   /* portions: u */
