@@ -14,10 +14,11 @@ from ._lib import GptqB200Error, ptr, register_status_buffer, require_cuda, stre
 LIB_PATH = Path(__file__).resolve().parent / 'libdense_b200.so'
 CONTROL_BYTES = 16384
 
-EPI_F32, EPI_T, EPI_GATED, EPI_QKV, EPI_LOGITS, EPI_TABLE = range(6)
+EPI_F32, EPI_T, EPI_GATED, EPI_QKV, EPI_LOGITS, EPI_TABLE, EPI_MIXED = range(7)
 ACT_CODE = {'silu': 0, 'gelu_tanh': 1}
 NORM_NONE, NORM_LAYER, NORM_RMS = range(3)
 MAX_NORM_GROUPS = 256
+SSM_CHUNK = 128
 DTYPE_CODE = {torch.bfloat16: 0, torch.float32: 1}
 
 _P, _I = c_void_p, c_int
@@ -56,8 +57,9 @@ class Gqa(ctypes.Structure):
 
 
 class Ssm(ctypes.Structure):
-	_fields_ = [(n, _I) for n in ('M', 'rows_per_seq', 'heads', 'vdim', 'state', 'groups', 'taps', 'z_at', 'conv_at', 'dt_at', 'conv_ld')] + [
-		('raw_ld', c_int64)] + [(n, _P) for n in ('raw', 'pos', 'conv_w', 'conv_b', 'dt_bias', 'a', 'd', 'ring', 's', 'u', 'out')] + [('out_ld', c_int64), ('status', _P)]
+	_fields_ = [(n, _I) for n in ('M', 'rows_per_seq', 'heads', 'vdim', 'state', 'groups', 'taps', 'z_at', 'conv_at', 'conv_ld')] + [
+		('raw_ld', c_int64), ('dt_ld', c_int64)] + [(n, _P) for n in ('raw', 'dt', 'pos', 'conv_w', 'conv_b', 'dt_bias', 'a', 'd', 'ring', 's', 'u', 'chunk_s', 'chunk_decay', 'out')] + [
+		('out_ld', c_int64), ('status', _P)]
 
 
 _SIGNATURES = {
@@ -80,12 +82,13 @@ _SIGNATURES = {
 	'dense_gqa_prefill_maps': (c_int, [_I, _I, _I]),
 	'dense_gqa_prefill': (c_int, [_P, _I, _P]),
 	'dense_ssm_step': (c_int, [_P, _P]),
-	'dense_ssm_conv': (c_int, [_P, _P]),
+	'dense_ssm_conv': (c_int, [_P, _I, _P]),
 	'dense_ssm_scan': (c_int, [_P, _P]),
+	'dense_ssm_chunked': (c_int, [_P, _P]),
 }
 
 _lib: Optional[ctypes.CDLL] = None
-launches = 0          # kernels launched through this binding (every entry point below that returns a status is one launch)
+launches = 0          # kernels launched through this binding (an entry point that returns a status is one launch unless its caller says more)
 
 
 def exported_symbols():
@@ -110,9 +113,9 @@ def lib() -> ctypes.CDLL:
 _MESSAGES = {-1: 'invalid argument', -2: 'shape violates a divisibility rule', -4: 'pointer or leading dimension misaligned', -5: 'CUDA error', -6: 'not supported'}
 
 
-def check(code: int, what: str):
+def check(code: int, what: str, kernels: int = 1):
 	global launches
-	launches += 1
+	launches += kernels
 	if code != 0:
 		extra = f' (cudaError {lib().dense_last_cuda_error()})' if code == -5 else ''
 		raise (ValueError if code in (-1, -2, -4) else GptqB200Error)(f'{what}: {_MESSAGES.get(code, "unknown error code")}{extra}')

@@ -332,6 +332,15 @@ __device__ __forceinline__ void epi_pair(const DenseEpi &e, int m, int n, float 
 			Elem<T>::store(o + 1, b);
 			break;
 		}
+		case DENSE_EPI_MIXED:
+			if (n < e.n_q) {
+				T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
+				Elem<T>::store(o, a);
+				Elem<T>::store(o + 1, b);
+			} else {
+				*reinterpret_cast<float2 *>(e.kv_out + (size_t)m * e.n_kv + (n - e.n_q)) = make_float2(a, b);
+			}
+			break;
 		case DENSE_EPI_TABLE: {
 			T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
 			const T *t = reinterpret_cast<const T *>(e.tab) + epi_tab_row(e, m) * e.tab_ld + e.tab_col + n;
@@ -374,7 +383,11 @@ __device__ __forceinline__ void epi_16(const DenseEpi &e, int m, int n, const fl
 		float4 *o = reinterpret_cast<float4 *>(reinterpret_cast<float *>(e.out) + (size_t)m * e.ldo + n);
 #pragma unroll
 		for (int i = 0; i < 4; ++i) o[i] = make_float4(v[4 * i] * e.scale, v[4 * i + 1] * e.scale, v[4 * i + 2] * e.scale, v[4 * i + 3] * e.scale);
-	} else if (e.mode == DENSE_EPI_T) {
+	} else if (e.mode == DENSE_EPI_MIXED && n >= e.n_q) {
+		float4 *o = reinterpret_cast<float4 *>(e.kv_out + (size_t)m * e.n_kv + (n - e.n_q));
+#pragma unroll
+		for (int i = 0; i < 4; ++i) o[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
+	} else if (e.mode == DENSE_EPI_T || e.mode == DENSE_EPI_MIXED) {
 		T *o = reinterpret_cast<T *>(e.out) + (size_t)m * e.ldo + n;
 #pragma unroll
 		for (int i = 0; i < 2; ++i) Elem<T>::store8(o + 8 * i, v + 8 * i);

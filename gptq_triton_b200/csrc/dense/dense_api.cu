@@ -73,8 +73,9 @@ static bool ssm_bad(const SsmArgs &a) {
 	if (a.M < 1 || a.rows_per_seq < 1 || a.M % a.rows_per_seq || a.heads < 1 || a.vdim < 1 || a.state < 1 || a.state > SS_MAX_STATE) return true;
 	if (a.groups < 1 || a.heads % a.groups || a.taps < 1 || a.taps > SS_MAX_TAPS) return true;
 	const int inner = a.heads * a.vdim, channels = inner + 2 * a.groups * a.state;
-	if (a.z_at < 0 || a.conv_at < 0 || a.dt_at < 0 || a.conv_ld < channels || a.z_at + inner > a.raw_ld || a.conv_at + channels > a.raw_ld || a.dt_at + a.heads > a.raw_ld) return true;
-	return !a.raw || !a.pos || !a.conv_w || !a.conv_b || !a.dt_bias || !a.a || !a.d || !a.ring || !a.s || !a.status;
+	if (a.z_at < 0 || a.conv_at < 0 || a.conv_ld < channels || a.z_at + inner > a.raw_ld || a.conv_at + a.conv_ld > a.raw_ld || a.dt_ld < a.heads) return true;
+	if (a.conv_ld % 16 || a.conv_at % 16 || a.z_at % 16 || a.raw_ld % 16) return true;
+	return !a.raw || !a.dt || !a.pos || !a.conv_w || !a.conv_b || !a.dt_bias || !a.a || !a.d || !a.ring || !a.s || !a.status;
 }
 
 }   // namespace gptq
@@ -103,6 +104,10 @@ int dense_matmul(const void *x, int64_t ldx, const void *w, int64_t ldw, int M, 
 		case DENSE_EPI_TABLE:
 			if (!epi->out || epi->ldo < n16 || epi->ldo % 8 || !epi->tab || !epi->tab_token || epi->tab_rows < 1) return GPTQ_ERR_INVALID;
 			if (epi->tab_col < 0 || epi->tab_col % 8 || epi->tab_ld % 8 || epi->tab_ld < epi->tab_col + n16 || !aligned16(epi->tab)) return GPTQ_ERR_ALIGN;
+			break;
+		case DENSE_EPI_MIXED:
+			if (!epi->out || epi->n_q < 16 || epi->n_q % 16 || epi->n_kv % 16 || epi->n_q + epi->n_kv != N || epi->ldo < epi->n_q || epi->ldo % 8) return GPTQ_ERR_INVALID;
+			if (epi->n_kv && !epi->kv_out) return GPTQ_ERR_INVALID;
 			break;
 		case DENSE_EPI_GATED:
 			if (!epi->out || N % 16 || epi->ldo < N / 2 || epi->ldo % 8) return GPTQ_ERR_INVALID;
@@ -213,13 +218,19 @@ int dense_ssm_step(const dense_ssm_t *a, void *stream) {
 	if (!a || ssm_bad(*a) || a->rows_per_seq != 1 || !a->out || a->out_ld < (int64_t)a->heads * a->vdim || a->M > 65535) return GPTQ_ERR_INVALID;
 	return ssm_step_launch(*a, reinterpret_cast<cudaStream_t>(stream));
 }
-int dense_ssm_conv(const dense_ssm_t *a, void *stream) {
-	if (!a || ssm_bad(*a) || !a->u) return GPTQ_ERR_INVALID;
-	return ssm_conv_launch(*a, reinterpret_cast<cudaStream_t>(stream));
+int dense_ssm_conv(const dense_ssm_t *a, int dtype, void *stream) {
+	if (!a || ssm_bad(*a) || !a->u || !aligned16(a->u) || !aligned16(a->raw) || (dtype != 0 && dtype != 1)) return GPTQ_ERR_INVALID;
+	return ssm_conv_launch(*a, dtype, reinterpret_cast<cudaStream_t>(stream));
 }
 int dense_ssm_scan(const dense_ssm_t *a, void *stream) {
 	if (!a || ssm_bad(*a) || !a->u || !a->out || a->out_ld < (int64_t)a->heads * a->vdim) return GPTQ_ERR_INVALID;
 	return ssm_scan_launch(*a, reinterpret_cast<cudaStream_t>(stream));
+}
+int dense_ssm_chunked(const dense_ssm_t *a, void *stream) {
+	if (!a || ssm_bad(*a) || !a->u || !a->out || a->out_ld % 2 || a->out_ld < (int64_t)a->heads * a->vdim || !a->chunk_s || !a->chunk_decay) return GPTQ_ERR_INVALID;
+	if (!aligned16(a->u) || !aligned16(a->raw) || !aligned16(a->out)) return GPTQ_ERR_ALIGN;
+	if ((long long)(a->M / a->rows_per_seq) * ((a->rows_per_seq + SS_CHUNK - 1) / SS_CHUNK) > 65535) return GPTQ_ERR_UNSUPPORTED;
+	return ssm_chunk_launch(*a, reinterpret_cast<cudaStream_t>(stream));
 }
 
 }   // extern "C"

@@ -1,4 +1,5 @@
-// Selective state-space recurrence (Mamba-2) token by token, fp32 throughout: decode steps and portions of any length.
+// Selective state-space recurrence (Mamba-2) token by token, fp32 throughout: decode steps and portions of any length.  (Longer
+// bf16 portions run in chunks, ssm_chunk.cu, behind the same convolution.)
 //
 //   ssm_step   one token per sequence: convolution, state update, output and gate in one kernel
 //   ssm_conv   portions: convolution and silu of all channels
@@ -18,8 +19,6 @@ namespace {
 constexpr int SS_RW = 4;                          // state rows per warp
 constexpr int SS_PV = SS_RW * DN_WARPS;           // value entries per CTA
 constexpr int SS_TB = 16;                         // tokens per staged block
-
-__device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
 struct Slice {                                    // channels that a CTA works on, in the order [x slice | B | C]
 	int x0, nx, b0, c0, N;
@@ -115,8 +114,8 @@ __global__ void __launch_bounds__(DN_THREADS) ssm_step_kernel(const SsmArgs p) {
 	pdl_wait();
 	pdl_trigger();
 	if (bad_position(p, pos)) return;
-	const float *raw = p.raw + (size_t)m * p.raw_ld;
-	const float dt_raw = __ldcg(raw + p.dt_at + head);
+	const float *raw = reinterpret_cast<const float *>(p.raw) + (size_t)m * p.raw_ld;
+	const float dt_raw = __ldcg(p.dt + (size_t)m * p.dt_ld + head);
 	const int row = p0 + warp * SS_RW + lane;     // lanes below SS_RW finish a row
 	const float z = lane < SS_RW && row < p.vdim ? __ldcg(raw + p.z_at + head * p.vdim + row) : 0.f;
 #pragma unroll
@@ -130,7 +129,7 @@ __global__ void __launch_bounds__(DN_THREADS) ssm_step_kernel(const SsmArgs p) {
 		}
 	}
 	__syncthreads();
-	const float dt = softplus(dt_raw + bias), decay = expf(a * dt);
+	const float dt = ssm_softplus(dt_raw + bias), decay = expf(a * dt);
 	float x[SS_RW], y[SS_RW];
 #pragma unroll
 	for (int r = 0; r < SS_RW; ++r) x[r] = warp * SS_RW + r < sl.nx ? s_u[warp * SS_RW + r] : 0.f;
@@ -141,41 +140,59 @@ __global__ void __launch_bounds__(DN_THREADS) ssm_step_kernel(const SsmArgs p) {
 		if (lane == r && row < p.vdim) p.out[(size_t)m * p.out_ld + head * p.vdim + row] = fmaf(d, x[r], y[r]) * silu_exact(z);
 }
 
-// thread per channel, a window of W >= taps inputs in registers over a block of tokens
-template <int W>
+template <typename T> __device__ __forceinline__ float2 load2(const T *p);
+template <> __device__ __forceinline__ float2 load2<float>(const float *p) { return __ldcg(reinterpret_cast<const float2 *>(p)); }
+template <> __device__ __forceinline__ float2 load2<bf16>(const bf16 *p) {
+	const uint32_t v = __ldcg(reinterpret_cast<const uint32_t *>(p));
+	return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xFFFF0000u));
+}
+__device__ __forceinline__ void store2(float *p, float2 v) { *reinterpret_cast<float2 *>(p) = v; }
+__device__ __forceinline__ void store2(bf16 *p, float2 v) { *reinterpret_cast<uint32_t *>(p) = pack_bf16(v.x, v.y); }
+
+// thread per pair of channels, a window of W >= taps inputs in registers over a block of tokens
+template <typename T, int W>
 __global__ void __launch_bounds__(DN_THREADS) ssm_conv_kernel(const SsmArgs p, int block) {
-	const int c = blockIdx.x * DN_THREADS + threadIdx.x, t0 = blockIdx.y * block, seq = blockIdx.z, T = p.rows_per_seq;
-	const int channels = p.heads * p.vdim + 2 * p.groups * p.state;
-	if (c >= channels) return;
-	float w[W], in[W];                            // in[W - 1]: the current token
+	constexpr int U = 8;                          // tokens whose inputs are requested together
+	const int c = (blockIdx.x * DN_THREADS + threadIdx.x) * 2, t0 = blockIdx.y * block, seq = blockIdx.z, n = p.rows_per_seq;
+	if (c >= p.heads * p.vdim + 2 * p.groups * p.state) return;          // (rows are padded to an even number)
+	const float2 zero = make_float2(0.f, 0.f);
+	float2 w[W], in[W];                           // in[W - 1]: the current token
 #pragma unroll
-	for (int k = 0; k < W; ++k) w[k] = W - 1 - k < p.taps ? __ldg(p.conv_w + (size_t)(p.taps - W + k) * p.conv_ld + c) : 0.f;
-	const float b = __ldg(p.conv_b + c);
+	for (int k = 0; k < W; ++k) w[k] = W - 1 - k < p.taps ? __ldg(reinterpret_cast<const float2 *>(p.conv_w + (size_t)(p.taps - W + k) * p.conv_ld + c)) : zero;
+	const float2 b = __ldg(reinterpret_cast<const float2 *>(p.conv_b + c));
 	pdl_wait();
 	pdl_trigger();
-	const int start = __ldcg(p.pos + (size_t)seq * T);
+	const int start = __ldcg(p.pos + (size_t)seq * n);
 	if (start < 0) {
 		atomicExch(p.status, DN_BAD_POSITION);
 		return;
 	}
-	const float *raw = p.raw + (size_t)seq * T * p.raw_ld + p.conv_at + c;
-	float *u = p.u + (size_t)seq * T * p.conv_ld + c;
+	const T *raw = reinterpret_cast<const T *>(p.raw) + (size_t)seq * n * p.raw_ld + p.conv_at + c;
+	T *u = reinterpret_cast<T *>(p.u) + (size_t)seq * n * p.conv_ld + c;
 	auto input = [&](int t) {                     // of this portion, of the ring, or zero before the sequence
-		if (t >= 0) return __ldcg(raw + (size_t)t * p.raw_ld);
-		return start + t >= 0 ? __ldcg(p.ring + ((size_t)seq * p.taps + (start + t) % p.taps) * p.conv_ld + c) : 0.f;
+		if (t >= 0) return load2<T>(raw + (size_t)t * p.raw_ld);
+		return start + t >= 0 ? load2<float>(p.ring + ((size_t)seq * p.taps + (start + t) % p.taps) * p.conv_ld + c) : zero;
 	};
 #pragma unroll
-	for (int k = 0; k < W - 1; ++k) in[k + 1] = W - 1 - k < p.taps ? input(t0 + k - (W - 1)) : 0.f;
-	const int t1 = min(t0 + block, T);
-#pragma unroll 4
-	for (int t = t0; t < t1; ++t) {
+	for (int k = 0; k < W - 1; ++k) in[k + 1] = W - 1 - k < p.taps ? input(t0 + k - (W - 1)) : zero;
+	const int t1 = min(t0 + block, n);
+	for (int t = t0; t < t1; t += U) {
+		float2 next[U];
 #pragma unroll
-		for (int k = 0; k < W - 1; ++k) in[k] = in[k + 1];
-		in[W - 1] = __ldcg(raw + (size_t)t * p.raw_ld);
-		float v = b;
+		for (int j = 0; j < U; ++j) next[j] = t + j < t1 ? load2<T>(raw + (size_t)(t + j) * p.raw_ld) : zero;
 #pragma unroll
-		for (int k = 0; k < W; ++k) v = fmaf(w[k], in[k], v);
-		u[(size_t)t * p.conv_ld] = silu_exact(v);
+		for (int j = 0; j < U; ++j) {
+#pragma unroll
+			for (int k = 0; k < W - 1; ++k) in[k] = in[k + 1];
+			in[W - 1] = next[j];
+			float2 v = b;
+#pragma unroll
+			for (int k = 0; k < W; ++k) {
+				v.x = fmaf(w[k].x, in[k].x, v.x);
+				v.y = fmaf(w[k].y, in[k].y, v.y);
+			}
+			if (t + j < t1) store2(u + (size_t)(t + j) * p.conv_ld, make_float2(silu_exact(v.x), silu_exact(v.y)));
+		}
 	}
 }
 
@@ -193,7 +210,7 @@ __global__ void __launch_bounds__(DN_THREADS) ssm_scan_kernel(const SsmArgs p) {
 	if (bad_position(p, start)) return;
 	State<NI> st;
 	st.load(s, p0 + warp * SS_RW, p.vdim, p.state, lane, start == 0);
-	const float *raw = p.raw + (size_t)seq * T * p.raw_ld, *u = p.u + (size_t)seq * T * p.conv_ld;
+	const float *raw = reinterpret_cast<const float *>(p.raw) + (size_t)seq * T * p.raw_ld, *u = reinterpret_cast<const float *>(p.u) + (size_t)seq * T * p.conv_ld;
 	const int row = p0 + warp * SS_RW + lane;
 	for (int t0 = 0; t0 < T; t0 += SS_TB) {
 		const int nt = min(SS_TB, T - t0), n = sl.count();
@@ -207,7 +224,7 @@ __global__ void __launch_bounds__(DN_THREADS) ssm_scan_kernel(const SsmArgs p) {
 			s_z[t][k] = silu_exact(__ldcg(raw + (size_t)(t0 + t) * p.raw_ld + p.z_at + sl.x0 + k));
 		}
 		if (tid < nt) {
-			const float dt = softplus(__ldcg(raw + (size_t)(t0 + tid) * p.raw_ld + p.dt_at + head) + bias);
+			const float dt = ssm_softplus(__ldcg(p.dt + ((size_t)seq * T + t0 + tid) * p.dt_ld + head) + bias);
 			s_dt[tid] = dt;
 			s_decay[tid] = expf(a * dt);
 		}
@@ -241,15 +258,18 @@ int ssm_step_launch(const SsmArgs &p, cudaStream_t stream) {
 	return dn_launch(ssm_step_kernel<8>, grid, block, 0, stream, p);
 }
 
-int ssm_conv_launch(const SsmArgs &p, cudaStream_t stream) {
-	const int channels = p.heads * p.vdim + 2 * p.groups * p.state, cb = (channels + DN_THREADS - 1) / DN_THREADS, seqs = p.M / p.rows_per_seq;
+template <typename T>
+static int conv_launch(const SsmArgs &p, cudaStream_t stream) {
+	const int pairs = (p.heads * p.vdim + 2 * p.groups * p.state + 1) / 2, cb = (pairs + DN_THREADS - 1) / DN_THREADS, seqs = p.M / p.rows_per_seq;
 	int block = 64;                               // tokens per CTA: fewer when that leaves SMs idle
 	while (block > 8 && (long long)cb * seqs * ((p.rows_per_seq + block - 1) / block) < 4 * dn_sm_count()) block /= 2;
 	const dim3 grid(cb, (p.rows_per_seq + block - 1) / block, seqs), threads(DN_THREADS);
-	if (p.taps <= 4) return dn_launch(ssm_conv_kernel<4>, grid, threads, 0, stream, p, block);
-	if (p.taps <= 8) return dn_launch(ssm_conv_kernel<8>, grid, threads, 0, stream, p, block);
-	return dn_launch(ssm_conv_kernel<16>, grid, threads, 0, stream, p, block);
+	if (p.taps <= 4) return dn_launch(ssm_conv_kernel<T, 4>, grid, threads, 0, stream, p, block);
+	if (p.taps <= 8) return dn_launch(ssm_conv_kernel<T, 8>, grid, threads, 0, stream, p, block);
+	return dn_launch(ssm_conv_kernel<T, 16>, grid, threads, 0, stream, p, block);
 }
+
+int ssm_conv_launch(const SsmArgs &p, int dtype, cudaStream_t stream) { return dtype ? conv_launch<float>(p, stream) : conv_launch<bf16>(p, stream); }
 
 int ssm_scan_launch(const SsmArgs &p, cudaStream_t stream) {
 	const dim3 grid((p.vdim + SS_PV - 1) / SS_PV, p.heads, p.M / p.rows_per_seq), block(DN_THREADS);

@@ -18,6 +18,10 @@ from .cache import Carried
 from .dense import Norm, RMSNorm, Stream, epilogue, pad_to, padded, project_stream
 
 
+# portions of more rows than this per sequence run in chunks (bf16)
+STEP_MAX_ROWS = 8
+
+
 @dataclass(frozen=True)
 class StateSpaceSpec:
 	heads: int
@@ -68,28 +72,50 @@ class StateSpaceMixer(nn.Module):
 
 	def forward(self, stream: Stream, cache, pos: torch.Tensor, rows_per_seq: int, start: Optional[int], control: torch.Tensor, norm: Optional[Norm] = None):
 		"""As GroupedAttention.forward; cache: ring and s, carried on here."""
-		s, dev, M = self.spec, control.device, stream.rows
-		raw = torch.empty((M, self.w_in.shape[0]), dtype=torch.float32, device=dev)
-		x = project_stream(stream, self.w_in, epilogue(_dense.EPI_F32, raw), control, final=norm)
+		s, dev, M, dt = self.spec, control.device, stream.rows, self.w_in.dtype
+		chunked = dt == torch.bfloat16 and rows_per_seq > STEP_MAX_ROWS
+		n, n_dt = self.dt_at, self.w_in.shape[0] - self.dt_at
+		# one matrix product; the step sizes stay fp32 when the rest becomes bf16
+		raw = torch.empty((M, n if chunked else n + n_dt), dtype=dt if chunked else torch.float32, device=dev)
+		steps = torch.empty((M, n_dt), dtype=torch.float32, device=dev) if chunked else raw[:, n:]
+		e = epilogue(_dense.EPI_MIXED if chunked else _dense.EPI_F32, raw)
+		if chunked:
+			e.n_q, e.n_kv, e.kv_out = n, n_dt, ptr(steps)
+		x = project_stream(stream, self.w_in, e, control, final=norm)
 		inner = padded(s.inner)
 		out = (torch.empty if inner == s.inner else torch.zeros)((M, inner), dtype=torch.float32, device=dev)
-		a = self.arguments(raw, cache, pos, rows_per_seq, out, control)
+		a = self.arguments(raw, steps, cache, pos, rows_per_seq, out, control)
 		lib, st = _dense.lib(), stream_ptr(dev)
 		if rows_per_seq == 1:
 			_dense.check(lib.dense_ssm_step(ctypes.byref(a), st), 'dense_ssm_step')
 		else:
-			u = torch.empty((M, padded(s.channels)), dtype=torch.float32, device=dev)
-			a.u = ptr(u)
-			_dense.check(lib.dense_ssm_conv(ctypes.byref(a), st), 'dense_ssm_conv')
-			_dense.check(lib.dense_ssm_scan(ctypes.byref(a), st), 'dense_ssm_scan')
+			scratch = self.portion_buffers(a, raw.dtype, chunked)      # noqa: F841 (alive until the launches)
+			_dense.check(lib.dense_ssm_conv(ctypes.byref(a), _dense.DTYPE_CODE[raw.dtype], st), 'dense_ssm_conv')
+			if chunked:
+				_dense.check(lib.dense_ssm_chunked(ctypes.byref(a), st), 'dense_ssm_chunked', 3)
+			else:
+				_dense.check(lib.dense_ssm_scan(ctypes.byref(a), st), 'dense_ssm_scan')
 		y = torch.empty((M, self.w_o.shape[0]), dtype=torch.float32, device=dev)
 		project_stream(Stream(s.inner, inner, stream.eps, x=out), self.w_o, epilogue(_dense.EPI_F32, y), control, keep=False, final=self.norm)
 		return x, y
 
-	def arguments(self, raw, cache, pos, rows_per_seq: int, out, control) -> '_dense.Ssm':
+	def arguments(self, raw, steps, cache, pos, rows_per_seq: int, out, control) -> '_dense.Ssm':
 		s, a = self.spec, _dense.Ssm()
 		a.M, a.rows_per_seq, a.heads, a.vdim, a.state, a.groups, a.taps = pos.numel(), rows_per_seq, s.heads, s.vdim, s.state, s.groups, s.taps
-		a.z_at, a.conv_at, a.dt_at, a.conv_ld, a.raw_ld = 0, self.conv_at, self.dt_at, padded(s.channels), raw.stride(0)
-		a.raw, a.pos, a.conv_w, a.conv_b, a.dt_bias, a.a, a.d = ptr(raw), ptr(pos), ptr(self.conv_w), ptr(self.conv_b), ptr(self.dt_bias), ptr(self.a), ptr(self.d)
+		a.z_at, a.conv_at, a.conv_ld, a.raw_ld, a.dt_ld = 0, self.conv_at, padded(s.channels), raw.stride(0), steps.stride(0)
+		a.raw, a.dt, a.pos, a.conv_w, a.conv_b, a.dt_bias, a.a, a.d = ptr(raw), ptr(steps), ptr(pos), ptr(self.conv_w), ptr(self.conv_b), ptr(self.dt_bias), ptr(self.a), ptr(self.d)
 		a.ring, a.s, a.out, a.out_ld, a.status = ptr(cache['ring']), ptr(cache['s']), ptr(out), out.stride(0), _dense.status_ptr(control)
 		return a
+
+	def portion_buffers(self, a: '_dense.Ssm', dtype: torch.dtype, chunked: bool):
+		"""Scratch of a portion, entered into `a`; returns what must stay alive."""
+		s, dev = self.spec, self.w_in.device
+		u = torch.empty((a.M, a.conv_ld), dtype=dtype, device=dev)
+		a.u = ptr(u)
+		if not chunked:
+			return (u,)
+		n = a.M // a.rows_per_seq * ((a.rows_per_seq + _dense.SSM_CHUNK - 1) // _dense.SSM_CHUNK)
+		states = torch.empty((n, s.heads, s.vdim, s.state), dtype=torch.float32, device=dev)
+		decay = torch.empty((n, s.heads), dtype=torch.float32, device=dev)
+		a.chunk_s, a.chunk_decay = ptr(states), ptr(decay)
+		return u, states, decay

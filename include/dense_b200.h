@@ -30,6 +30,8 @@ extern "C" {
 #define DENSE_EPI_LOGITS  4            /* F32, and with `best` set the greedy choice per row (decode rows only) */
 #define DENSE_EPI_TABLE   5            /* out in the activation dtype = act(result) * tab[token, tab_col + n] */
 
+#define DENSE_EPI_MIXED   6            /* the first n_q columns in the activation dtype to out, n_kv further ones in fp32 to kv_out [M, n_kv] */
+
 /* activations of GATED and TABLE */
 #define DENSE_ACT_SILU 0
 #define DENSE_ACT_GELU 1               /* the tanh form */
@@ -157,24 +159,28 @@ typedef struct {
 	int *status;
 } dense_gqa_t;
 
-/* Selective state-space recurrence with a short causal convolution in front (Mamba-2).  A raw row is fp32
- * [z: inner | x: inner, B: groups * state, C: groups * state | dt: heads], inner = heads * vdim, sections at z_at, conv_at, dt_at.
+/* Selective state-space recurrence with a short causal convolution in front (Mamba-2).  A raw row is
+ * [z: inner | x: inner, B: groups * state, C: groups * state], inner = heads * vdim, sections at z_at and conv_at; dt is separate.
  *   u = silu(conv(x, B, C) + conv_b);  dt = softplus(dt + dt_bias);  S = exp(a * dt) S + dt x B^T;  y = S C + d * x;  out = y * silu(z)
  * The last `taps` convolution inputs of a sequence are kept in a ring (slot = position mod taps).  At position 0 the state and
  * the inputs before it are taken as zero, whatever the buffers hold. */
+#define DENSE_SSM_CHUNK 128
 typedef struct {
 	int M, rows_per_seq;
 	int heads, vdim, state, groups, taps;
-	int z_at, conv_at, dt_at, conv_ld; /* conv_ld: padded number of convolution channels */
-	int64_t raw_ld;
-	const float *raw;                  /* [M, raw_ld] */
+	int z_at, conv_at, conv_ld;        /* conv_ld: padded number of convolution channels */
+	int64_t raw_ld, dt_ld;
+	const void *raw;                   /* [M, raw_ld] */
+	const float *dt;                   /* [M, dt_ld] */
 	const int32_t *pos;                /* [M] */
 	const float *conv_w, *conv_b;      /* [taps, conv_ld] (last tap: the current token), [conv_ld] */
 	const float *dt_bias, *a, *d;      /* [heads] */
 	float *ring;                       /* [sequences, taps, conv_ld] */
 	float *s;                          /* [sequences, heads, vdim, state] */
-	float *u;                          /* scratch of portions: [M, conv_ld] */
-	float *out;                        /* [M, out_ld] fp32 */
+	void *u;                           /* scratch of portions: [M, conv_ld], the type of raw */
+	float *chunk_s;                    /* scratch of dense_ssm_chunked: [sequences, chunks, heads, vdim, state] */
+	float *chunk_decay;                /* [sequences, chunks, heads] */
+	float *out;                        /* [M, out_ld] */
 	int64_t out_ld;
 	int *status;
 } dense_ssm_t;
@@ -207,9 +213,10 @@ int dense_gqa_merge(const dense_gqa_t *args, int dtype, void *stream);       /* 
 int dense_gqa_prefill_maps(int maps, int dim, int vdim);
 int dense_gqa_prefill(const dense_gqa_t *args, int start, void *stream);
 
-int dense_ssm_step(const dense_ssm_t *args, void *stream);                   /* rows_per_seq = 1 */
-int dense_ssm_conv(const dense_ssm_t *args, void *stream);                   /* portions: u */
-int dense_ssm_scan(const dense_ssm_t *args, void *stream);                   /* portions: out, state, ring */
+int dense_ssm_step(const dense_ssm_t *args, void *stream);                   /* rows_per_seq = 1, raw fp32 */
+int dense_ssm_conv(const dense_ssm_t *args, int dtype, void *stream);        /* portions: u */
+int dense_ssm_scan(const dense_ssm_t *args, void *stream);                   /* portions, raw and u fp32: out, state, ring, token by token */
+int dense_ssm_chunked(const dense_ssm_t *args, void *stream);                /* the same for bf16 raw and u in chunks (three kernels) */
 
 #ifdef __cplusplus
 }

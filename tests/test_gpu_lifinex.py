@@ -293,7 +293,7 @@ def test_state_space_prompt_portions_and_steps(control, dtype, H, P, N, G, taps,
 		for n in cuts:
 			out.append(run_mixer(mix, cache, h[p:p + n], p, control, decode=n == 1))
 			p += n
-		assert err(torch.cat(out), ref) <= (1e-5 if dtype == F32 else 1.5e-2), cuts
+		assert err(torch.cat(out), ref) <= (1e-5 if dtype == F32 else 3e-2), cuts
 
 
 @pytest.mark.parametrize('dtype', [F32, B16])
@@ -309,7 +309,9 @@ def test_one_input_that_the_state_must_keep(control, dtype, at):
 	w_in = W['in'].clone()
 	w_in[-H:] = 0
 	w_in[-H:, 0] = 1.0                                             # dt is large at this token only
-	W = {**W, 'in': w_in, 'dt_bias': torch.full((H,), -9.0).bfloat16(), 'A_log': torch.full((H,), -9.0).bfloat16(), 'D': torch.zeros(H).bfloat16()}
+	bias = W['conv.b'].clone()
+	bias[H * P:] = 1.5                                             # B and C point the same way: their product does not vanish by chance
+	W = {**W, 'in': w_in, 'conv.b': bias, 'dt_bias': torch.full((H,), -9.0).bfloat16(), 'A_log': torch.full((H,), -9.0).bfloat16(), 'D': torch.zeros(H).bfloat16()}
 	ref = O.mamba2(h.double(), double(W), mixer, 1e-5)
 	quiet = O.mamba2(torch.cat([h[:at], h[at:at + 1] * 0, h[at + 1:]]).double(), double(W), mixer, 1e-5)
 	assert at > 390 or float((ref - quiet)[-1].abs().max()) > 0.5 * float(ref[-1].abs().max())
@@ -321,8 +323,7 @@ def test_one_input_that_the_state_must_keep(control, dtype, at):
 		for n in cuts:
 			out.append(run_mixer(mix, cache, h[p:p + n], p, control, decode=n == 1))
 			p += n
-		# (heads of a group share B . C, which is small at some tokens: the norm magnifies what rounding leaves there)
-		assert err(torch.cat(out), ref) <= (2e-4 if dtype == F32 else 2e-2), cuts
+		assert err(torch.cat(out), ref) <= (2e-5 if dtype == F32 else 3e-2), cuts
 
 
 @pytest.mark.parametrize('dtype', [F32, B16])
@@ -339,7 +340,7 @@ def test_states_that_forget_at_once_and_never(control, dtype):
 		for n in cuts:
 			out.append(run_mixer(mix, cache, h[p:p + n], p, control, decode=n == 1))
 			p += n
-		assert err(torch.cat(out), ref) <= (2e-5 if dtype == F32 else 2e-2), cuts
+		assert err(torch.cat(out), ref) <= (2e-5 if dtype == F32 else 4e-2), cuts
 
 
 # ---- whole models ------------------------------------------------------------------------------------------------------------

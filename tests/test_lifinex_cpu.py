@@ -155,7 +155,7 @@ def test_arguments_are_refused_on_the_host(lib):
 	a.maps = 3
 	assert lib.dense_gqa_append(ctypes.byref(a), 0, None) == -1
 	s = _dense.Ssm()
-	assert lib.dense_ssm_step(ctypes.byref(s), None) == -1 and lib.dense_ssm_conv(None, None) == -1 and lib.dense_ssm_scan(ctypes.byref(s), None) == -1
+	assert lib.dense_ssm_step(ctypes.byref(s), None) == -1 and lib.dense_ssm_conv(None, 0, None) == -1 and lib.dense_ssm_chunked(ctypes.byref(s), None) == -1 and lib.dense_ssm_scan(ctypes.byref(s), None) == -1
 	r = _dense.Rows()
 	r.x_in, r.width, r.ld, r.eps, r.status, r.fin_norm, r.fin_groups = p, 48, 48, 1e-5, p, _dense.NORM_RMS, 5
 	assert lib.dense_prepare_rows(ctypes.byref(r), 1, ctypes.c_void_p(p), 48, 0, None) == -1          # 48 entries in 5 parts
