@@ -1109,6 +1109,13 @@ def befalix_config(G, layers, hid, inter, H, D, R, V, C, vocab=32000):
 	return G.BefalixConfig.from_dict({'vocab': vocab, 'width': hid, 'norm': {'eps': 1e-6}, 'residual_mult': 1.0, 'logit_scale': 1.0, 'layers': [layer] * layers})
 
 
+def befalix_work(model, layers: int, ctx: int, t: int):
+	"""(bytes of a decode step at context ctx, operations of a prompt of t tokens)."""
+	s = model.layers[0].mixer.spec
+	nbytes = sum(b.numel() * b.element_size() for b in model.buffers()) + layers * ctx * s.row * 2
+	return nbytes, t * 2.0 * sum(b.numel() for l in model.layers for b in l.buffers() if b.dim() == 2) + layers * float(t) * (t + 1) * s.heads * (s.dim + s.rot_dim + s.vdim)
+
+
 def befalix_arm(args):
 	"""Prints one JSON line: per size, prompt tokens/s and decode ms per step of a Befalix model (bf16 weights, random) and of a
 	4-bit LLaMA with the same hidden size, MLP, heads and number of layers, and every kernel's fraction of its roofline."""
@@ -1132,8 +1139,7 @@ def befalix_arm(args):
 		model = G.synthetic_befalix(cfg, seed=1, device=dev)
 		engine = G.BefalixEngine(model, batch=1, max_seq=max_seq)
 		rate, ms = engine_rates(engine, cfg.vocab_size, args.steps)
-		nbytes = sum(b.numel() * b.element_size() for b in model.buffers()) + layers * (PROMPT + args.steps // 2) * model.layers[0].mixer.spec.row * 2
-		flops = PROMPT * 2.0 * sum(b.numel() for l in model.layers for n, b in l.named_buffers() if b.dim() == 2) + layers * float(PROMPT) * (PROMPT + 1) * H * (D + R + V)
+		nbytes, flops = befalix_work(model, layers, PROMPT + args.steps // 2, PROMPT)
 		rec = {'hidden': hid, 'intermediate': inter, 'heads': H, 'layers': layers,
 			   'befalix': {'prefill_tokens_s': round(rate), 'decode_ms_per_step': round(ms, 4), 'decode_tokens_s': round(1e3 / ms, 1), 'decode_frac_hbm': round(nbytes / ms / 1e6 / hbm, 3),
 						   'prefill_frac_tensor': round(flops * rate / PROMPT / 1e12 / tflops, 3), 'kernels': befalix_kernels(G, engine, hbm, tflops)}}
@@ -1156,6 +1162,209 @@ def befalix_arm(args):
 					  'peak_source': source, 'kernel_status': _lib.kernel_status(dev), 'clocks': sampler.stop(), 'cases': cases}))
 
 
+# ------------------------------------------------------------------------------------------
+# --workload lifinex: differential attention and state-space layers beside the latent-attention design at equal size
+# ------------------------------------------------------------------------------------------
+def lifinex_config(G, runs, hid, inter, vocab=32000, max_positions=4096):
+	"""`runs` layer runs, attention and state-space layers in turn (runs = 8: six layers, two of them run twice)."""
+	ff = {'kind': 'dense', 'ff': inter}
+	H = hid // 128
+	att = {'type': 'attention', 'mlp': ff, 'mixer': {'heads': H, 'kv_heads': H // 4, 'dim': 64, 'vdim': 128, 'scale': 0.125, 'softcap': 30.0, 'diff': 0.3}}
+	ssm = {'type': 'mamba2', 'mlp': ff, 'mixer': {'heads': hid // 32, 'vdim': 64, 'state': 128, 'groups': 8, 'conv': 4, 'norm_groups': 8}}
+	layers, loop = {8: ([att, ssm] * 3, (2, 4, 2)), 4: ([ssm, att, ssm], (1, 2, 2)), 2: ([att, ssm], (0, 1, 1))}[runs]
+	return G.LifinexConfig.from_dict({'vocab': vocab, 'width': hid, 'layers': layers, 'norm': {'eps': 1e-6}, 'max_positions': max_positions, 'token_side': {'dim': 256},
+									  'loop': dict(zip(('start', 'stop', 'times'), loop))})
+
+
+def lifinex_work(model, ctx: int, t: int):
+	"""(bytes of a decode step at context ctx, operations of a prompt of t tokens) that the design needs: weights as often as
+	their layers run, cache rows, carried state (read and written); products, both attention maps, the recurrence's state
+	update and output."""
+	cfg = model.config
+	size = lambda m: sum(b.numel() * b.element_size() for b in m.buffers())
+	mats = lambda m: sum(b.numel() for b in m.buffers() if b.dim() == 2 and b.shape[0] > 32)
+	nbytes, flops = model.head.numel() * 2, 0.0
+	for i, entry in cfg.runs():
+		layer, s = model.layers[i], cfg.layers[i].mixer
+		nbytes += size(layer)
+		flops += 2.0 * t * mats(layer)
+		if entry is not None:
+			nbytes += model.loop_x.numel() * 2
+			flops += 2.0 * t * model.loop_x.numel()
+		if hasattr(s, 'softcap'):
+			nbytes += ctx * s.kv_heads * (s.maps * s.dim + s.vdim) * 2
+			flops += float(t) * (t + 1) * s.heads * s.maps * (s.dim + s.vdim)
+		else:
+			nbytes += 2 * s.heads * s.vdim * s.state * 4
+			flops += 4.0 * t * s.heads * s.vdim * s.state
+	if cfg.loop is not None:
+		nbytes += model.loop_x0.numel() * 2
+		flops += 2.0 * t * model.loop_x0.numel()
+	return nbytes, flops
+
+
+def lifinex_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: int = PROMPT):
+	"""Every kernel of the design alone, on rotating copies of its operands (see befalix_kernels)."""
+	import ctypes
+	import torch
+	from gptq_triton_b200 import _dense
+	from gptq_triton_b200._lib import stream_ptr
+	from gptq_triton_b200.cache import StaticCache
+	from gptq_triton_b200.dense import Stream, epilogue, linear, matmul, padded, prepare_rows, project_stream
+	m, cfg, dev, ctl = engine.model, engine.cfg, engine.device, engine.control
+	lib, sp = _dense.lib(), lambda: stream_ptr(dev)
+	W, bf = m.embed.shape[1], torch.bfloat16
+	att = next(l for l in m.layers if hasattr(l.mixer, 'lam'))
+	ssm = next(l for l in m.layers if not hasattr(l.mixer, 'lam'))
+	out = {}
+
+	def record(name, us, nbytes=None, flops=None):
+		r = {'us': round(us, 2)}
+		if nbytes is not None:
+			r['frac_hbm'] = round(nbytes / us / 1e3 / hbm, 3)
+		if flops is not None:
+			r['frac_tensor'] = round(flops / us / 1e6 / tflops, 3)
+		out[name] = r
+	esz = lambda *ws: sum(w.numel() * w.element_size() for w in ws)
+	copies = lambda w, limit=320e6: [w] + [w.clone() for _ in range(max(3, min(80, int(limit / esz(w)))))]
+	call = lambda fn, *a: _dense.check(fn(*a, sp()), 'bench')
+
+	def rows(M):
+		return Stream(cfg.width, W, cfg.norm_eps).then(torch.randn((M, W), device=dev), torch.randn((M, W), device=dev))
+	for M, phase in ((1, 'decode'), (t, 'prompt')):
+		decode = M == 1
+		st = rows(M)
+		h = torch.randn((M, W), device=dev).to(bf)
+		start = ctx if decode else 0
+		pos = torch.arange(start, start + M, dtype=torch.int32, device=dev)
+
+		def gemm(name, w, epi, norm=None, x=None):
+			if decode and x is None:          # the kernel forms its rows itself
+				fns = [lambda c=c: project_stream(st, c, epi, ctl, final=norm) for c in copies(w)]
+			else:
+				xin = h if x is None else x
+				fns = [lambda c=c: matmul(xin, c, epi, ctl) for c in copies(w)]
+			record(f'{phase} {name}', graph_us(fns), **({'nbytes': esz(w)} if decode else {'flops': 2.0 * M * w.numel()}))
+		f32 = lambda n: torch.empty((M, n), device=dev)
+		if not decode:
+			record('prompt rows (residual, norm)', graph_us([lambda: prepare_rows(st, ctl, bf, True, att.mixer_norm)] * 4), t * W * (4 + 4 + 4 + 2))
+		# ---- attention ----
+		mx, s = att.mixer, att.mixer.spec
+		raw = torch.randn((M, mx.w_in.shape[0]), device=dev)
+		gemm('attention in-projection', mx.w_in, epilogue(_dense.EPI_F32, raw), att.mixer_norm)
+		n = max(2, min(80, int(320e6 / (ctx * s.kv_heads * (s.maps * mx.D + mx.V) * 2)))) if decode else 2
+		caches = [{k: torch.randn_like(v.float()).to(bf) for k, v in StaticCache([s.cache_layout(engine.max_seq)], 1, bf, dev)[0].items()} for _ in range(n)]
+		o = torch.empty((M, s.heads * mx.V), dtype=bf, device=dev)
+		keep, args = [], []
+		for c in caches:
+			a = mx.arguments(raw, c, pos, M, cfg.norm_eps, ctl)
+			keep.append(mx.buffers(a, o, engine.max_seq if decode else 1))
+			args.append(a)
+		row = s.kv_heads * (s.maps * mx.D + mx.V)
+		if decode:
+			call(lib.dense_gqa_append, ctypes.byref(args[0]), 0)
+			record('decode attention norms, cache row', graph_us([lambda a=a: call(lib.dense_gqa_append, ctypes.byref(a), 0) for a in args]), esz(raw) * 2)
+			for a in args:
+				call(lib.dense_gqa_append, ctypes.byref(a), 0)
+			record('decode attention', graph_us([lambda a=a: call(lib.dense_gqa_attend, ctypes.byref(a), 0) for a in args]), (ctx + 1) * row * 2)
+			record('decode attention merge', graph_us([lambda a=a: call(lib.dense_gqa_merge, ctypes.byref(a), 0) for a in args]),
+				   s.heads * s.maps * args[0].splits * (mx.V + 2) * 4)
+		else:
+			record('prompt attention norms, cache rows', graph_us([lambda a=a: call(lib.dense_gqa_append, ctypes.byref(a), 0) for a in args] * 2), esz(raw) + M * (row + s.heads * s.maps * mx.D) * 2)
+			record('prompt attention', graph_us([lambda a=a: call(lib.dense_gqa_prefill, ctypes.byref(a), 0) for a in args] * 2), flops=float(t) * (t + 1) * s.heads * s.maps * (s.dim + s.vdim))
+		y = f32(W)
+		gemm('attention out-projection', mx.w_o, epilogue(_dense.EPI_F32, y), x=o)
+		if decode:
+			parts = ['decode attention in-projection', 'decode attention norms, cache row', 'decode attention', 'decode attention merge', 'decode attention out-projection']
+			record('decode attention block (sum)', sum(out[k]['us'] for k in parts), esz(mx.w_in, mx.w_o) + (ctx + 1) * row * 2)
+		# ---- state space ----
+		mx, s = ssm.mixer, ssm.mixer.spec
+		if decode:
+			raw = torch.randn((M, mx.w_in.shape[0]), device=dev)
+			steps, e = raw[:, mx.dt_at:], epilogue(_dense.EPI_F32, raw)
+		else:
+			raw, steps = torch.randn((M, mx.dt_at), device=dev).to(bf), torch.randn((M, mx.w_in.shape[0] - mx.dt_at), device=dev)
+			e = epilogue(_dense.EPI_MIXED, raw)
+			e.n_q, e.n_kv, e.kv_out = mx.dt_at, steps.shape[1], steps.data_ptr()
+		gemm('state-space in-projection', mx.w_in, e, ssm.mixer_norm)
+		state = 4 * s.heads * s.vdim * s.state
+		g = torch.randn((M, padded(s.inner)), device=dev)
+		args = []
+		for _ in range(max(2, min(80, int(320e6 / state))) if decode else 2):
+			c = StaticCache([s.cache_layout()], 1, bf, dev)[0]
+			a = mx.arguments(raw, steps, c, pos, M, g, ctl)
+			keep.append((c, None if decode else mx.portion_buffers(a, bf, True)))
+			args.append(a)
+		if decode:
+			record('decode state-space step', graph_us([lambda a=a: call(lib.dense_ssm_step, ctypes.byref(a)) for a in args]), 2 * state + esz(raw, g) + 4 * (s.taps + 1) * a.conv_ld)
+		else:
+			record('prompt state-space convolution', graph_us([lambda a=a: call(lib.dense_ssm_conv, ctypes.byref(a), 0) for a in args] * 2), M * a.conv_ld * 4)
+			record('prompt state-space recurrence', graph_us([lambda a=a: call(lib.dense_ssm_chunked, ctypes.byref(a)) for a in args] * 2), M * a.conv_ld * 2 + M * s.inner * 6 + esz(steps) + 2 * state)
+			gs = Stream(s.inner, padded(s.inner), cfg.norm_eps, x=g)
+			record('prompt state-space norm', graph_us([lambda: prepare_rows(gs, ctl, bf, False, mx.norm)] * 4), M * s.inner * 6)
+		if decode:
+			gs = Stream(s.inner, padded(s.inner), cfg.norm_eps, x=g)
+			record('decode state-space norm, out-projection', graph_us([lambda c=c: project_stream(gs, c, epilogue(_dense.EPI_F32, y), ctl, keep=False, final=mx.norm) for c in copies(mx.w_o)]),
+				   esz(mx.w_o))
+		else:
+			gemm('state-space out-projection', mx.w_o, epilogue(_dense.EPI_F32, y), x=g.to(bf))
+		# ---- feed-forward, side input, pass entry, logits ----
+		act = torch.empty((M, att.mlp.down.shape[1]), dtype=bf, device=dev)
+		gemm('gate/up', att.mlp.gate_up, att.mlp.gated(act), att.mlp_norm)
+		gemm('down', att.mlp.down, epilogue(_dense.EPI_F32, y), x=act)
+		tok = torch.arange(M, device=dev) % cfg.vocab_size
+		side = torch.empty((M, att.side.gate.shape[0]), dtype=bf, device=dev)
+		gemm('side gate', att.side.gate, att.side.gated(side, m.side, tok))
+		gemm('side projection', att.side.proj, epilogue(_dense.EPI_F32, y), x=side)
+		gemm('pass entry', m.loop_x, epilogue(_dense.EPI_F32, y))
+		if decode:
+			logits = torch.empty((1, padded(cfg.vocab_size)), device=dev)
+			record('decode logits', graph_us([lambda w=w: project_stream(st, w, epilogue(_dense.EPI_LOGITS, logits), ctl, keep=False, final=m.norm) for w in copies(m.head)]), esz(m.head))
+	return out
+
+
+def lifinex_arm(args):
+	"""Prints one JSON line: per size, prompt tokens/s and decode ms per step of a Lifinex model and of a Befalix model (both
+	bf16, random weights) with the same hidden size, MLP and number of layer runs, and every kernel's fraction of its roofline."""
+	import torch
+	import gptq_triton_b200 as G
+	from gptq_triton_b200 import _lib
+	torch.cuda.set_device(0)
+	dev = torch.device('cuda', 0)
+	hbm, source = measured_peaks()
+	peaks = ROOT / 'MEASURED_PEAKS.json'
+	tflops = float(json.load(open(peaks))['bf16_tflops']) if peaks.exists() else 1590.0
+	sampler = ClockSampler(0, None)
+	sampler.start()
+	cases = {}
+	for name, runs, hid, inter, H, D, R, V, C in BEFALIX_CASES:
+		if args.case and name not in args.case.split(','):
+			continue
+		max_seq = PROMPT + args.steps + 64
+		cfg = lifinex_config(G, runs, hid, inter)
+		engine = G.LifinexEngine(G.synthetic_lifinex(cfg, seed=1, device=dev), batch=1, max_seq=max_seq)
+		rate, ms = engine_rates(engine, cfg.vocab_size, args.steps)
+		nbytes, flops = lifinex_work(engine.model, PROMPT + args.steps // 2, PROMPT)
+		rec = {'hidden': hid, 'intermediate': inter, 'layer_runs': runs,
+			   'lifinex': {'prefill_tokens_s': round(rate), 'decode_ms_per_step': round(ms, 4), 'decode_tokens_s': round(1e3 / ms, 1), 'decode_frac_hbm': round(nbytes / ms / 1e6 / hbm, 3),
+						   'prefill_frac_tensor': round(flops * rate / PROMPT / 1e12 / tflops, 3), 'kernels': lifinex_kernels(G, engine, hbm, tflops)}}
+		engine.close()
+		del engine
+		torch.cuda.empty_cache()
+		cfg = befalix_config(G, runs, hid, inter, H, D, R, V, C)
+		engine = G.BefalixEngine(G.synthetic_befalix(cfg, seed=1, device=dev), batch=1, max_seq=max_seq)
+		rate, ms = engine_rates(engine, cfg.vocab_size, args.steps)
+		nbytes, flops = befalix_work(engine.model, runs, PROMPT + args.steps // 2, PROMPT)
+		rec['befalix'] = {'prefill_tokens_s': round(rate), 'decode_ms_per_step': round(ms, 4), 'decode_tokens_s': round(1e3 / ms, 1), 'decode_frac_hbm': round(nbytes / ms / 1e6 / hbm, 3),
+						  'prefill_frac_tensor': round(flops * rate / PROMPT / 1e12 / tflops, 3), 'kernels': befalix_kernels(G, engine, hbm, tflops)}
+		engine.close()
+		del engine
+		torch.cuda.empty_cache()
+		cases[name] = rec
+	print(json.dumps({'workload': 'lifinex', 'prompt': PROMPT, 'batch': 1, 'data': 'synthetic', 'weights': 'bf16 (random)', 'hbm_gbs': hbm, 'bf16_tflops': tflops,
+					  'peak_source': source, 'kernel_status': _lib.kernel_status(dev), 'clocks': sampler.stop(), 'cases': cases}))
+
+
 def main():
 	ap = argparse.ArgumentParser()
 	ap.add_argument('--gpus', type=int, default=1)
@@ -1167,9 +1376,10 @@ def main():
 	ap.add_argument('--no-parity', action='store_true', help='skip the greedy-decoding parity check before the timed region')
 	ap.add_argument('--no-prefill', action='store_true', help='skip the prefill-kernel record')
 	ap.add_argument('--config4', default='auto', choices=['auto', 'on', 'off'], help='also measure the 65B-architecture batch-16 configuration as a sub-record (auto: with 2 or more GPUs)')
-	ap.add_argument('--workload', default='llama7b', choices=['llama7b', 'llama65b-b16', 'befalix'],
-					help='llama65b-b16: 65B architecture, batch 16 (tensor-parallel runs); befalix: latent-attention models beside LLaMA at equal sizes')
-	ap.add_argument('--case', default='', help='befalix: sizes to run (2048, 4096, 8192), separated by commas')
+	ap.add_argument('--workload', default='llama7b', choices=['llama7b', 'llama65b-b16', 'befalix', 'lifinex'],
+					help='llama65b-b16: 65B architecture, batch 16 (tensor-parallel runs); befalix: latent-attention models beside LLaMA at equal sizes; lifinex: '
+						 'differential attention and state-space layers beside befalix at equal sizes')
+	ap.add_argument('--case', default='', help='befalix, lifinex: sizes to run (2048, 4096, 8192), separated by commas')
 	ap.add_argument('--no-graph', action='store_true', help='do not capture the decode step in a CUDA graph')
 	ap.add_argument('--kernel-case', default=None, choices=['gateup', 'qkv', 'o', 'down', 'prefill', 'attn', 'lmhead', 'chain', 'qkvattn', 'latent-prefill', 'latent-decode'], help='profiling aid: run a few launches of one kernel and exit')
 	ap.add_argument('--m', type=int, default=1, help='batch rows for --kernel-case')
@@ -1179,6 +1389,8 @@ def main():
 		kernel_case(args)
 	elif args.workload == 'befalix':
 		befalix_arm(args)
+	elif args.workload == 'lifinex':
+		lifinex_arm(args)
 	elif args.impl == 'reference':
 		reference_arm(args)
 	else:
