@@ -113,6 +113,8 @@ __device__ __forceinline__ float block_sum(float v, float *slot) {
 
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
+// for results that become bf16
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 // 0.5 z (1 + tanh u) with 1 + tanh u = 2 / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_tanh(float z) { return z / (1.f + expf(-1.5957691216057308f * fmaf(0.044715f * z, z * z, z))); }
 __device__ __forceinline__ float activation(int act, float z) { return act == DENSE_ACT_GELU ? gelu_tanh(z) : silu_exact(z); }

@@ -12,9 +12,12 @@
 //                     keys, is an operand whose other dimension is contiguous, so it needs no transposed copy)
 // The weights are split into a bf16 high part and a bf16 remainder, which together take the columns of the fp32 scores they
 // replace; O is rescaled only when a row's maximum has grown by more than 2^8 (see latent_prefill.cu).
-// The soft cap keeps the order of scores, so the maximum is taken before it.  tanh costs two special-function operations when it
-// is built from an exponential and a reciprocal, which would make it three per score with the softmax's own; arguments of at most 1
-// (a warp looks at its own) take a polynomial on the FMA units instead.  Every wait is bounded.
+// Capped scores lie in [-cap, cap]: as long as 2^(cap * log2 e) and its inverse are far from the ends of the fp32 range (and of the
+// bf16 range, which is the same), zero serves as the reference point of every softmax and there is no running maximum.  A larger
+// cap, or none, takes the maximum (before the cap, which keeps the order) as above.
+// tanh costs two special-function operations when it is built from an exponential and a reciprocal, which would make it three per
+// score with the softmax's own; arguments of at most 1 take a polynomial on the FMA units instead, two scores per instruction.
+// That arguments are small follows from the norm weights (`bound`), else a warp looks at its own.  Every wait is bounded.
 #include <algorithm>
 
 #include "gqa.cuh"
@@ -52,6 +55,30 @@ __device__ __forceinline__ float tanh_any(float x) {
 	return fmaf(-2.f, r, 1.f);
 }
 
+// two fp32 operations per instruction
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float a, float b) {
+	f32x2 r;
+	asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+	return r;
+}
+__device__ __forceinline__ void unpack2(f32x2 v, float &a, float &b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+	f32x2 r;
+	asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+	return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+	f32x2 r;
+	asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+	return r;
+}
+__device__ __forceinline__ f32x2 add2(f32x2 a, f32x2 b) {
+	f32x2 r;
+	asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+	return r;
+}
+
 enum { SCORE_PLAIN, SCORE_SMALL, SCORE_ANY };             // no cap, cap with small arguments, cap
 template <int KIND>
 __device__ __forceinline__ float gp_score(float v, float cap2) {
@@ -78,6 +105,48 @@ __device__ __forceinline__ float gp_weights(const float (&s)[32], uint32_t (&out
 	return t0 + t1;
 }
 
+// The same with reference point zero.  SMALL: cap * tanh by the polynomial, its coefficients times the cap; else by the exponential.
+template <bool SMALL>
+__device__ __forceinline__ float gp_weights_fixed(const float (&s)[32], uint32_t (&out)[32], float cap2, bool edge, int last) {
+	f32x2 total = pack2(0.f, 0.f);
+	const float c0 = 9.999993948e-01f * cap2, c1 = -3.332895137e-01f * cap2, c2 = 1.328072065e-01f * cap2, c3 = -5.158598840e-02f * cap2, c4 = 1.672085518e-02f * cap2,
+				c5 = -3.058229038e-03f * cap2;
+#pragma unroll
+	for (int k = 0; k < 16; ++k) {
+		float a, b;
+		if (SMALL) {
+			const f32x2 x = pack2(s[2 * k], s[2 * k + 1]), u = mul2(x, x);
+			f32x2 r = fma2(u, pack2(c5, c5), pack2(c4, c4));
+			r = fma2(r, u, pack2(c3, c3));
+			r = fma2(r, u, pack2(c2, c2));
+			r = fma2(r, u, pack2(c1, c1));
+			r = fma2(r, u, pack2(c0, c0));
+			unpack2(mul2(r, x), a, b);
+		} else {
+			a = cap2 * tanh_any(s[2 * k]);
+			b = cap2 * tanh_any(s[2 * k + 1]);
+		}
+		a = ex2(a);
+		b = ex2(b);
+		if (edge) {
+			a = 2 * k > last ? 0.f : a;
+			b = 2 * k + 1 > last ? 0.f : b;
+		}
+		const f32x2 ab = pack2(a, b);
+		total = add2(total, ab);
+		const uint32_t hi = pack_bf16(a, b);
+		out[k] = hi;
+		float la, lb;
+		unpack2(fma2(pack2(__uint_as_float(hi << 16), __uint_as_float(hi & 0xFFFF0000u)), pack2(-1.f, -1.f), ab), la, lb);
+		out[16 + k] = pack_bf16(la, lb);
+	}
+	float t0, t1;
+	unpack2(total, t0, t1);
+	return t0 + t1;
+}
+
+enum { MODE_PLAIN, MODE_CAP, MODE_FIXED };                // no cap; cap and running maximum; cap and reference point zero
+
 // Descriptor of V as the B operand: the contiguous dimension is N (values).  Chunks of 64 value columns lie GP_CHUNK apart, a
 // chunk holds rows of 128 bytes (one key each) in groups of 8 keys, 1024 bytes apart; 128-byte swizzle.
 __device__ __forceinline__ uint64_t desc_values(uint32_t addr) {
@@ -90,7 +159,7 @@ __device__ __forceinline__ uint64_t desc_values(uint32_t addr) {
 	return d;
 }
 
-template <int MAPS, bool CAP>
+template <int MAPS, int MODE>
 __global__ void __launch_bounds__(MAPS * (GP_MAP_THREADS + 32) + 32, 1) gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_constant__ CUtensorMap tmk,
 																		   const __grid_constant__ CUtensorMap tmv, const GqaArgs p, int t, int start, const GpPlan pl,
 																		   uint32_t tmem_cols) {
@@ -230,6 +299,8 @@ __global__ void __launch_bounds__(MAPS * (GP_MAP_THREADS + 32) + 32, 1) gqa_pref
 		const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
 		const uint32_t ts = tmem + i * GP_T + half * 64 + lane_base, to = tmem + MAPS * GP_T + i * p.vdim + lane_base;
 		const float cap2 = p.cap * GQ_LOG2E;
+		constexpr bool CAP = MODE == MODE_CAP;
+		const bool bounded = p.bound > 0.f && p.bound <= 0.98f;          // (queries and keys are rounded to bf16)
 		float ref = 0.f, sum = 0.f;
 		bool ok = true;
 		auto wait = [&](uint32_t bar, int k) {
@@ -245,6 +316,35 @@ __global__ void __launch_bounds__(MAPS * (GP_MAP_THREADS + 32) + 32, 1) gqa_pref
 			ok = ok && wait(bar_s + 8 * i, j);
 			const int last = pos - j * GP_T - half * 64;                                     // last visible key of this half
 			const bool edge = j * GP_T + half * 64 + 63 > start + q0 + (warp & 3) * 32;      // this warp's first row does not see all of them
+			if (MODE == MODE_FIXED) {
+				if (ok) {
+#pragma unroll 1
+					for (int c = 0; c < 2; ++c) {
+						float s[32];
+						uint32_t out[32];                // 16 columns of high parts, 16 of remainders
+						tmem_ld32(ts + c * 32, s);
+						tmem_ld_wait();
+						tmem_settle(s);
+						bool small = bounded;
+						if (!bounded) {
+							float g0 = fabsf(s[0]), g1 = fabsf(s[1]);
+#pragma unroll
+							for (int k = 2; k < 32; k += 2) {
+								g0 = fmaxf(g0, fabsf(s[k]));
+								g1 = fmaxf(g1, fabsf(s[k + 1]));
+							}
+							small = !__any_sync(0xffffffffu, fmaxf(g0, g1) > 1.f);
+						}
+						if (small) sum += gp_weights_fixed<true>(s, out, cap2, edge, last - 32 * c);
+						else sum += gp_weights_fixed<false>(s, out, cap2, edge, last - 32 * c);
+						tmem_st32(ts + c * 32, out);
+					}
+					tmem_st_wait();
+				}
+				tc_fence_before();
+				mbar_arrive(bar_p + 8 * i);
+				continue;
+			}
 			float mx = -INFINITY, big = 0.f;
 			if (ok) {
 				float s[2][32];
@@ -437,11 +537,10 @@ int gqa_prefill_launch(const GqaArgs &p, int start, cudaStream_t stream) {
 	uint32_t cols = 32;
 	while (cols < (uint32_t)(maps * (GP_T + p.vdim))) cols *= 2;
 	const dim3 grid(p.heads * (p.maps / maps) * ((t + GP_T - 1) / GP_T)), block(maps * (GP_MAP_THREADS + 32) + 32);
-	if (maps == 2)
-		return p.cap > 0.f ? dn_launch(gqa_prefill_kernel<2, true>, grid, block, pl.smem, stream, tmq, tmk, tmv, p, t, start, pl, cols)
-						   : dn_launch(gqa_prefill_kernel<2, false>, grid, block, pl.smem, stream, tmq, tmk, tmv, p, t, start, pl, cols);
-	return p.cap > 0.f ? dn_launch(gqa_prefill_kernel<1, true>, grid, block, pl.smem, stream, tmq, tmk, tmv, p, t, start, pl, cols)
-					   : dn_launch(gqa_prefill_kernel<1, false>, grid, block, pl.smem, stream, tmq, tmk, tmv, p, t, start, pl, cols);
+	const int mode = p.cap <= 0.f ? MODE_PLAIN : p.cap * GQ_LOG2E <= 100.f ? MODE_FIXED : MODE_CAP;
+	auto go = [&](auto kernel) { return dn_launch(kernel, grid, block, pl.smem, stream, tmq, tmk, tmv, p, t, start, pl, cols); };
+	if (maps == 2) return mode == MODE_PLAIN ? go(gqa_prefill_kernel<2, MODE_PLAIN>) : mode == MODE_CAP ? go(gqa_prefill_kernel<2, MODE_CAP>) : go(gqa_prefill_kernel<2, MODE_FIXED>);
+	return mode == MODE_PLAIN ? go(gqa_prefill_kernel<1, MODE_PLAIN>) : mode == MODE_CAP ? go(gqa_prefill_kernel<1, MODE_CAP>) : go(gqa_prefill_kernel<1, MODE_FIXED>);
 }
 
 }   // namespace gptq

@@ -13,6 +13,13 @@ namespace gptq {
 
 namespace {
 
+// 2^x; underflow to zero is what a decay wants
+__device__ __forceinline__ float ex2f_fast(float x) {
+	float r;
+	asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+	return r;
+}
+
 constexpr int SC_L = SS_CHUNK;                    // tokens per chunk
 constexpr int SC_P = 64;                          // value entries per CTA
 constexpr int SC_PAD = 8;                         // bf16 entries behind a staged row, against bank conflicts
@@ -61,24 +68,32 @@ __device__ __forceinline__ void chunk_decays(const SsmArgs &p, const Chunk &k, i
 	}
 }
 
-// rows of `cols` bf16 entries (zero beyond `n` rows and `cols` columns, up to `width`) into shared memory
+// rows of `cols` bf16 entries (zero beyond `n` rows and `cols` columns, up to `width`) into shared memory; aligned rows arrive
+// asynchronously (cp_async_wait)
 __device__ __forceinline__ void stage_rows(bf16 *dst, int ld, const bf16 *src, size_t src_ld, int rows, int n, int cols, int width, bool vec) {
-	const int units = width >> 3;
-	for (int i = threadIdx.x; i < rows * units; i += DN_THREADS) {
-		const int r = i / units, c = (i - r * units) * 8;
-		uint4 v = make_uint4(0u, 0u, 0u, 0u);
-		if (r < n) {
-			const bf16 *s = src + (size_t)r * src_ld + c;
-			if (vec && c + 8 <= cols) {
-				v = __ldcg(reinterpret_cast<const uint4 *>(s));
-			} else {
+	const int units = width >> 3, step_r = DN_THREADS / units, step_c = DN_THREADS - step_r * units;
+	int r = threadIdx.x / units, c = threadIdx.x - r * units;
+#pragma unroll 1
+	for (; r < rows; r += step_r) {
+		bf16 *d = dst + (size_t)r * ld + 8 * c;
+		const bf16 *s = src + (size_t)r * src_ld + 8 * c;
+		if (vec && r < n && 8 * c + 8 <= cols) {
+			cp_async16(d, s);
+		} else {
+			uint4 v = make_uint4(0u, 0u, 0u, 0u);
+			if (r < n) {
 				unsigned short e[8];
 #pragma unroll
-				for (int j = 0; j < 8; ++j) e[j] = c + j < cols ? __ldcg(reinterpret_cast<const unsigned short *>(s) + j) : (unsigned short)0;
+				for (int j = 0; j < 8; ++j) e[j] = 8 * c + j < cols ? __ldcg(reinterpret_cast<const unsigned short *>(s) + j) : (unsigned short)0;
 				v = make_uint4(e[0] | (uint32_t)e[1] << 16, e[2] | (uint32_t)e[3] << 16, e[4] | (uint32_t)e[5] << 16, e[6] | (uint32_t)e[7] << 16);
 			}
+			*reinterpret_cast<uint4 *>(d) = v;
 		}
-		*reinterpret_cast<uint4 *>(dst + (size_t)r * ld + c) = v;
+		c += step_c;
+		if (c >= units) {
+			c -= units;
+			++r;
+		}
 	}
 }
 __device__ __forceinline__ void split2(float a, float b, uint32_t &hi, uint32_t &lo) {
@@ -107,23 +122,25 @@ __global__ void __launch_bounds__(DN_THREADS, 2) ssm_chunk_state_kernel(const Ss
 	pdl_wait();
 	pdl_trigger();
 	const bf16 *u = reinterpret_cast<const bf16 *>(p.u) + ((size_t)k.seq * p.rows_per_seq + k.t0) * p.conv_ld;
-	if (warp == 0) chunk_decays(p, k, lane, s_dt, s_sum);
-	stage_rows(sb, ldb, u + k.inner + k.g * p.state, p.conv_ld, SC_L, k.nt, p.state, nw, vec);
 	stage_rows(sxh, LDX, u + k.head * p.vdim + k.p0, p.conv_ld, SC_L, k.nt, k.np, SC_P, vec);
+	stage_rows(sb, ldb, u + k.inner + k.g * p.state, p.conv_ld, SC_L, k.nt, p.state, nw, vec);
+	cp_async_commit();
+	if (warp == 0) chunk_decays(p, k, lane, s_dt, s_sum);
+	cp_async_wait<0>();
 	__syncthreads();
 	const float end = s_sum[SC_L - 1];
 	for (int i = tid; i < SC_L * SC_P / 2; i += DN_THREADS) {          // inputs times decay to the chunk's end and step size
 		const int t = i / (SC_P / 2), c = (i - t * (SC_P / 2)) * 2;
 		uint32_t *h = reinterpret_cast<uint32_t *>(sxh + t * LDX + c);
 		const uint32_t v = *h;
-		const float f = exp2f(end - s_sum[t]) * s_dt[t];
+		const float f = ex2f_fast(end - s_sum[t]) * s_dt[t];
 		uint32_t hi, lo;
 		split2(__uint_as_float(v << 16) * f, __uint_as_float(v & 0xFFFF0000u) * f, hi, lo);
 		*h = hi;
 		*reinterpret_cast<uint32_t *>(sxl + t * LDX + c) = lo;
 	}
 	__syncthreads();
-	if (tid == 0 && k.p0 == 0) p.chunk_decay[((size_t)k.seq * chunks + k.c) * p.heads + k.head] = exp2f(end);
+	if (tid == 0 && k.p0 == 0) p.chunk_decay[((size_t)k.seq * chunks + k.c) * p.heads + k.head] = ex2f_fast(end);
 	// warp: 16 value entries, half of the state entries in passes of 32
 	const int pr = (warp & 3) * 16, hw = sc_round(nw / 2, 16), n_lo = (warp >> 2) * hw, n_hi = min(n_lo + hw, nw);
 	if (pr >= k.np) return;
@@ -207,19 +224,9 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 	pdl_trigger();
 	const size_t row0 = (size_t)k.seq * p.rows_per_seq + k.t0;
 	const bf16 *u = reinterpret_cast<const bf16 *>(p.u) + row0 * p.conv_ld, *raw = reinterpret_cast<const bf16 *>(p.raw) + row0 * p.raw_ld;
-	if (warp == 0) chunk_decays(p, k, lane, s_dt, s_sum);
 	stage_rows(sb, ldb, u + k.inner + k.g * p.state, p.conv_ld, SC_L, k.nt, p.state, nw, vec);
 	stage_rows(sx, LDX, u + k.head * p.vdim + k.p0, p.conv_ld, SC_L, k.nt, k.np, SC_P, vec);
-	const float *prev = p.chunk_s + (((size_t)k.seq * chunks + k.c) * p.heads + k.head) * p.vdim * p.state + (size_t)k.p0 * p.state;
-	for (int i = tid; i < pw * (nw / 2); i += DN_THREADS) {            // state in front of the chunk, in two parts
-		const int r = i / (nw / 2), n = (i - r * (nw / 2)) * 2;
-		const float a = r < k.np && n < p.state ? __ldcg(prev + (size_t)r * p.state + n) : 0.f;
-		const float b = r < k.np && n + 1 < p.state ? __ldcg(prev + (size_t)r * p.state + n + 1) : 0.f;
-		uint32_t hi, lo;
-		split2(a, b, hi, lo);
-		*reinterpret_cast<uint32_t *>(ssh + r * ldb + n) = hi;
-		*reinterpret_cast<uint32_t *>(ssl + r * ldb + n) = lo;
-	}
+	cp_async_commit();
 	// C of this warp's 16 tokens, as A fragments
 	const int r0 = warp * 16;
 	uint32_t cf[NK][4];
@@ -236,6 +243,39 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 				else cf[s][e] = (n < p.state ? (uint32_t)__ldcg(src) : 0u) | (n + 1 < p.state ? (uint32_t)__ldcg(src + 1) << 16 : 0u);
 			}
 		}
+	if (warp == 0) chunk_decays(p, k, lane, s_dt, s_sum);
+	// state in front of the chunk, in two parts; eight requests of a thread at a time
+	const float *prev = p.chunk_s + (((size_t)k.seq * chunks + k.c) * p.heads + k.head) * p.vdim * p.state + (size_t)k.p0 * p.state;
+	auto put = [&](int r, int n, float a, float b) {
+		uint32_t hi, lo;
+		split2(a, b, hi, lo);
+		*reinterpret_cast<uint32_t *>(ssh + r * ldb + n) = hi;
+		*reinterpret_cast<uint32_t *>(ssl + r * ldb + n) = lo;
+	};
+	if (p.state % 16 == 0) {                          // rows without padding, consecutive in memory
+		const int quads = p.state >> 2, all = k.np * quads;
+		for (int i0 = tid; i0 < all; i0 += 8 * DN_THREADS) {
+			float4 v[8];
+#pragma unroll
+			for (int j = 0; j < 8; ++j)
+				if (i0 + j * DN_THREADS < all) v[j] = __ldcg(reinterpret_cast<const float4 *>(prev) + i0 + j * DN_THREADS);
+#pragma unroll
+			for (int j = 0; j < 8; ++j) {
+				const int i = i0 + j * DN_THREADS, r = i / quads, n = (i - r * quads) * 4;
+				if (i < all) {
+					put(r, n, v[j].x, v[j].y);
+					put(r, n + 2, v[j].z, v[j].w);
+				}
+			}
+		}
+		for (int i = tid; i < (pw - k.np) * (nw / 2); i += DN_THREADS) put(k.np + i / (nw / 2), i % (nw / 2) * 2, 0.f, 0.f);
+	} else {
+		for (int i = tid; i < pw * (nw / 2); i += DN_THREADS) {
+			const int r = i / (nw / 2), n = (i - r * (nw / 2)) * 2;
+			put(r, n, r < k.np && n < p.state ? __ldcg(prev + (size_t)r * p.state + n) : 0.f, r < k.np && n + 1 < p.state ? __ldcg(prev + (size_t)r * p.state + n + 1) : 0.f);
+		}
+	}
+	cp_async_wait<0>();
 	__syncthreads();
 	float acc[SC_P / 8][4];
 #pragma unroll
@@ -260,7 +300,7 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 				}
 			}
 		}
-		const float e0 = exp2f(si0), e1 = exp2f(si1);
+		const float e0 = ex2f_fast(si0), e1 = ex2f_fast(si1);
 #pragma unroll
 		for (int q = 0; q < SC_P / 8; ++q) {
 			acc[q][0] *= e0;
@@ -287,7 +327,7 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 #pragma unroll
 				for (int e = 0; e < 4; ++e) {
 					const int j = j0 + 8 * h + 2 * tig + (e & 1), i = r0 + gid + 8 * (e >> 1);
-					gm[h][e] = j <= i ? gm[h][e] * exp2f(((e >> 1) ? si1 : si0) - s_sum[j]) * s_dt[j] : 0.f;
+					gm[h][e] = j <= i ? gm[h][e] * ex2f_fast(((e >> 1) ? si1 : si0) - s_sum[j]) * s_dt[j] : 0.f;
 				}
 			uint32_t ah[4], al[4];               // accumulator layout = A fragment layout, two 8-column tiles side by side
 			split2(gm[0][0], gm[0][1], ah[0], al[0]);
@@ -319,11 +359,11 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 					float *o = p.out + (row0 + t) * p.out_ld + col;
 					if (vec) {                       // even columns: both entries are there
 						const uint32_t xv = *reinterpret_cast<const uint32_t *>(x), zv = __ldcg(reinterpret_cast<const uint32_t *>(z));
-						*reinterpret_cast<float2 *>(o) = make_float2(fmaf(d, __uint_as_float(xv << 16), acc[q][2 * h]) * silu_exact(__uint_as_float(zv << 16)),
-																   fmaf(d, __uint_as_float(xv & 0xFFFF0000u), acc[q][2 * h + 1]) * silu_exact(__uint_as_float(zv & 0xFFFF0000u)));
+						*reinterpret_cast<float2 *>(o) = make_float2(fmaf(d, __uint_as_float(xv << 16), acc[q][2 * h]) * silu_fast(__uint_as_float(zv << 16)),
+																   fmaf(d, __uint_as_float(xv & 0xFFFF0000u), acc[q][2 * h + 1]) * silu_fast(__uint_as_float(zv & 0xFFFF0000u)));
 					} else {
-						o[0] = fmaf(d, __bfloat162float(x[0]), acc[q][2 * h]) * silu_exact(Elem<bf16>::ldcg(z));
-						if (c + 1 < k.np) o[1] = fmaf(d, __bfloat162float(x[1]), acc[q][2 * h + 1]) * silu_exact(Elem<bf16>::ldcg(z + 1));
+						o[0] = fmaf(d, __bfloat162float(x[0]), acc[q][2 * h]) * silu_fast(Elem<bf16>::ldcg(z));
+						if (c + 1 < k.np) o[1] = fmaf(d, __bfloat162float(x[1]), acc[q][2 * h + 1]) * silu_fast(Elem<bf16>::ldcg(z + 1));
 					}
 				}
 			}

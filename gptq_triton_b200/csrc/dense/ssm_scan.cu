@@ -191,7 +191,7 @@ __global__ void __launch_bounds__(DN_THREADS) ssm_conv_kernel(const SsmArgs p, i
 				v.x = fmaf(w[k].x, in[k].x, v.x);
 				v.y = fmaf(w[k].y, in[k].y, v.y);
 			}
-			if (t + j < t1) store2(u + (size_t)(t + j) * p.conv_ld, make_float2(silu_exact(v.x), silu_exact(v.y)));
+			if (t + j < t1) store2(u + (size_t)(t + j) * p.conv_ld, sizeof(T) == 2 ? make_float2(silu_fast(v.x), silu_fast(v.y)) : make_float2(silu_exact(v.x), silu_exact(v.y)));
 		}
 	}
 }

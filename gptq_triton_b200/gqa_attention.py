@@ -57,6 +57,10 @@ class GroupedAttention(nn.Module):
 		self.register_buffer('w_o', pad_to(o.reshape(width, H, V), w, H, self.V).reshape(w, H * self.V).contiguous())
 		self.register_buffer('q_norm', None if q_norm is None else pad_to(q_norm.float(), self.D))
 		self.register_buffer('k_norm', None if k_norm is None else pad_to(k_norm.float(), self.D))
+		# vectors of unit root mean square have length sqrt(dim): what the norm weights say about the argument of the cap's tanh
+		self.bound = 0.0
+		if spec.softcap and q_norm is not None and k_norm is not None:
+			self.bound = D * float(q_norm.abs().max()) * float(k_norm.abs().max()) * abs(spec.scale) / spec.softcap
 
 	def forward(self, stream: Stream, cache, pos: torch.Tensor, rows_per_seq: int, start: Optional[int], control: torch.Tensor, norm: Optional[Norm] = None):
 		"""stream: M = sequences * rows_per_seq rows at positions pos (int32 [M]); cache: k and v [sequences, max_seq, ...], written
@@ -83,7 +87,7 @@ class GroupedAttention(nn.Module):
 		s, a = self.spec, _dense.Gqa()
 		a.M, a.rows_per_seq, a.heads, a.kv_heads, a.maps = pos.numel(), rows_per_seq, s.heads, s.kv_heads, s.maps
 		a.dim, a.vdim, a.dim_true, a.vdim_true, a.max_seq, a.splits = self.D, self.V, s.dim, s.vdim, cache['k'].shape[1], 1
-		a.scale, a.cap, a.eps, a.lambda_ = s.scale, s.softcap or 0.0, eps, self.lam
+		a.scale, a.cap, a.eps, a.lambda_, a.bound = s.scale, s.softcap or 0.0, eps, self.lam, self.bound
 		a.out_norm, a.out_mul = int(s.maps == 2), 1.0 - s.diff if s.maps == 2 else 1.0
 		a.pos, a.raw, a.raw_ld, a.q_norm, a.k_norm = ptr(pos), ptr(raw), raw.stride(0), ptr(self.q_norm), ptr(self.k_norm)
 		a.k_cache, a.v_cache, a.status = ptr(cache['k']), ptr(cache['v']), _dense.status_ptr(control)

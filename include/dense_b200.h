@@ -143,6 +143,7 @@ typedef struct {
 	int dim_true, vdim_true;           /* what the norms average over */
 	int max_seq, splits;
 	float scale, cap, eps, lambda, out_mul;
+	float bound;                       /* |q . k * scale / cap| is known to be at most this (0: nothing known); used by the prompt kernel */
 	int out_norm;
 	const int32_t *pos;                /* [M] */
 	const void *raw;                   /* [M, raw_ld] fp32 */
