@@ -85,6 +85,7 @@ _SIGNATURES = {
 	'dense_ssm_conv': (c_int, [_P, _I, _P]),
 	'dense_ssm_scan': (c_int, [_P, _P]),
 	'dense_ssm_chunked': (c_int, [_P, _P]),
+	'dense_ssm_chunked_scratch': (c_int, [_P]),
 }
 
 _lib: Optional[ctypes.CDLL] = None

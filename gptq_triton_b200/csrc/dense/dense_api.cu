@@ -226,11 +226,12 @@ int dense_ssm_scan(const dense_ssm_t *a, void *stream) {
 	if (!a || ssm_bad(*a) || !a->u || !a->out || a->out_ld < (int64_t)a->heads * a->vdim) return GPTQ_ERR_INVALID;
 	return ssm_scan_launch(*a, reinterpret_cast<cudaStream_t>(stream));
 }
+int dense_ssm_chunked_scratch(const dense_ssm_t *a) { return a && !ssm_bad(*a) && ssm_tc_ok(*a) ? 0 : 1; }
 int dense_ssm_chunked(const dense_ssm_t *a, void *stream) {
-	if (!a || ssm_bad(*a) || !a->u || !a->out || a->out_ld % 2 || a->out_ld < (int64_t)a->heads * a->vdim || !a->chunk_s || !a->chunk_decay) return GPTQ_ERR_INVALID;
+	if (!a || ssm_bad(*a) || !a->u || !a->out || a->out_ld % 2 || a->out_ld < (int64_t)a->heads * a->vdim || (!ssm_tc_ok(*a) && (!a->chunk_s || !a->chunk_decay))) return GPTQ_ERR_INVALID;
 	if (!aligned16(a->u) || !aligned16(a->raw) || !aligned16(a->out)) return GPTQ_ERR_ALIGN;
 	if ((long long)(a->M / a->rows_per_seq) * ((a->rows_per_seq + SS_CHUNK - 1) / SS_CHUNK) > 65535) return GPTQ_ERR_UNSUPPORTED;
-	return ssm_chunk_launch(*a, reinterpret_cast<cudaStream_t>(stream));
+	return ssm_tc_ok(*a) ? ssm_tc_launch(*a, reinterpret_cast<cudaStream_t>(stream)) : ssm_chunk_launch(*a, reinterpret_cast<cudaStream_t>(stream));
 }
 
 }   // extern "C"

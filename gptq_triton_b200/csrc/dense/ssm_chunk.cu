@@ -1,5 +1,5 @@
-// The recurrence of ssm_scan.cu for bf16 prompts, in chunks of 128 tokens: what a chunk adds is a few small matrix products, only
-// the state goes from chunk to chunk.  With s_i the sum of a * dt over the chunk's tokens up to i (fp32, in base 2),
+// The recurrence of ssm_scan.cu for bf16 prompts of any sizes (ssm_tc.cu takes those that fit its tiles), in chunks of 128 tokens: what a chunk adds is a few small matrix products, only
+// the state goes from chunk to chunk.  With s_i the sum of a * dt over the chunk's tokens up to i (base 2),
 //   ssm_chunk_state   S_c = sum_j 2^(s_last - s_j) dt_j x_j B_j^T                          per chunk and head, all at once
 //   ssm_chunk_pass    state in front of every chunk: S <- 2^s_last S + S_c                 over the chunks, all entries at once
 //   ssm_chunk_out     y_i = 2^s_i S C_i + sum_{j <= i} (C_i . B_j) 2^(s_i - s_j) dt_j x_j + d x_i, times silu(z_i)
@@ -42,29 +42,38 @@ __device__ __forceinline__ Chunk chunk_of(const SsmArgs &p, int chunks) {
 	return k;
 }
 
-// step sizes of the chunk and prefix sums of a * dt * log2(e); tokens behind the end have step size 0.  One warp.
-__device__ __forceinline__ void chunk_decays(const SsmArgs &p, const Chunk &k, int lane, float *s_dt, float *s_sum) {
+// Step sizes of the chunk and prefix sums of a * dt * log2(e), formed in fp64 and kept in two parts (differences must stay exact behind
+// tokens that decay by orders of magnitude); tokens behind the end have step size 0.  One warp.
+struct Decays {
+	float dt[SC_L], hi[SC_L], lo[SC_L];
+	__device__ float between(int i, int j) const { return (hi[i] - hi[j]) + (lo[i] - lo[j]); }
+};
+__device__ __forceinline__ void chunk_decays(const SsmArgs &p, const Chunk &k, int lane, Decays &out) {
 	const float bias = __ldg(p.dt_bias + k.head), a = __ldg(p.a + k.head) * 1.4426950408889634f;
 	constexpr int PER = SC_L / 32;
-	float dt[PER], run = 0.f;
+	float dt[PER];
+	double run = 0.0;
 #pragma unroll
 	for (int i = 0; i < PER; ++i) {
 		const int t = lane * PER + i;
 		dt[i] = t < k.nt ? ssm_softplus(__ldcg(p.dt + ((size_t)k.seq * p.rows_per_seq + k.t0 + t) * p.dt_ld + k.head) + bias) : 0.f;
-		run += a * dt[i];
+		run += (double)(a * dt[i]);
 	}
-	float before = run;
+	double before = run;
 #pragma unroll
 	for (int d = 1; d < 32; d <<= 1) {
-		const float v = __shfl_up_sync(0xffffffffu, before, d);
+		const double v = __shfl_up_sync(0xffffffffu, before, d);
 		if (lane >= d) before += v;
 	}
 	before -= run;
 #pragma unroll
 	for (int i = 0; i < PER; ++i) {
-		before += a * dt[i];
-		s_dt[lane * PER + i] = dt[i];
-		s_sum[lane * PER + i] = before;
+		before += (double)(a * dt[i]);
+		const int t = lane * PER + i;
+		const float hi = (float)before;
+		out.dt[t] = dt[i];
+		out.hi[t] = hi;
+		out.lo[t] = (float)(before - (double)hi);
 	}
 }
 
@@ -112,7 +121,7 @@ __host__ __device__ __forceinline__ int sc_round(int n, int to) { return (n + to
 // ---- state that a chunk adds: [value entries x tokens] times [tokens x state entries] ---------------------------------------------
 __global__ void __launch_bounds__(DN_THREADS, 2) ssm_chunk_state_kernel(const SsmArgs p, int chunks) {
 	extern __shared__ __align__(16) unsigned char cs_smem[];
-	__shared__ float s_dt[SC_L], s_sum[SC_L];
+	__shared__ Decays s_d;
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
 	const Chunk k = chunk_of(p, chunks);
 	const int nw = sc_round(p.state, 16), ldb = nw + SC_PAD;
@@ -125,22 +134,21 @@ __global__ void __launch_bounds__(DN_THREADS, 2) ssm_chunk_state_kernel(const Ss
 	stage_rows(sxh, LDX, u + k.head * p.vdim + k.p0, p.conv_ld, SC_L, k.nt, k.np, SC_P, vec);
 	stage_rows(sb, ldb, u + k.inner + k.g * p.state, p.conv_ld, SC_L, k.nt, p.state, nw, vec);
 	cp_async_commit();
-	if (warp == 0) chunk_decays(p, k, lane, s_dt, s_sum);
+	if (warp == 0) chunk_decays(p, k, lane, s_d);
 	cp_async_wait<0>();
 	__syncthreads();
-	const float end = s_sum[SC_L - 1];
 	for (int i = tid; i < SC_L * SC_P / 2; i += DN_THREADS) {          // inputs times decay to the chunk's end and step size
 		const int t = i / (SC_P / 2), c = (i - t * (SC_P / 2)) * 2;
 		uint32_t *h = reinterpret_cast<uint32_t *>(sxh + t * LDX + c);
 		const uint32_t v = *h;
-		const float f = ex2f_fast(end - s_sum[t]) * s_dt[t];
+		const float f = ex2f_fast(s_d.between(SC_L - 1, t)) * s_d.dt[t];
 		uint32_t hi, lo;
 		split2(__uint_as_float(v << 16) * f, __uint_as_float(v & 0xFFFF0000u) * f, hi, lo);
 		*h = hi;
 		*reinterpret_cast<uint32_t *>(sxl + t * LDX + c) = lo;
 	}
 	__syncthreads();
-	if (tid == 0 && k.p0 == 0) p.chunk_decay[((size_t)k.seq * chunks + k.c) * p.heads + k.head] = ex2f_fast(end);
+	if (tid == 0 && k.p0 == 0) p.chunk_decay[((size_t)k.seq * chunks + k.c) * p.heads + k.head] = ex2f_fast(s_d.hi[SC_L - 1] + s_d.lo[SC_L - 1]);
 	// warp: 16 value entries, half of the state entries in passes of 32
 	const int pr = (warp & 3) * 16, hw = sc_round(nw / 2, 16), n_lo = (warp >> 2) * hw, n_hi = min(n_lo + hw, nw);
 	if (pr >= k.np) return;
@@ -213,7 +221,7 @@ __global__ void __launch_bounds__(DN_THREADS) ssm_chunk_pass_kernel(const SsmArg
 template <int NK>                        // 16-entry steps of the state: state <= 16 * NK
 __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kernel(const SsmArgs p, int chunks) {
 	extern __shared__ __align__(16) unsigned char co_smem[];
-	__shared__ float s_dt[SC_L], s_sum[SC_L];
+	__shared__ Decays s_d;
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
 	const Chunk k = chunk_of(p, chunks);
 	const int nw = sc_round(p.state, 16), nk = nw >> 4, ldb = nw + SC_PAD, pw = sc_round(k.np, 16);
@@ -243,7 +251,7 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 				else cf[s][e] = (n < p.state ? (uint32_t)__ldcg(src) : 0u) | (n + 1 < p.state ? (uint32_t)__ldcg(src + 1) << 16 : 0u);
 			}
 		}
-	if (warp == 0) chunk_decays(p, k, lane, s_dt, s_sum);
+	if (warp == 0) chunk_decays(p, k, lane, s_d);
 	// state in front of the chunk, in two parts; eight requests of a thread at a time
 	const float *prev = p.chunk_s + (((size_t)k.seq * chunks + k.c) * p.heads + k.head) * p.vdim * p.state + (size_t)k.p0 * p.state;
 	auto put = [&](int r, int n, float a, float b) {
@@ -280,7 +288,7 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 	float acc[SC_P / 8][4];
 #pragma unroll
 	for (int q = 0; q < SC_P / 8; ++q) acc[q][0] = acc[q][1] = acc[q][2] = acc[q][3] = 0.f;
-	const float si0 = s_sum[r0 + gid], si1 = s_sum[r0 + gid + 8];
+	const int i0 = r0 + gid, i1 = i0 + 8;
 	if (r0 < k.nt) {
 		// ---- from the state: rows of S are value entries, columns state entries ----
 		const uint32_t s_off = (uint32_t)(((lane >> 4) * 8 + (lane & 7)) * ldb + ((lane >> 3) & 1) * 8) * 2;      // two 8-row groups x two 8-column halves
@@ -300,7 +308,7 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 				}
 			}
 		}
-		const float e0 = ex2f_fast(si0), e1 = ex2f_fast(si1);
+		const float e0 = ex2f_fast(s_d.hi[i0] + s_d.lo[i0]), e1 = ex2f_fast(s_d.hi[i1] + s_d.lo[i1]);
 #pragma unroll
 		for (int q = 0; q < SC_P / 8; ++q) {
 			acc[q][0] *= e0;
@@ -327,7 +335,7 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 #pragma unroll
 				for (int e = 0; e < 4; ++e) {
 					const int j = j0 + 8 * h + 2 * tig + (e & 1), i = r0 + gid + 8 * (e >> 1);
-					gm[h][e] = j <= i ? gm[h][e] * ex2f_fast(((e >> 1) ? si1 : si0) - s_sum[j]) * s_dt[j] : 0.f;
+					gm[h][e] = j <= i ? gm[h][e] * ex2f_fast(s_d.between(i, j)) * s_d.dt[j] : 0.f;
 				}
 			uint32_t ah[4], al[4];               // accumulator layout = A fragment layout, two 8-column tiles side by side
 			split2(gm[0][0], gm[0][1], ah[0], al[0]);

@@ -1,0 +1,412 @@
+// The chunked recurrence (see ssm_chunk.cu for the arithmetic) on the 5th-generation tensor cores, one kernel per prompt portion: a CTA
+// owns up to 64 value entries of one head and walks the chunks of 128 tokens, the state stays in tensor memory from the first to
+// the last.  Per chunk, with s_i the prefix sums of a * dt (base 2), w_j = log2(dt_j) - s_j, all fp32:
+//   G  = C B^T                                  128 x 128, in tensor memory
+//   M  = G_ij 2^(s_i + w_j), j <= i             written over G as bf16 high parts and remainders
+//   Ya = M X,  Yi = C S                         S as two bf16 parts in shared memory
+//   y  = 2^s_i Yi + Ya + d x, times silu(z)
+//   S <- 2^s_last S + sum_j B_j (2^(s_last - s_j) dt_j x_j)^T     accumulates in tensor memory; the scaled inputs as two bf16 parts
+// Differences of prefix sums must stay exact behind tokens that decay by orders of magnitude, so the sums are formed in fp64 and kept as
+// an fp32 value hi and a remainder lo; log2(dt_j) joins the remainder of the second one.
+//   warps 0-7   scale the inputs, split and decay S, form M, write y        warp 8   TMA: C, B, X tiles, two stages
+//   warp 10     step sizes and prefix sums of the next chunk                 warp 9   MMA
+// B and C are operands in both roles (rows of tokens as rows, and as the summed dimension); shared memory holds them once, in the
+// 128-byte-swizzled layout that serves both.  Every wait is bounded.
+#include <algorithm>
+
+#include "prefill_common.cuh"
+#include "ssm.cuh"
+
+namespace gptq {
+
+namespace {
+
+constexpr int ST_L = SS_CHUNK, ST_P = 64;
+constexpr int ST_CHUNK = ST_L * 128;                    // bytes of a 128 x 64 bf16 tile
+constexpr int ST_WORK = 256, ST_THREADS = ST_WORK + 96;
+constexpr uint32_t T_G = 0, T_YI = 256, T_YA = 320, T_S = 384;      // tensor memory columns: two G / M buffers, Yi, Ya, S
+
+struct StPlan {
+	int nc;                                             // 64-column tiles of C
+	uint32_t stage;
+	size_t smem;
+};
+__host__ __device__ inline StPlan st_plan(int state) {
+	StPlan pl;
+	pl.nc = (state + 63) / 64;
+	pl.stage = (uint32_t)(pl.nc + 2 + 1) * ST_CHUNK;      // C, B (always two tiles: 128 rows of S), X
+	pl.smem = 2 * (size_t)pl.stage + 4 * ST_CHUNK + 2 * ST_L * (2 * sizeof(float) + sizeof(bf16)) + 128;
+	return pl;
+}
+
+// operand whose other dimension is contiguous: 64-column tiles ST_CHUNK apart, groups of 8 rows of 128 bytes
+__device__ __forceinline__ uint64_t desc_rows(uint32_t addr) {
+	uint64_t d = 0;
+	d |= (uint64_t)((addr & 0x3FFFFu) >> 4);
+	d |= (uint64_t)(ST_CHUNK >> 4) << 16;
+	d |= (uint64_t)(1024 >> 4) << 32;
+	d |= (uint64_t)1 << 46;
+	d |= (uint64_t)2 << 61;
+	return d;
+}
+__device__ __forceinline__ void st_split(float a, float b, uint32_t &hi, uint32_t &lo) {
+	hi = pack_bf16(a, b);
+	lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xFFFF0000u));
+}
+
+__global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_constant__ CUtensorMap tmu, const SsmArgs p, int seq) {
+	extern __shared__ __align__(1024) unsigned char st_smem[];
+	const StPlan pl = st_plan(p.state);
+	const uint32_t base = smem_u32(st_smem), sxs = base + 2 * pl.stage, sst = sxs + 2 * ST_CHUNK;      // scaled inputs, S: high parts, remainders
+	// prefix sums: hi, log2(dt) - lo, lo (bf16 is enough for it); two stages each
+	float *s_hi = reinterpret_cast<float *>(st_smem + 2 * (size_t)pl.stage + 4 * ST_CHUNK), *s_w = s_hi + 2 * ST_L;
+	bf16 *s_lo = reinterpret_cast<bf16 *>(s_w + 2 * ST_L);
+	uint64_t *bars = reinterpret_cast<uint64_t *>(s_lo + 2 * ST_L);
+	const uint32_t b0 = smem_u32(bars);
+	const uint32_t bar_full = b0, bar_empty = b0 + 16, bar_g = b0 + 32, bar_r = b0 + 48, bar_m = b0 + 56, bar_y = b0 + 64, bar_u = b0 + 72, bar_end = b0 + 80;
+	uint32_t *s_tmem = reinterpret_cast<uint32_t *>(bars + 11);
+	volatile int *s_abort = reinterpret_cast<volatile int *>(s_tmem + 1);
+	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+	const int slices = (p.vdim + ST_P - 1) / ST_P, head = blockIdx.x / slices, p0 = (blockIdx.x - head * slices) * ST_P;
+	const int np = min(ST_P, p.vdim - p0), g = head / (p.heads / p.groups), inner = p.heads * p.vdim;
+	const int T = p.rows_per_seq, n = (T + ST_L - 1) / ST_L;
+	if (base & 1023u) {                                 // (dynamic shared memory starts on a 1 KB boundary when there is no other)
+		if (tid == 0) atomicExch(p.status, 2);
+		return;
+	}
+	if (tid == 0) {
+		for (int s = 0; s < 2; ++s) {
+			mbar_init(bar_full + 8 * s, 1 + 32);
+			mbar_init(bar_empty + 8 * s, ST_WORK + 1);
+			mbar_init(bar_g + 8 * s, 1);
+		}
+		mbar_init(bar_r, ST_WORK);
+		mbar_init(bar_m, ST_WORK);
+		mbar_init(bar_y, 1);
+		mbar_init(bar_u, 1);
+		mbar_init(bar_end, 1);
+		*s_abort = 0;
+		fence_mbar_init();
+	}
+	if (warp == 9) {
+		tmem_alloc(smem_u32(s_tmem), 512);
+		tmem_relinquish();
+	}
+	tc_fence_before();
+	__syncthreads();
+	tc_fence_after();
+	const uint32_t tmem = *s_tmem;
+	auto fail = [&]() {
+		*s_abort = 1;
+		atomicExch(p.status, 3);
+	};
+	auto wait_one = [&](uint32_t bar, int k) {            // one thread
+		if (wait_fast(bar, k & 1, s_abort)) return true;
+		fail();
+		return false;
+	};
+	auto wait_warp = [&](uint32_t bar, int k) {           // a whole warp, one answer
+		const bool got = wait_fast(bar, k & 1, s_abort);
+		if (__all_sync(0xffffffffu, got)) return true;
+		fail();
+		return false;
+	};
+	pdl_wait();
+	pdl_trigger();
+	const int start = __ldcg(p.pos + (size_t)seq * T);
+
+	if (warp == 8) {
+		if (lane == 0) {
+			int done = 0;
+			for (int c = 0; c < n; ++c) {
+				const int s = c & 1;
+				if (*s_abort || !wait_one(bar_empty + 8 * s, (c >> 1) + 1)) break;
+				const uint32_t dst = base + s * pl.stage;
+				mbar_arrive_expect_tx(bar_full + 8 * s, pl.stage);
+				for (int i = 0; i < pl.nc; ++i) tma_load_2d(dst + i * ST_CHUNK, &tmu, inner + (p.groups + g) * p.state + 64 * i, c * ST_L, bar_full + 8 * s);
+				for (int i = 0; i < 2; ++i) tma_load_2d(dst + (pl.nc + i) * ST_CHUNK, &tmu, inner + g * p.state + 64 * i, c * ST_L, bar_full + 8 * s);
+				tma_load_2d(dst + (pl.nc + 2) * ST_CHUNK, &tmu, head * p.vdim + p0, c * ST_L, bar_full + 8 * s);
+				done = c + 1;
+			}
+			// no copy may be in flight when the CTA ends
+			for (int c = max(0, done - 2); c < done; ++c) mbar_wait_bounded(bar_full + 8 * (c & 1), (c >> 1) & 1, ATTN_SPIN);
+		}
+		__syncwarp();
+	} else if (warp == 10) {
+		const float bias = __ldg(p.dt_bias + head), a = __ldg(p.a + head) * 1.4426950408889634f;
+		constexpr int PER = ST_L / 32;
+		const float *src = p.dt + (size_t)seq * T * p.dt_ld + head;
+		for (int c = 0; c < n; ++c) {
+			float dt[PER];
+			double run = 0.0;
+#pragma unroll
+			for (int i = 0; i < PER; ++i) {
+				const int t = c * ST_L + lane * PER + i;
+				dt[i] = t < T ? __ldcg(src + (size_t)t * p.dt_ld) : 0.f;
+			}
+#pragma unroll
+			for (int i = 0; i < PER; ++i) {
+				dt[i] = c * ST_L + lane * PER + i < T ? ssm_softplus(dt[i] + bias) : 0.f;      // behind the end: no input, no decay
+				run += (double)(a * dt[i]);
+			}
+			double before = run;
+#pragma unroll
+			for (int d = 1; d < 32; d <<= 1) {
+				const double v = __shfl_up_sync(0xffffffffu, before, d);
+				if (lane >= d) before += v;
+			}
+			before -= run;
+			if (!wait_warp(bar_empty + 8 * (c & 1), (c >> 1) + 1)) break;
+#pragma unroll
+			for (int i = 0; i < PER; ++i) {
+				before += (double)(a * dt[i]);
+				const int at = (c & 1) * ST_L + lane * PER + i;
+				const float hi = (float)before;
+				const bf16 lo = __float2bfloat16_rn((float)(before - (double)hi));
+				s_hi[at] = hi;
+				s_lo[at] = lo;
+				s_w[at] = log2f(dt[i]) - __bfloat162float(lo);          // dt = 0: weight 2^-inf = 0
+			}
+			mbar_arrive(bar_full + 8 * (c & 1));
+		}
+	} else if (warp == 9) {
+		if (lane == 0) {
+			const uint32_t fmt = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(ST_L >> 4) << 24);          // D fp32, A/B bf16, M = 128
+			const uint32_t nw = (uint32_t)((np + 15) / 16 * 16), at_n = (nw >> 3) << 17;
+			const uint32_t id_g = fmt | ((uint32_t)(ST_L >> 3) << 17), id_y = fmt | (1u << 16) | at_n, id_u = id_y | (1u << 15);
+			const int steps = p.state >> 4;
+			auto issue_g = [&](int c) {                   // C and B tiles have arrived
+				const uint32_t st = base + (c & 1) * pl.stage;
+				for (int k = 0; k < steps; ++k) {
+					const uint32_t off = (k >> 2) * ST_CHUNK + (k & 3) * 32;
+					umma_f16(tmem + T_G + (c & 1) * ST_L, smem_desc_sw128(st + off), smem_desc_sw128(st + pl.nc * ST_CHUNK + off), id_g, k ? 1u : 0u);
+				}
+				umma_commit(bar_g + 8 * (c & 1));
+			};
+			bool ok = wait_one(bar_full, 0);
+			tc_fence_after();
+			if (ok) issue_g(0);
+			for (int c = 0; c < n && ok; ++c) {
+				const uint32_t st = base + (c & 1) * pl.stage, sx = st + (pl.nc + 2) * ST_CHUNK;
+				if (!(ok = wait_one(bar_r, c))) break;
+				tc_fence_after();
+				for (int part = 0; part < 2; ++part)
+					for (int k = 0; k < steps; ++k)
+						umma_f16(tmem + T_YI, smem_desc_sw128(st + (k >> 2) * ST_CHUNK + (k & 3) * 32), desc_rows(sst + part * ST_CHUNK) + 128 * k, id_y, part | k ? 1u : 0u);
+				for (int part = 0; part < 2; ++part)
+#pragma unroll
+					for (int k = 0; k < ST_L / 16; ++k)
+						umma_f16(tmem + T_S, desc_rows(st + pl.nc * ST_CHUNK) + 128 * k, desc_rows(sxs + part * ST_CHUNK) + 128 * k, id_u, 1u);
+				umma_commit(bar_u);
+				if (c + 1 < n) {
+					if (!(ok = wait_one(bar_full + 8 * ((c + 1) & 1), (c + 1) >> 1))) break;
+					tc_fence_after();
+					issue_g(c + 1);
+				}
+				if (!(ok = wait_one(bar_m, c))) break;
+				tc_fence_after();
+#pragma unroll
+				for (int part = 0; part < 2; ++part)
+#pragma unroll
+					for (int k = 0; k < ST_L / 16; ++k)
+						umma_f16_ts(tmem + T_YA, tmem + T_G + (c & 1) * ST_L + (k >> 1) * 32 + part * 16 + (k & 1) * 8, desc_rows(sx) + 128 * k, id_y, part | k ? 1u : 0u);
+				umma_commit(bar_y);
+				umma_commit(bar_empty + 8 * (c & 1));
+			}
+			umma_commit(bar_end);                         // every MMA has completed before tensor memory goes back
+			mbar_wait_bounded(bar_end, 0, ATTN_SPIN);
+		}
+		__syncwarp();
+	} else {
+		const int q = warp & 3, h = warp >> 2, row = q * 32 + lane;          // token of the chunk, or state entry
+		const uint32_t lanes = (uint32_t)(q * 32) << 16;
+		const bool cols = 32 * h < np;                                       // this half of the value entries exists
+		const float d = __ldg(p.d + head);
+		// ---- state of the sequence into tensor memory: row = state entry, column = value entry ----
+		float *state = p.s + ((size_t)seq * p.heads + head) * p.vdim * p.state + (size_t)p0 * p.state;
+		if (cols) {
+			uint32_t v[32];
+#pragma unroll
+			for (int i = 0; i < 32; ++i) v[i] = start > 0 && row < p.state && 32 * h + i < np ? __float_as_uint(__ldcg(state + (size_t)(32 * h + i) * p.state + row)) : 0u;
+			tmem_st32(tmem + T_S + lanes + 32 * h, v);
+			tmem_st_wait();
+		}
+		const bf16 *zrow = reinterpret_cast<const bf16 *>(p.raw) + (size_t)seq * T * p.raw_ld + p.z_at + head * p.vdim + p0 + 32 * h;
+		float *orow = p.out + (size_t)seq * T * p.out_ld + head * p.vdim + p0 + 32 * h;
+		bool ok = true;
+		for (int c = 0; c < n && ok; ++c) {
+			const int s = c & 1, t = c * ST_L + row;
+			unsigned char *stage = st_smem + (size_t)s * pl.stage, *xt = stage + (size_t)(pl.nc + 2) * ST_CHUNK;
+			const float *hi_j = s_hi + s * ST_L, *w = s_w + s * ST_L;
+			if (!(ok = wait_warp(bar_full + 8 * s, c >> 1))) break;
+			if (c && !(ok = wait_warp(bar_u, c - 1))) break;
+			tc_fence_after();
+			const float end = hi_j[ST_L - 1], end_lo = __bfloat162float(s_lo[s * ST_L + ST_L - 1]);
+			// ---- inputs times step size and decay to the chunk's end: element by element, so the tile's layout does not matter ----
+			{
+				const int trow = tid >> 1;                                  // two threads per token, half a row each
+				const float f = ex2((end - hi_j[trow]) + (end_lo + w[trow]));
+#pragma unroll
+				for (int i = 0; i < 4; ++i) {
+					const uint32_t off = (uint32_t)trow * 128 + (uint32_t)(((tid & 1) * 4 + i + trow) & 7) * 16;      // (rotated against bank conflicts)
+					const uint4 x = *reinterpret_cast<const uint4 *>(xt + off);
+					const uint32_t xs[4] = {x.x, x.y, x.z, x.w};
+					uint32_t hi[4], lo[4];
+#pragma unroll
+					for (int j = 0; j < 4; ++j) st_split(__uint_as_float(xs[j] << 16) * f, __uint_as_float(xs[j] & 0xFFFF0000u) * f, hi[j], lo[j]);
+					unsigned char *dst = st_smem + 2 * (size_t)pl.stage + off;
+					*reinterpret_cast<uint4 *>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+					*reinterpret_cast<uint4 *>(dst + ST_CHUNK) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+				}
+			}
+			// ---- S in two parts for Yi, then decayed ----
+			if (cols) {
+				float v[32];
+				tmem_ld32(tmem + T_S + lanes + 32 * h, v);
+				tmem_ld_wait();
+				tmem_settle(v);
+				unsigned char *dst = st_smem + 2 * (size_t)pl.stage + 2 * ST_CHUNK + row * 128;
+#pragma unroll
+				for (int i = 0; i < 4; ++i) {
+					uint32_t hi[4], lo[4];
+#pragma unroll
+					for (int j = 0; j < 4; ++j) st_split(v[8 * i + 2 * j], v[8 * i + 2 * j + 1], hi[j], lo[j]);
+					const int unit = ((4 * h + i) ^ (row & 7)) * 16;
+					*reinterpret_cast<uint4 *>(dst + unit) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+					*reinterpret_cast<uint4 *>(dst + ST_CHUNK + unit) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+				}
+				const float f = ex2(end + end_lo);
+				uint32_t o[32];
+#pragma unroll
+				for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(v[i] * f);
+				tmem_st32(tmem + T_S + lanes + 32 * h, o);
+				tmem_st_wait();
+			}
+			fence_proxy_async();
+			tc_fence_before();
+			mbar_arrive(bar_r);
+			uint32_t z[16];                                                 // gates of this thread's outputs, requested early
+#pragma unroll
+			for (int i = 0; i < 4; ++i) {
+				uint4 v = make_uint4(0u, 0u, 0u, 0u);
+				if (t < T && 32 * h + 8 * i < np) v = __ldcg(reinterpret_cast<const uint4 *>(zrow + (size_t)t * p.raw_ld) + i);
+				z[4 * i] = v.x;
+				z[4 * i + 1] = v.y;
+				z[4 * i + 2] = v.z;
+				z[4 * i + 3] = v.w;
+			}
+			// ---- M over G: this thread's row, half of the columns ----
+			if (!(ok = wait_warp(bar_g + 8 * s, c >> 1))) break;
+			tc_fence_after();
+			const float si = hi_j[row], si_lo = __bfloat162float(s_lo[s * ST_L + row]);
+#pragma unroll 1
+			for (int b = 0; b < 2; ++b) {
+				const int j0 = 64 * h + 32 * b;
+				const uint32_t at = tmem + T_G + s * ST_L + lanes + j0;
+				uint32_t out[32];
+				if (j0 > q * 32) {                                          // above the diagonal
+#pragma unroll
+					for (int i = 0; i < 32; ++i) out[i] = 0u;
+				} else {
+					float v[32];
+					tmem_ld32(at, v);
+					tmem_ld_wait();
+					tmem_settle(v);
+					const bool edge = j0 == q * 32;
+#pragma unroll
+					for (int i = 0; i < 8; ++i) {
+						const float4 wj = *reinterpret_cast<const float4 *>(w + j0 + 4 * i), hj = *reinterpret_cast<const float4 *>(hi_j + j0 + 4 * i);
+						v[4 * i] *= ex2((si - hj.x) + (si_lo + wj.x));
+						v[4 * i + 1] *= ex2((si - hj.y) + (si_lo + wj.y));
+						v[4 * i + 2] *= ex2((si - hj.z) + (si_lo + wj.z));
+						v[4 * i + 3] *= ex2((si - hj.w) + (si_lo + wj.w));
+					}
+					if (edge) {
+#pragma unroll
+						for (int i = 0; i < 32; ++i) v[i] = i <= lane ? v[i] : 0.f;
+					}
+#pragma unroll
+					for (int i = 0; i < 16; ++i) st_split(v[2 * i], v[2 * i + 1], out[i], out[16 + i]);
+				}
+				tmem_st32(at, out);
+			}
+			tmem_st_wait();
+			tc_fence_before();
+			mbar_arrive(bar_m);
+			// ---- y ----
+			if (!(ok = wait_warp(bar_y, c))) break;
+			tc_fence_after();
+			if (cols) {
+				const float e = ex2(si + si_lo);
+#pragma unroll
+				for (int b = 0; b < 2; ++b) {
+					float yi[16], ya[16];
+					tmem_ld16(tmem + T_YI + lanes + 32 * h + 16 * b, yi);
+					tmem_ld16(tmem + T_YA + lanes + 32 * h + 16 * b, ya);
+					tmem_ld_wait();
+					tmem_settle(yi);
+					tmem_settle(ya);
+					if (t < T && 32 * h + 16 * b < np) {
+#pragma unroll
+						for (int u = 0; u < 2; ++u) {
+							const uint4 x = *reinterpret_cast<const uint4 *>(xt + row * 128 + ((4 * h + 2 * b + u) ^ (row & 7)) * 16);
+							const uint32_t xs[4] = {x.x, x.y, x.z, x.w};
+							float o[8];
+#pragma unroll
+							for (int j = 0; j < 4; ++j) {
+								const int i = 8 * u + 2 * j;
+								const uint32_t zz = z[8 * b + 4 * u + j];
+								o[2 * j] = fmaf(d, __uint_as_float(xs[j] << 16), fmaf(e, yi[i], ya[i])) * silu_fast(__uint_as_float(zz << 16));
+								o[2 * j + 1] = fmaf(d, __uint_as_float(xs[j] & 0xFFFF0000u), fmaf(e, yi[i + 1], ya[i + 1])) * silu_fast(__uint_as_float(zz & 0xFFFF0000u));
+							}
+							Elem<float>::store8(orow + (size_t)t * p.out_ld + 16 * b + 8 * u, o);
+						}
+					}
+				}
+			}
+			tc_fence_before();
+			mbar_arrive(bar_empty + 8 * s);
+		}
+		if (ok && cols && wait_warp(bar_u, n - 1)) {
+			tc_fence_after();
+			float v[32];
+			tmem_ld32(tmem + T_S + lanes + 32 * h, v);
+			tmem_ld_wait();
+			tmem_settle(v);
+#pragma unroll
+			for (int i = 0; i < 32; ++i)
+				if (row < p.state && 32 * h + i < np) state[(size_t)(32 * h + i) * p.state + row] = v[i];
+		}
+		// ---- the convolution's last inputs ----
+		const int last = min(T, p.taps);
+		const bool shared = p0 == 0 && head % (p.heads / p.groups) == 0;
+		const int count = np + (shared ? 2 * p.state : 0);
+		const bf16 *in = reinterpret_cast<const bf16 *>(p.raw) + (size_t)seq * T * p.raw_ld + p.conv_at;
+		float *ring = p.ring + (size_t)seq * p.taps * p.conv_ld;
+		for (int i = tid; i < last * count; i += ST_WORK) {
+			const int tt = T - last + i / count, e = i % count;
+			const int ch = e < np ? head * p.vdim + p0 + e : e < np + p.state ? inner + g * p.state + e - np : inner + (p.groups + g) * p.state + e - np - p.state;
+			ring[(size_t)((start + tt) % p.taps) * p.conv_ld + ch] = Elem<bf16>::ldcg(in + (size_t)tt * p.raw_ld + ch);
+		}
+	}
+	tc_fence_before();
+	__syncthreads();
+	if (warp == 9) tmem_dealloc(tmem, 512);
+}
+
+}   // namespace
+
+bool ssm_tc_ok(const SsmArgs &p) { return p.vdim % 16 == 0 && p.state % 16 == 0 && p.state <= 128 && p.out_ld % 4 == 0; }
+
+int ssm_tc_launch(const SsmArgs &p, cudaStream_t stream) {
+	const int T = p.rows_per_seq, seqs = p.M / T, slices = (p.vdim + ST_P - 1) / ST_P;
+	for (int b = 0; b < seqs; ++b) {
+		alignas(64) CUtensorMap tmu;
+		const bf16 *u = reinterpret_cast<const bf16 *>(p.u) + (size_t)b * T * p.conv_ld;
+		if (int rc = dense_tensor_map(u, T, p.conv_ld, p.conv_ld, ST_L, 64, &tmu)) return rc;
+		if (int rc = dn_launch(ssm_tc_kernel, dim3(p.heads * slices), dim3(ST_THREADS), st_plan(p.state).smem, stream, tmu, p, b)) return rc;
+	}
+	return GPTQ_OK;
+}
+
+}   // namespace gptq

@@ -92,7 +92,8 @@ class StateSpaceMixer(nn.Module):
 			scratch = self.portion_buffers(a, raw.dtype, chunked)      # noqa: F841 (alive until the launches)
 			_dense.check(lib.dense_ssm_conv(ctypes.byref(a), _dense.DTYPE_CODE[raw.dtype], st), 'dense_ssm_conv')
 			if chunked:
-				_dense.check(lib.dense_ssm_chunked(ctypes.byref(a), st), 'dense_ssm_chunked', 3)
+				kernels = 3 if lib.dense_ssm_chunked_scratch(ctypes.byref(a)) else M // rows_per_seq
+				_dense.check(lib.dense_ssm_chunked(ctypes.byref(a), st), 'dense_ssm_chunked', kernels)
 			else:
 				_dense.check(lib.dense_ssm_scan(ctypes.byref(a), st), 'dense_ssm_scan')
 		y = torch.empty((M, self.w_o.shape[0]), dtype=torch.float32, device=dev)
@@ -113,6 +114,8 @@ class StateSpaceMixer(nn.Module):
 		u = torch.empty((a.M, a.conv_ld), dtype=dtype, device=dev)
 		a.u = ptr(u)
 		if not chunked:
+			return (u,)
+		if not _dense.lib().dense_ssm_chunked_scratch(ctypes.byref(a)):
 			return (u,)
 		n = a.M // a.rows_per_seq * ((a.rows_per_seq + _dense.SSM_CHUNK - 1) // _dense.SSM_CHUNK)
 		states = torch.empty((n, s.heads, s.vdim, s.state), dtype=torch.float32, device=dev)

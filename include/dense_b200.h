@@ -217,7 +217,10 @@ int dense_gqa_prefill(const dense_gqa_t *args, int start, void *stream);
 int dense_ssm_step(const dense_ssm_t *args, void *stream);                   /* rows_per_seq = 1, raw fp32 */
 int dense_ssm_conv(const dense_ssm_t *args, int dtype, void *stream);        /* portions: u */
 int dense_ssm_scan(const dense_ssm_t *args, void *stream);                   /* portions, raw and u fp32: out, state, ring, token by token */
-int dense_ssm_chunked(const dense_ssm_t *args, void *stream);                /* the same for bf16 raw and u in chunks (three kernels) */
+/* The same for bf16 raw and u in chunks.  One tensor-core kernel per sequence when vdim and state are multiples of 16 and state is at
+ * most 128, else three kernels, which need chunk_s and chunk_decay (dense_ssm_chunked_scratch = 1). */
+int dense_ssm_chunked(const dense_ssm_t *args, void *stream);
+int dense_ssm_chunked_scratch(const dense_ssm_t *args);
 
 #ifdef __cplusplus
 }
