@@ -1288,7 +1288,7 @@ def lifinex_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: 
 			e.n_q, e.n_kv, e.kv_out = mx.dt_at, steps.shape[1], steps.data_ptr()
 		gemm('state-space in-projection', mx.w_in, e, ssm.mixer_norm)
 		state = 4 * s.heads * s.vdim * s.state
-		g = torch.randn((M, padded(s.inner)), device=dev)
+		g = torch.randn((M, padded(s.inner)), device=dev).to(raw.dtype)
 		args = []
 		for _ in range(max(2, min(80, int(320e6 / state))) if decode else 2):
 			c = StaticCache([s.cache_layout()], 1, bf, dev)[0]
@@ -1299,15 +1299,15 @@ def lifinex_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: 
 			record('decode state-space step', graph_us([lambda a=a: call(lib.dense_ssm_step, ctypes.byref(a)) for a in args]), 2 * state + esz(raw, g) + 4 * (s.taps + 1) * a.conv_ld)
 		else:
 			record('prompt state-space convolution', graph_us([lambda a=a: call(lib.dense_ssm_conv, ctypes.byref(a), 0) for a in args] * 2), M * a.conv_ld * 4)
-			record('prompt state-space recurrence', graph_us([lambda a=a: call(lib.dense_ssm_chunked, ctypes.byref(a)) for a in args] * 2), M * a.conv_ld * 2 + M * s.inner * 6 + esz(steps) + 2 * state)
+			record('prompt state-space recurrence', graph_us([lambda a=a: call(lib.dense_ssm_chunked, ctypes.byref(a)) for a in args] * 2), M * a.conv_ld * 2 + M * s.inner * 4 + esz(steps) + 2 * state)
 			gs = Stream(s.inner, padded(s.inner), cfg.norm_eps, x=g)
-			record('prompt state-space norm', graph_us([lambda: prepare_rows(gs, ctl, bf, False, mx.norm)] * 4), M * s.inner * 6)
+			record('prompt state-space norm', graph_us([lambda: prepare_rows(gs, ctl, bf, False, mx.norm)] * 4), M * s.inner * 4)
 		if decode:
 			gs = Stream(s.inner, padded(s.inner), cfg.norm_eps, x=g)
 			record('decode state-space norm, out-projection', graph_us([lambda c=c: project_stream(gs, c, epilogue(_dense.EPI_F32, y), ctl, keep=False, final=mx.norm) for c in copies(mx.w_o)]),
 				   esz(mx.w_o))
 		else:
-			gemm('state-space out-projection', mx.w_o, epilogue(_dense.EPI_F32, y), x=g.to(bf))
+			gemm('state-space out-projection', mx.w_o, epilogue(_dense.EPI_F32, y), x=g)
 		# ---- feed-forward, side input, pass entry, logits ----
 		act = torch.empty((M, att.mlp.down.shape[1]), dtype=bf, device=dev)
 		gemm('gate/up', att.mlp.gate_up, att.mlp.gated(act), att.mlp_norm)

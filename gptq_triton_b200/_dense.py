@@ -25,7 +25,7 @@ _P, _I = c_void_p, c_int
 
 
 class Rows(ctypes.Structure):
-	_fields_ = [('x_in', _P), ('x_out', _P), ('y', _P), ('gain', _P), ('shift', _P), ('fin_w', _P), ('fin_b', _P), ('table', _P), ('token', _P),
+	_fields_ = [('x_in', _P), ('x_t', _I), ('x_out', _P), ('y', _P), ('gain', _P), ('shift', _P), ('fin_w', _P), ('fin_b', _P), ('table', _P), ('token', _P),
 				('vocab', c_int64), ('pos_table', _P), ('pos', _P), ('max_pos', _I), ('y_norm', _I), ('fin_norm', _I), ('fin_groups', _I), ('width', _I), ('ld', _I), ('eps', c_float), ('status', _P)]
 
 

@@ -52,6 +52,7 @@ template <> struct Elem<bf16> {
 	static __device__ __forceinline__ float ldcg(const bf16 *p) {
 		return __uint_as_float((uint32_t)__ldcg(reinterpret_cast<const unsigned short *>(p)) << 16);
 	}
+	static __device__ __forceinline__ float4 ldcg4(const bf16 *p) { return unpack(__ldcg(reinterpret_cast<const uint2 *>(p))); }
 	static __device__ __forceinline__ float ldg(const bf16 *p) { return __uint_as_float((uint32_t)__ldg(reinterpret_cast<const unsigned short *>(p)) << 16); }
 	static __device__ __forceinline__ void store(bf16 *p, float v) { *p = __float2bfloat16_rn(v); }
 };
@@ -63,6 +64,7 @@ template <> struct Elem<float> {
 		store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
 	}
 	static __device__ __forceinline__ float ldcg(const float *p) { return __ldcg(p); }
+	static __device__ __forceinline__ float4 ldcg4(const float *p) { return __ldcg(reinterpret_cast<const float4 *>(p)); }
 	static __device__ __forceinline__ float ldg(const float *p) { return __ldg(p); }
 	static __device__ __forceinline__ void store(float *p, float v) { *p = v; }
 };
@@ -150,17 +152,26 @@ __device__ __forceinline__ float4 rp_affine(float4 v, float mean, float inv, con
 
 // The RMS norm of equal parts of row x (global memory, `width` columns): a warp sums a share of a part, the shares of a part
 // are added in order.  inv: fin_groups (or DN_WARPS, if that is more) floats of shared memory.
-template <typename T>
-__device__ void norm_parts(const RowPrep &p, const float *x, T *dst, float *inv) {
+template <typename T, typename S>
+__device__ void norm_parts(const RowPrep &p, const S *x, T *dst, float *inv) {
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n = p.width / p.fin_groups;
-	const int shares = p.fin_groups >= DN_WARPS ? 1 : DN_WARPS / p.fin_groups, per = (n + shares - 1) / shares;
+	const int shares = p.fin_groups >= DN_WARPS ? 1 : DN_WARPS / p.fin_groups;
+	const bool quads = n % 4 == 0;                      // parts are whole groups of four entries (of the padded row, which is aligned)
+	const int per = quads ? ((n >> 2) + shares - 1) / shares * 4 : (n + shares - 1) / shares;
 	for (int i = warp; i < p.fin_groups * shares; i += DN_WARPS) {
 		const int g = i / shares, c0 = (i - g * shares) * per, c1 = min(c0 + per, n);
 		float s = 0.f;
+		if (quads) {
 #pragma unroll 8
-		for (int c = c0 + lane; c < c1; c += 32) {
-			const float v = __ldcg(x + (size_t)g * n + c);
-			s = fmaf(v, v, s);
+			for (int c = c0 + 4 * lane; c < c1; c += 128) {
+				const float4 v = Elem<S>::ldcg4(x + (size_t)g * n + c);
+				s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+			}
+		} else {
+			for (int c = c0 + lane; c < c1; c += 32) {
+				const float v = Elem<S>::ldcg(x + (size_t)g * n + c);
+				s = fmaf(v, v, s);
+			}
 		}
 		s = warp_sum(s);
 		if (lane == 0) inv[i] = s;
@@ -176,7 +187,7 @@ __device__ void norm_parts(const RowPrep &p, const float *x, T *dst, float *inv)
 	if (tid < p.fin_groups) inv[tid] = f;
 	__syncthreads();
 	for (int u = tid; u < p.ld >> 2; u += DN_THREADS) {
-		const float4 v = __ldcg(reinterpret_cast<const float4 *>(x) + u);
+		const float4 v = Elem<S>::ldcg4(x + 4 * u);
 		const int c = 4 * u, g = min(c / n, p.fin_groups - 1), edge = (g + 1) * n;
 		const float f0 = inv[g];
 		float4 w = p.fin_w ? __ldg(reinterpret_cast<const float4 *>(p.fin_w) + u) : make_float4(1.f, 1.f, 1.f, 1.f);
@@ -198,7 +209,8 @@ __device__ void prepare_row(const RowPrep &p, int m, T *dst, bool write_x, float
 	size_t xb = (size_t)m * p.ld, pb = 0;
 	const size_t yb = xb;
 	if (p.fin_groups > 1) {
-		norm_parts<T>(p, p.x_in + xb, dst, red + 4 * DN_WARPS);
+		if (p.x_t) norm_parts<T, T>(p, reinterpret_cast<const T *>(p.x_in) + xb, dst, red + 4 * DN_WARPS);
+		else norm_parts<T, float>(p, reinterpret_cast<const float *>(p.x_in) + xb, dst, red + 4 * DN_WARPS);
 		return;
 	}
 	if (p.table) {
@@ -218,7 +230,7 @@ __device__ void prepare_row(const RowPrep &p, int m, T *dst, bool write_x, float
 		}
 	}
 	auto read_x = [&](int u) {
-		if (!p.table) return __ldcg(reinterpret_cast<const float4 *>(p.x_in + xb) + u);
+		if (!p.table) return p.x_t ? Elem<T>::ldcg4(reinterpret_cast<const T *>(p.x_in) + xb + 4 * u) : __ldcg(reinterpret_cast<const float4 *>(reinterpret_cast<const float *>(p.x_in) + xb) + u);
 		const float4 v = Elem<T>::load4(reinterpret_cast<const T *>(p.table) + xb + 4 * u);
 		return p.pos_table ? add4(v, Elem<T>::load4(reinterpret_cast<const T *>(p.pos_table) + pb + 4 * u)) : v;
 	};

@@ -48,7 +48,7 @@ static bool rows_bad(const RowPrep &r, int dtype) {
 	if ((r.fin_w || r.fin_b) && r.fin_norm == DENSE_NORM_NONE) return true;
 	if (r.fin_groups < 1 || r.fin_groups > DENSE_MAX_NORM_GROUPS) return true;
 	if (r.fin_groups > 1 && (r.fin_norm != DENSE_NORM_RMS || r.width % r.fin_groups || r.table || r.y || r.x_out || r.fin_b)) return true;
-	if (r.x_out && r.x_out == r.x_in) return true;
+	if (r.x_out && (const void *)r.x_out == r.x_in) return true;
 	return !aligned16(r.pos_table) || !aligned16(r.x_in) || !aligned16(r.x_out) || !aligned16(r.y) || !aligned16(r.gain) || !aligned16(r.shift) || !aligned16(r.fin_w) || !aligned16(r.fin_b) || !aligned16(r.table);
 }
 

@@ -364,14 +364,14 @@ __global__ void __launch_bounds__(DN_THREADS, NK > 8 ? 1 : 2) ssm_chunk_out_kern
 				if (t < k.nt && c < k.np) {
 					const int col = k.head * p.vdim + k.p0 + c;
 					const bf16 *x = sx + t * LDX + c, *z = raw + (size_t)t * p.raw_ld + p.z_at + col;
-					float *o = p.out + (row0 + t) * p.out_ld + col;
+					bf16 *o = reinterpret_cast<bf16 *>(p.out) + (row0 + t) * p.out_ld + col;
 					if (vec) {                       // even columns: both entries are there
 						const uint32_t xv = *reinterpret_cast<const uint32_t *>(x), zv = __ldcg(reinterpret_cast<const uint32_t *>(z));
-						*reinterpret_cast<float2 *>(o) = make_float2(fmaf(d, __uint_as_float(xv << 16), acc[q][2 * h]) * silu_fast(__uint_as_float(zv << 16)),
-																   fmaf(d, __uint_as_float(xv & 0xFFFF0000u), acc[q][2 * h + 1]) * silu_fast(__uint_as_float(zv & 0xFFFF0000u)));
+						*reinterpret_cast<uint32_t *>(o) = pack_bf16(fmaf(d, __uint_as_float(xv << 16), acc[q][2 * h]) * silu_fast(__uint_as_float(zv << 16)),
+																 fmaf(d, __uint_as_float(xv & 0xFFFF0000u), acc[q][2 * h + 1]) * silu_fast(__uint_as_float(zv & 0xFFFF0000u)));
 					} else {
-						o[0] = fmaf(d, __bfloat162float(x[0]), acc[q][2 * h]) * silu_fast(Elem<bf16>::ldcg(z));
-						if (c + 1 < k.np) o[1] = fmaf(d, __bfloat162float(x[1]), acc[q][2 * h + 1]) * silu_fast(Elem<bf16>::ldcg(z + 1));
+						Elem<bf16>::store(o, fmaf(d, __bfloat162float(x[0]), acc[q][2 * h]) * silu_fast(Elem<bf16>::ldcg(z)));
+						if (c + 1 < k.np) Elem<bf16>::store(o + 1, fmaf(d, __bfloat162float(x[1]), acc[q][2 * h + 1]) * silu_fast(Elem<bf16>::ldcg(z + 1)));
 					}
 				}
 			}

@@ -137,7 +137,7 @@ __global__ void __launch_bounds__(DN_THREADS) ssm_step_kernel(const SsmArgs p) {
 	st.store(s, p0 + warp * SS_RW, p.vdim, p.state, lane);
 #pragma unroll
 	for (int r = 0; r < SS_RW; ++r)
-		if (lane == r && row < p.vdim) p.out[(size_t)m * p.out_ld + head * p.vdim + row] = fmaf(d, x[r], y[r]) * silu_exact(z);
+		if (lane == r && row < p.vdim) reinterpret_cast<float *>(p.out)[(size_t)m * p.out_ld + head * p.vdim + row] = fmaf(d, x[r], y[r]) * silu_exact(z);
 }
 
 template <typename T> __device__ __forceinline__ float2 load2(const T *p);
@@ -236,7 +236,7 @@ __global__ void __launch_bounds__(DN_THREADS) ssm_scan_kernel(const SsmArgs p) {
 			st.step(x, &s_u[t][sl.nx], &s_u[t][sl.nx + sl.N], s_dt[t], s_decay[t], p.state, lane, y);
 #pragma unroll
 			for (int r = 0; r < SS_RW; ++r)
-				if (lane == r && row < p.vdim) p.out[((size_t)seq * T + t0 + t) * p.out_ld + head * p.vdim + row] = fmaf(d, x[r], y[r]) * s_z[t][warp * SS_RW + r];
+				if (lane == r && row < p.vdim) reinterpret_cast<float *>(p.out)[((size_t)seq * T + t0 + t) * p.out_ld + head * p.vdim + row] = fmaf(d, x[r], y[r]) * s_z[t][warp * SS_RW + r];
 		}
 	}
 	st.store(s, p0 + warp * SS_RW, p.vdim, p.state, lane);

@@ -11,7 +11,9 @@
 //   warps 0-7   scale the inputs, split and decay S, form M, write y        warp 8   TMA: C, B, X tiles, two stages
 //   warp 10     step sizes and prefix sums of the next chunk                 warp 9   MMA
 // B and C are operands in both roles (rows of tokens as rows, and as the summed dimension); shared memory holds them once, in the
-// 128-byte-swizzled layout that serves both.  Every wait is bounded.
+// 128-byte-swizzled layout that serves both.  The two parts of S are one operand of twice the width, their products are added when
+// y is formed.  One thread issues every MMA, so it only adds constants to descriptors.  Gates and outputs pass through the
+// input tile, which nobody needs any more, so that global memory sees whole rows.  Every wait is bounded.
 #include <algorithm>
 
 #include "prefill_common.cuh"
@@ -24,7 +26,7 @@ namespace {
 constexpr int ST_L = SS_CHUNK, ST_P = 64;
 constexpr int ST_CHUNK = ST_L * 128;                    // bytes of a 128 x 64 bf16 tile
 constexpr int ST_WORK = 256, ST_THREADS = ST_WORK + 96;
-constexpr uint32_t T_G = 0, T_YI = 256, T_YA = 320, T_S = 384;      // tensor memory columns: two G / M buffers, Yi, Ya, S
+constexpr uint32_t T_G = 0, T_YI = 256, T_YA = 384, T_S = 448;      // tensor memory columns: two G / M buffers, Yi (both parts of S), Ya, S
 
 struct StPlan {
 	int nc;                                             // 64-column tiles of C
@@ -172,14 +174,22 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 	} else if (warp == 9) {
 		if (lane == 0) {
 			const uint32_t fmt = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(ST_L >> 4) << 24);          // D fp32, A/B bf16, M = 128
-			const uint32_t nw = (uint32_t)((np + 15) / 16 * 16), at_n = (nw >> 3) << 17;
-			const uint32_t id_g = fmt | ((uint32_t)(ST_L >> 3) << 17), id_y = fmt | (1u << 16) | at_n, id_u = id_y | (1u << 15);
+			const uint32_t wide = (uint32_t)(ST_L >> 3) << 17, at_n = (uint32_t)((np + 15) / 16 * 2) << 17;
+			const uint32_t id_g = fmt | wide, id_i = fmt | wide | (1u << 16), id_y = fmt | at_n | (1u << 16), id_u = id_y | (1u << 15);
 			const int steps = p.state >> 4;
+			const uint64_t d_c = smem_desc_sw128(base), d_bk = smem_desc_sw128(base + pl.nc * ST_CHUNK), d_bm = desc_rows(base + pl.nc * ST_CHUNK),
+						   d_x = desc_rows(base + (pl.nc + 2) * ST_CHUNK), d_xs = desc_rows(sxs), d_s = desc_rows(sst);
+			const uint32_t stage16 = pl.stage >> 4;
+			constexpr uint32_t C16 = ST_CHUNK >> 4;
 			auto issue_g = [&](int c) {                   // C and B tiles have arrived
-				const uint32_t st = base + (c & 1) * pl.stage;
+				uint64_t a = d_c + (c & 1) * stage16, b = d_bk + (c & 1) * stage16;
+				const uint32_t d = tmem + T_G + (c & 1) * ST_L;
+#pragma unroll 1
 				for (int k = 0; k < steps; ++k) {
-					const uint32_t off = (k >> 2) * ST_CHUNK + (k & 3) * 32;
-					umma_f16(tmem + T_G + (c & 1) * ST_L, smem_desc_sw128(st + off), smem_desc_sw128(st + pl.nc * ST_CHUNK + off), id_g, k ? 1u : 0u);
+					umma_f16(d, a, b, id_g, k ? 1u : 0u);
+					const uint32_t next = (k & 3) == 3 ? C16 - 6 : 2;          // 16 entries further: 32 bytes, or the next tile
+					a += next;
+					b += next;
 				}
 				umma_commit(bar_g + 8 * (c & 1));
 			};
@@ -187,16 +197,21 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 			tc_fence_after();
 			if (ok) issue_g(0);
 			for (int c = 0; c < n && ok; ++c) {
-				const uint32_t st = base + (c & 1) * pl.stage, sx = st + (pl.nc + 2) * ST_CHUNK;
+				const uint32_t so = (c & 1) * stage16;
 				if (!(ok = wait_one(bar_r, c))) break;
 				tc_fence_after();
-				for (int part = 0; part < 2; ++part)
-					for (int k = 0; k < steps; ++k)
-						umma_f16(tmem + T_YI, smem_desc_sw128(st + (k >> 2) * ST_CHUNK + (k & 3) * 32), desc_rows(sst + part * ST_CHUNK) + 128 * k, id_y, part | k ? 1u : 0u);
+				const uint64_t bm = d_bm + so, x = d_x + so;
+				uint64_t a = d_c + so, b = d_s;
+#pragma unroll 1
+				for (int k = 0; k < steps; ++k) {
+					umma_f16(tmem + T_YI, a, b, id_i, k ? 1u : 0u);
+					a += (k & 3) == 3 ? C16 - 6 : 2;
+					b += 128;                                              // 16 rows of 128 bytes
+				}
+#pragma unroll
 				for (int part = 0; part < 2; ++part)
 #pragma unroll
-					for (int k = 0; k < ST_L / 16; ++k)
-						umma_f16(tmem + T_S, desc_rows(st + pl.nc * ST_CHUNK) + 128 * k, desc_rows(sxs + part * ST_CHUNK) + 128 * k, id_u, 1u);
+					for (int k = 0; k < ST_L / 16; ++k) umma_f16(tmem + T_S, bm + 128 * k, d_xs + part * C16 + 128 * k, id_u, 1u);
 				umma_commit(bar_u);
 				if (c + 1 < n) {
 					if (!(ok = wait_one(bar_full + 8 * ((c + 1) & 1), (c + 1) >> 1))) break;
@@ -205,11 +220,11 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 				}
 				if (!(ok = wait_one(bar_m, c))) break;
 				tc_fence_after();
+				const uint32_t m = tmem + T_G + (c & 1) * ST_L;
 #pragma unroll
 				for (int part = 0; part < 2; ++part)
 #pragma unroll
-					for (int k = 0; k < ST_L / 16; ++k)
-						umma_f16_ts(tmem + T_YA, tmem + T_G + (c & 1) * ST_L + (k >> 1) * 32 + part * 16 + (k & 1) * 8, desc_rows(sx) + 128 * k, id_y, part | k ? 1u : 0u);
+					for (int k = 0; k < ST_L / 16; ++k) umma_f16_ts(tmem + T_YA, m + (k >> 1) * 32 + part * 16 + (k & 1) * 8, x + 128 * k, id_y, part | k ? 1u : 0u);
 				umma_commit(bar_y);
 				umma_commit(bar_empty + 8 * (c & 1));
 			}
@@ -231,11 +246,14 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 			tmem_st32(tmem + T_S + lanes + 32 * h, v);
 			tmem_st_wait();
 		}
-		const bf16 *zrow = reinterpret_cast<const bf16 *>(p.raw) + (size_t)seq * T * p.raw_ld + p.z_at + head * p.vdim + p0 + 32 * h;
-		float *orow = p.out + (size_t)seq * T * p.out_ld + head * p.vdim + p0 + 32 * h;
+		// a warp's part of z and y: 32 tokens x 64 bytes; four lanes per row when it meets global memory
+		const int cr = q * 32 + (lane >> 2), cu = lane & 3;
+		const bool ccol = 32 * h + 8 * cu < np;
+		const bf16 *zg = reinterpret_cast<const bf16 *>(p.raw) + (size_t)seq * T * p.raw_ld + p.z_at + head * p.vdim + p0 + 32 * h + 8 * cu;
+		bf16 *og = reinterpret_cast<bf16 *>(p.out) + (size_t)seq * T * p.out_ld + head * p.vdim + p0 + 32 * h + 8 * cu;
 		bool ok = true;
 		for (int c = 0; c < n && ok; ++c) {
-			const int s = c & 1, t = c * ST_L + row;
+			const int s = c & 1, t0 = c * ST_L;
 			unsigned char *stage = st_smem + (size_t)s * pl.stage, *xt = stage + (size_t)(pl.nc + 2) * ST_CHUNK;
 			const float *hi_j = s_hi + s * ST_L, *w = s_w + s * ST_L;
 			if (!(ok = wait_warp(bar_full + 8 * s, c >> 1))) break;
@@ -285,20 +303,17 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 			fence_proxy_async();
 			tc_fence_before();
 			mbar_arrive(bar_r);
-			uint32_t z[16];                                                 // gates of this thread's outputs, requested early
+			uint4 z[4];                                                      // gates, requested early
 #pragma unroll
-			for (int i = 0; i < 4; ++i) {
-				uint4 v = make_uint4(0u, 0u, 0u, 0u);
-				if (t < T && 32 * h + 8 * i < np) v = __ldcg(reinterpret_cast<const uint4 *>(zrow + (size_t)t * p.raw_ld) + i);
-				z[4 * i] = v.x;
-				z[4 * i + 1] = v.y;
-				z[4 * i + 2] = v.z;
-				z[4 * i + 3] = v.w;
-			}
+			for (int i = 0; i < 4; ++i)
+				z[i] = ccol && t0 + cr + 8 * i < T ? __ldcg(reinterpret_cast<const uint4 *>(zg + (size_t)(t0 + cr + 8 * i) * p.raw_ld)) : make_uint4(0u, 0u, 0u, 0u);
 			// ---- M over G: this thread's row, half of the columns ----
 			if (!(ok = wait_warp(bar_g + 8 * s, c >> 1))) break;
 			tc_fence_after();
 			const float si = hi_j[row], si_lo = __bfloat162float(s_lo[s * ST_L + row]);
+			// left of the diagonal's 32 x 32 blocks the factor splits at the block's first row r: 2^(s_i - s_r) * 2^(s_r - s_j) dt_j, both at
+			// most of the order of one; a lane computes the second one for one column
+			const float rh = hi_j[q * 32], rl = __bfloat162float(s_lo[s * ST_L + q * 32]), from_r = ex2((si - rh) + (si_lo - rl));
 #pragma unroll 1
 			for (int b = 0; b < 2; ++b) {
 				const int j0 = 64 * h + 32 * b;
@@ -310,20 +325,21 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 				} else {
 					float v[32];
 					tmem_ld32(at, v);
-					tmem_ld_wait();
-					tmem_settle(v);
-					const bool edge = j0 == q * 32;
+					const float wl = w[j0 + lane], hl = hi_j[j0 + lane];
+					if (j0 < q * 32) {
+						const float to_r = ex2((rh - hl) + (rl + wl));
+						tmem_ld_wait();
+						tmem_settle(v);
 #pragma unroll
-					for (int i = 0; i < 8; ++i) {
-						const float4 wj = *reinterpret_cast<const float4 *>(w + j0 + 4 * i), hj = *reinterpret_cast<const float4 *>(hi_j + j0 + 4 * i);
-						v[4 * i] *= ex2((si - hj.x) + (si_lo + wj.x));
-						v[4 * i + 1] *= ex2((si - hj.y) + (si_lo + wj.y));
-						v[4 * i + 2] *= ex2((si - hj.z) + (si_lo + wj.z));
-						v[4 * i + 3] *= ex2((si - hj.w) + (si_lo + wj.w));
-					}
-					if (edge) {
+						for (int i = 0; i < 32; ++i) v[i] *= from_r * __shfl_sync(0xffffffffu, to_r, i);
+					} else {
+						tmem_ld_wait();
+						tmem_settle(v);
 #pragma unroll
-						for (int i = 0; i < 32; ++i) v[i] = i <= lane ? v[i] : 0.f;
+						for (int i = 0; i < 32; ++i) {
+							const float f = ex2((si - __shfl_sync(0xffffffffu, hl, i)) + (si_lo + __shfl_sync(0xffffffffu, wl, i)));
+							v[i] = i <= lane ? v[i] * f : 0.f;
+						}
 					}
 #pragma unroll
 					for (int i = 0; i < 16; ++i) st_split(v[2 * i], v[2 * i + 1], out[i], out[16 + i]);
@@ -338,31 +354,47 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 			tc_fence_after();
 			if (cols) {
 				const float e = ex2(si + si_lo);
+				unsigned char *own = xt + row * 128;
+				auto unit = [&](int r, int u) { return ((4 * h + u) ^ (r & 7)) * 16; };
+				uint4 x[4];
+#pragma unroll
+				for (int u = 0; u < 4; ++u) x[u] = *reinterpret_cast<const uint4 *>(own + unit(row, u));
+				__syncwarp();
+#pragma unroll
+				for (int i = 0; i < 4; ++i) *reinterpret_cast<uint4 *>(xt + (cr + 8 * i) * 128 + unit(cr + 8 * i, cu)) = z[i];
+				__syncwarp();
 #pragma unroll
 				for (int b = 0; b < 2; ++b) {
-					float yi[16], ya[16];
-					tmem_ld16(tmem + T_YI + lanes + 32 * h + 16 * b, yi);
+					float y0[16], y1[16], ya[16];
+					tmem_ld16(tmem + T_YI + lanes + 32 * h + 16 * b, y0);
+					tmem_ld16(tmem + T_YI + ST_P + lanes + 32 * h + 16 * b, y1);
 					tmem_ld16(tmem + T_YA + lanes + 32 * h + 16 * b, ya);
 					tmem_ld_wait();
-					tmem_settle(yi);
+					tmem_settle(y0);
+					tmem_settle(y1);
 					tmem_settle(ya);
-					if (t < T && 32 * h + 16 * b < np) {
 #pragma unroll
-						for (int u = 0; u < 2; ++u) {
-							const uint4 x = *reinterpret_cast<const uint4 *>(xt + row * 128 + ((4 * h + 2 * b + u) ^ (row & 7)) * 16);
-							const uint32_t xs[4] = {x.x, x.y, x.z, x.w};
-							float o[8];
+					for (int u = 0; u < 2; ++u) {
+						uint4 *at = reinterpret_cast<uint4 *>(own + unit(row, 2 * b + u));
+						const uint4 zv = *at, xv = x[2 * b + u];
+						const uint32_t zs[4] = {zv.x, zv.y, zv.z, zv.w}, xs[4] = {xv.x, xv.y, xv.z, xv.w};
+						uint32_t o[4];
 #pragma unroll
-							for (int j = 0; j < 4; ++j) {
-								const int i = 8 * u + 2 * j;
-								const uint32_t zz = z[8 * b + 4 * u + j];
-								o[2 * j] = fmaf(d, __uint_as_float(xs[j] << 16), fmaf(e, yi[i], ya[i])) * silu_fast(__uint_as_float(zz << 16));
-								o[2 * j + 1] = fmaf(d, __uint_as_float(xs[j] & 0xFFFF0000u), fmaf(e, yi[i + 1], ya[i + 1])) * silu_fast(__uint_as_float(zz & 0xFFFF0000u));
-							}
-							Elem<float>::store8(orow + (size_t)t * p.out_ld + 16 * b + 8 * u, o);
+						for (int j = 0; j < 4; ++j) {
+							const int i = 8 * u + 2 * j;
+							const float a0 = fmaf(d, __uint_as_float(xs[j] << 16), fmaf(e, y0[i] + y1[i], ya[i]));
+							const float a1 = fmaf(d, __uint_as_float(xs[j] & 0xFFFF0000u), fmaf(e, y0[i + 1] + y1[i + 1], ya[i + 1]));
+							o[j] = pack_bf16(a0 * silu_fast(__uint_as_float(zs[j] << 16)), a1 * silu_fast(__uint_as_float(zs[j] & 0xFFFF0000u)));
 						}
+						*at = make_uint4(o[0], o[1], o[2], o[3]);
 					}
 				}
+				__syncwarp();
+#pragma unroll
+				for (int i = 0; i < 4; ++i)
+					if (ccol && t0 + cr + 8 * i < T)
+						*reinterpret_cast<uint4 *>(og + (size_t)(t0 + cr + 8 * i) * p.out_ld) = *reinterpret_cast<const uint4 *>(xt + (cr + 8 * i) * 128 + unit(cr + 8 * i, cu));
+				fence_proxy_async();                          // the tile is written by a copy next
 			}
 			tc_fence_before();
 			mbar_arrive(bar_empty + 8 * s);
@@ -396,7 +428,7 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 
 }   // namespace
 
-bool ssm_tc_ok(const SsmArgs &p) { return p.vdim % 16 == 0 && p.state % 16 == 0 && p.state <= 128 && p.out_ld % 4 == 0; }
+bool ssm_tc_ok(const SsmArgs &p) { return p.vdim % 16 == 0 && p.state % 16 == 0 && p.state <= 128 && p.out_ld % 8 == 0; }
 
 int ssm_tc_launch(const SsmArgs &p, cudaStream_t stream) {
 	const int T = p.rows_per_seq, seqs = p.M / T, slices = (p.vdim + ST_P - 1) / ST_P;

@@ -37,7 +37,8 @@ def pad_to(t: torch.Tensor, *shape: int) -> torch.Tensor:
 @dataclass
 class Stream:
 	"""The residual stream between two sublayers, not yet formed: rows of `table` by token (plus rows of `pos_table` by
-	position), or x (+ norm(y) * gain + shift).  The next projection (or the row kernel) forms it."""
+	position), or x (+ norm(y) * gain + shift).  The next projection (or the row kernel) forms it.  x is fp32, or (rows that are
+	not the residual stream) in the activation dtype."""
 	width: int
 	ld: int
 	eps: float
@@ -72,7 +73,7 @@ class Stream:
 			if self.pos_table is not None:
 				r.pos_table, r.pos, r.max_pos = ptr(self.pos_table), ptr(self.pos), self.pos_table.shape[0]
 		else:
-			r.x_in = ptr(self.x)
+			r.x_in, r.x_t = ptr(self.x), int(self.x.dtype != torch.float32)
 		r.x_out, r.y, r.y_norm, r.gain, r.shift = ptr(x_out), ptr(self.y), self.y_norm, ptr(self.gain), ptr(self.shift)
 		r.fin_groups = 1
 		if final is not None:

@@ -83,7 +83,7 @@ class StateSpaceMixer(nn.Module):
 			e.n_q, e.n_kv, e.kv_out = n, n_dt, ptr(steps)
 		x = project_stream(stream, self.w_in, e, control, final=norm)
 		inner = padded(s.inner)
-		out = (torch.empty if inner == s.inner else torch.zeros)((M, inner), dtype=torch.float32, device=dev)
+		out = (torch.empty if inner == s.inner else torch.zeros)((M, inner), dtype=raw.dtype, device=dev)
 		a = self.arguments(raw, steps, cache, pos, rows_per_seq, out, control)
 		lib, st = _dense.lib(), stream_ptr(dev)
 		if rows_per_seq == 1:

@@ -46,7 +46,8 @@ extern "C" {
  * shift absent: 0).  x_out (optional, never the same as x_in) receives x.  The prepared row is fin_norm(x) * fin_w + fin_b (each
  * optional); an RMS norm may work on fin_groups equal parts of the row, each by its own mean square (then y must be absent). */
 typedef struct {
-	const float *x_in;
+	const void *x_in;                  /* fp32, or (x_t) in the activation dtype */
+	int x_t;
 	float *x_out;
 	const float *y;
 	const float *gain, *shift;
@@ -181,7 +182,7 @@ typedef struct {
 	void *u;                           /* scratch of portions: [M, conv_ld], the type of raw */
 	float *chunk_s;                    /* scratch of dense_ssm_chunked: [sequences, chunks, heads, vdim, state] */
 	float *chunk_decay;                /* [sequences, chunks, heads] */
-	float *out;                        /* [M, out_ld] */
+	void *out;                         /* [M, out_ld], the type of raw */
 	int64_t out_ld;
 	int *status;
 } dense_ssm_t;
