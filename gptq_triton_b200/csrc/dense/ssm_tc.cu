@@ -12,8 +12,9 @@
 //   warp 10     step sizes and prefix sums of the next chunk                 warp 9   MMA
 // B and C are operands in both roles (rows of tokens as rows, and as the summed dimension); shared memory holds them once, in the
 // 128-byte-swizzled layout that serves both.  The two parts of S are one operand of twice the width, their products are added when
-// y is formed.  One thread issues every MMA, so it only adds constants to descriptors.  Gates and outputs pass through the
-// input tile, which nobody needs any more, so that global memory sees whole rows.  Every wait is bounded.
+// y is formed.  An MMA whose first operand comes from shared memory costs about 120 cycles however narrow it is, so the products
+// of a chunk take about as long as the other warps' work; these prepare the next chunk between forming M and reading y.
+// Outputs pass through the input tile, which nobody needs any more, so that global memory sees whole rows.  Every wait is bounded.
 #include <algorithm>
 
 #include "prefill_common.cuh"
@@ -26,7 +27,7 @@ namespace {
 constexpr int ST_L = SS_CHUNK, ST_P = 64;
 constexpr int ST_CHUNK = ST_L * 128;                    // bytes of a 128 x 64 bf16 tile
 constexpr int ST_WORK = 256, ST_THREADS = ST_WORK + 96;
-constexpr uint32_t T_G = 0, T_YI = 256, T_YA = 384, T_S = 448;      // tensor memory columns: two G / M buffers, Yi (both parts of S), Ya, S
+constexpr uint32_t T_G = 0, T_YI = 128, T_YA = 384, T_S = 448;      // tensor memory columns: G / M, two buffers of Yi (both parts of S), Ya, S
 
 struct StPlan {
 	int nc;                                             // 64-column tiles of C
@@ -80,8 +81,8 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 		for (int s = 0; s < 2; ++s) {
 			mbar_init(bar_full + 8 * s, 1 + 32);
 			mbar_init(bar_empty + 8 * s, ST_WORK + 1);
-			mbar_init(bar_g + 8 * s, 1);
 		}
+		mbar_init(bar_g, 1);
 		mbar_init(bar_r, ST_WORK);
 		mbar_init(bar_m, ST_WORK);
 		mbar_init(bar_y, 1);
@@ -183,15 +184,14 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 			constexpr uint32_t C16 = ST_CHUNK >> 4;
 			auto issue_g = [&](int c) {                   // C and B tiles have arrived
 				uint64_t a = d_c + (c & 1) * stage16, b = d_bk + (c & 1) * stage16;
-				const uint32_t d = tmem + T_G + (c & 1) * ST_L;
 #pragma unroll 1
 				for (int k = 0; k < steps; ++k) {
-					umma_f16(d, a, b, id_g, k ? 1u : 0u);
+					umma_f16(tmem + T_G, a, b, id_g, k ? 1u : 0u);
 					const uint32_t next = (k & 3) == 3 ? C16 - 6 : 2;          // 16 entries further: 32 bytes, or the next tile
 					a += next;
 					b += next;
 				}
-				umma_commit(bar_g + 8 * (c & 1));
+				umma_commit(bar_g);
 			};
 			bool ok = wait_one(bar_full, 0);
 			tc_fence_after();
@@ -204,7 +204,7 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 				uint64_t a = d_c + so, b = d_s;
 #pragma unroll 1
 				for (int k = 0; k < steps; ++k) {
-					umma_f16(tmem + T_YI, a, b, id_i, k ? 1u : 0u);
+					umma_f16(tmem + T_YI + (c & 1) * 2 * ST_P, a, b, id_i, k ? 1u : 0u);
 					a += (k & 3) == 3 ? C16 - 6 : 2;
 					b += 128;                                              // 16 rows of 128 bytes
 				}
@@ -213,20 +213,19 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 #pragma unroll
 					for (int k = 0; k < ST_L / 16; ++k) umma_f16(tmem + T_S, bm + 128 * k, d_xs + part * C16 + 128 * k, id_u, 1u);
 				umma_commit(bar_u);
+				if (!(ok = wait_one(bar_m, c))) break;
+				tc_fence_after();
+#pragma unroll
+				for (int part = 0; part < 2; ++part)
+#pragma unroll
+					for (int k = 0; k < ST_L / 16; ++k) umma_f16_ts(tmem + T_YA, tmem + T_G + (k >> 1) * 32 + part * 16 + (k & 1) * 8, x + 128 * k, id_y, part | k ? 1u : 0u);
+				umma_commit(bar_y);
+				umma_commit(bar_empty + 8 * (c & 1));
 				if (c + 1 < n) {
 					if (!(ok = wait_one(bar_full + 8 * ((c + 1) & 1), (c + 1) >> 1))) break;
 					tc_fence_after();
 					issue_g(c + 1);
 				}
-				if (!(ok = wait_one(bar_m, c))) break;
-				tc_fence_after();
-				const uint32_t m = tmem + T_G + (c & 1) * ST_L;
-#pragma unroll
-				for (int part = 0; part < 2; ++part)
-#pragma unroll
-					for (int k = 0; k < ST_L / 16; ++k) umma_f16_ts(tmem + T_YA, m + (k >> 1) * 32 + part * 16 + (k & 1) * 8, x + 128 * k, id_y, part | k ? 1u : 0u);
-				umma_commit(bar_y);
-				umma_commit(bar_empty + 8 * (c & 1));
 			}
 			umma_commit(bar_end);                         // every MMA has completed before tensor memory goes back
 			mbar_wait_bounded(bar_end, 0, ATTN_SPIN);
@@ -246,38 +245,33 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 			tmem_st32(tmem + T_S + lanes + 32 * h, v);
 			tmem_st_wait();
 		}
-		// a warp's part of z and y: 32 tokens x 64 bytes; four lanes per row when it meets global memory
+		// a warp's part of z and y: 32 tokens x 64 bytes; four lanes per row where they meet global memory (rows lie far apart there)
 		const int cr = q * 32 + (lane >> 2), cu = lane & 3;
 		const bool ccol = 32 * h + 8 * cu < np;
 		const bf16 *zg = reinterpret_cast<const bf16 *>(p.raw) + (size_t)seq * T * p.raw_ld + p.z_at + head * p.vdim + p0 + 32 * h + 8 * cu;
 		bf16 *og = reinterpret_cast<bf16 *>(p.out) + (size_t)seq * T * p.out_ld + head * p.vdim + p0 + 32 * h + 8 * cu;
-		bool ok = true;
-		for (int c = 0; c < n && ok; ++c) {
-			const int s = c & 1, t0 = c * ST_L;
-			unsigned char *stage = st_smem + (size_t)s * pl.stage, *xt = stage + (size_t)(pl.nc + 2) * ST_CHUNK;
-			const float *hi_j = s_hi + s * ST_L, *w = s_w + s * ST_L;
-			if (!(ok = wait_warp(bar_full + 8 * s, c >> 1))) break;
-			if (c && !(ok = wait_warp(bar_u, c - 1))) break;
-			tc_fence_after();
-			const float end = hi_j[ST_L - 1], end_lo = __bfloat162float(s_lo[s * ST_L + ST_L - 1]);
-			// ---- inputs times step size and decay to the chunk's end: element by element, so the tile's layout does not matter ----
-			{
-				const int trow = tid >> 1;                                  // two threads per token, half a row each
-				const float f = ex2((end - hi_j[trow]) + (end_lo + w[trow]));
+		auto input_tile = [&](int c) { return st_smem + (size_t)(c & 1) * pl.stage + (size_t)(pl.nc + 2) * ST_CHUNK; };
+		// operands of chunk c that follow from the state and the inputs (both operands of chunk c - 1 have been read)
+		auto prepare = [&](int c) {
+			const unsigned char *xt = input_tile(c);
+			const float *hi_j = s_hi + (c & 1) * ST_L, *w = s_w + (c & 1) * ST_L;
+			const float end = hi_j[ST_L - 1], end_lo = __bfloat162float(s_lo[(c & 1) * ST_L + ST_L - 1]);
+			// inputs times step size and decay to the chunk's end: element by element, so the tile's layout does not matter
+			const int trow = tid >> 1;                                  // two threads per token, half a row each
+			const float fx = ex2((end - hi_j[trow]) + (end_lo + w[trow]));
 #pragma unroll
-				for (int i = 0; i < 4; ++i) {
-					const uint32_t off = (uint32_t)trow * 128 + (uint32_t)(((tid & 1) * 4 + i + trow) & 7) * 16;      // (rotated against bank conflicts)
-					const uint4 x = *reinterpret_cast<const uint4 *>(xt + off);
-					const uint32_t xs[4] = {x.x, x.y, x.z, x.w};
-					uint32_t hi[4], lo[4];
+			for (int i = 0; i < 4; ++i) {
+				const uint32_t off = (uint32_t)trow * 128 + (uint32_t)(((tid & 1) * 4 + i + trow) & 7) * 16;      // (rotated against bank conflicts)
+				const uint4 x = *reinterpret_cast<const uint4 *>(xt + off);
+				const uint32_t xs[4] = {x.x, x.y, x.z, x.w};
+				uint32_t hi[4], lo[4];
 #pragma unroll
-					for (int j = 0; j < 4; ++j) st_split(__uint_as_float(xs[j] << 16) * f, __uint_as_float(xs[j] & 0xFFFF0000u) * f, hi[j], lo[j]);
-					unsigned char *dst = st_smem + 2 * (size_t)pl.stage + off;
-					*reinterpret_cast<uint4 *>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-					*reinterpret_cast<uint4 *>(dst + ST_CHUNK) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-				}
+				for (int j = 0; j < 4; ++j) st_split(__uint_as_float(xs[j] << 16) * fx, __uint_as_float(xs[j] & 0xFFFF0000u) * fx, hi[j], lo[j]);
+				unsigned char *dst = st_smem + 2 * (size_t)pl.stage + off;
+				*reinterpret_cast<uint4 *>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+				*reinterpret_cast<uint4 *>(dst + ST_CHUNK) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
 			}
-			// ---- S in two parts for Yi, then decayed ----
+			// S in two parts for Yi, then decayed
 			if (cols) {
 				float v[32];
 				tmem_ld32(tmem + T_S + lanes + 32 * h, v);
@@ -303,12 +297,18 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 			fence_proxy_async();
 			tc_fence_before();
 			mbar_arrive(bar_r);
+		};
+		bool ok = wait_warp(bar_full, 0);
+		if (ok) prepare(0);
+		for (int c = 0; c < n && ok; ++c) {
+			const int s = c & 1, t0 = c * ST_L;
+			const float *hi_j = s_hi + s * ST_L, *w = s_w + s * ST_L;
 			uint4 z[4];                                                      // gates, requested early
 #pragma unroll
 			for (int i = 0; i < 4; ++i)
 				z[i] = ccol && t0 + cr + 8 * i < T ? __ldcg(reinterpret_cast<const uint4 *>(zg + (size_t)(t0 + cr + 8 * i) * p.raw_ld)) : make_uint4(0u, 0u, 0u, 0u);
 			// ---- M over G: this thread's row, half of the columns ----
-			if (!(ok = wait_warp(bar_g + 8 * s, c >> 1))) break;
+			if (!(ok = wait_warp(bar_g, c))) break;
 			tc_fence_after();
 			const float si = hi_j[row], si_lo = __bfloat162float(s_lo[s * ST_L + row]);
 			// left of the diagonal's 32 x 32 blocks the factor splits at the block's first row r: 2^(s_i - s_r) * 2^(s_r - s_j) dt_j, both at
@@ -317,7 +317,7 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 #pragma unroll 1
 			for (int b = 0; b < 2; ++b) {
 				const int j0 = 64 * h + 32 * b;
-				const uint32_t at = tmem + T_G + s * ST_L + lanes + j0;
+				const uint32_t at = tmem + T_G + lanes + j0;
 				uint32_t out[32];
 				if (j0 > q * 32) {                                          // above the diagonal
 #pragma unroll
@@ -349,51 +349,71 @@ __global__ void __launch_bounds__(ST_THREADS, 1) ssm_tc_kernel(const __grid_cons
 			tmem_st_wait();
 			tc_fence_before();
 			mbar_arrive(bar_m);
+			// ---- what does not depend on the products: gates, inputs of this row ----
+			unsigned char *xt = input_tile(c), *own = xt + row * 128;
+			auto unit = [&](int r, int u) { return ((4 * h + u) ^ (r & 7)) * 16; };
+#pragma unroll
+			for (int i = 0; i < 4; ++i) asm volatile("" : "+r"(z[i].x), "+r"(z[i].y), "+r"(z[i].z), "+r"(z[i].w));      // not to be waited for any earlier
+			uint4 x[4];
+			float gate[32];
+			if (cols) {
+#pragma unroll
+				for (int u = 0; u < 4; ++u) {
+					x[u] = *reinterpret_cast<const uint4 *>(own + unit(row, u));
+					const uint32_t zs[4] = {z[u].x, z[u].y, z[u].z, z[u].w};
+#pragma unroll
+					for (int j = 0; j < 4; ++j) {
+						gate[8 * u + 2 * j] = silu_fast(__uint_as_float(zs[j] << 16));
+						gate[8 * u + 2 * j + 1] = silu_fast(__uint_as_float(zs[j] & 0xFFFF0000u));
+					}
+				}
+			}
+			if (c + 1 < n) {
+				if (!(ok = wait_warp(bar_full + 8 * (s ^ 1), (c + 1) >> 1)) || !(ok = wait_warp(bar_u, c))) break;
+				tc_fence_after();
+				prepare(c + 1);
+			}
 			// ---- y ----
 			if (!(ok = wait_warp(bar_y, c))) break;
 			tc_fence_after();
 			if (cols) {
 				const float e = ex2(si + si_lo);
-				unsigned char *own = xt + row * 128;
-				auto unit = [&](int r, int u) { return ((4 * h + u) ^ (r & 7)) * 16; };
-				uint4 x[4];
-#pragma unroll
-				for (int u = 0; u < 4; ++u) x[u] = *reinterpret_cast<const uint4 *>(own + unit(row, u));
-				__syncwarp();
-#pragma unroll
-				for (int i = 0; i < 4; ++i) *reinterpret_cast<uint4 *>(xt + (cr + 8 * i) * 128 + unit(cr + 8 * i, cu)) = z[i];
-				__syncwarp();
+				const uint32_t yi = tmem + T_YI + s * 2 * ST_P + lanes + 32 * h, ya = tmem + T_YA + lanes + 32 * h;
 #pragma unroll
 				for (int b = 0; b < 2; ++b) {
-					float y0[16], y1[16], ya[16];
-					tmem_ld16(tmem + T_YI + lanes + 32 * h + 16 * b, y0);
-					tmem_ld16(tmem + T_YI + ST_P + lanes + 32 * h + 16 * b, y1);
-					tmem_ld16(tmem + T_YA + lanes + 32 * h + 16 * b, ya);
+					float y0[16], y1[16], y2[16];
+					tmem_ld16(yi + 16 * b, y0);
+					tmem_ld16(yi + ST_P + 16 * b, y1);
+					tmem_ld16(ya + 16 * b, y2);
 					tmem_ld_wait();
 					tmem_settle(y0);
 					tmem_settle(y1);
-					tmem_settle(ya);
+					tmem_settle(y2);
 #pragma unroll
 					for (int u = 0; u < 2; ++u) {
-						uint4 *at = reinterpret_cast<uint4 *>(own + unit(row, 2 * b + u));
-						const uint4 zv = *at, xv = x[2 * b + u];
-						const uint32_t zs[4] = {zv.x, zv.y, zv.z, zv.w}, xs[4] = {xv.x, xv.y, xv.z, xv.w};
+						const uint4 xv = x[2 * b + u];
+						const uint32_t xs[4] = {xv.x, xv.y, xv.z, xv.w};
 						uint32_t o[4];
 #pragma unroll
 						for (int j = 0; j < 4; ++j) {
 							const int i = 8 * u + 2 * j;
-							const float a0 = fmaf(d, __uint_as_float(xs[j] << 16), fmaf(e, y0[i] + y1[i], ya[i]));
-							const float a1 = fmaf(d, __uint_as_float(xs[j] & 0xFFFF0000u), fmaf(e, y0[i + 1] + y1[i + 1], ya[i + 1]));
-							o[j] = pack_bf16(a0 * silu_fast(__uint_as_float(zs[j] << 16)), a1 * silu_fast(__uint_as_float(zs[j] & 0xFFFF0000u)));
+							const float a0 = fmaf(d, __uint_as_float(xs[j] << 16), fmaf(e, y0[i] + y1[i], y2[i]));
+							const float a1 = fmaf(d, __uint_as_float(xs[j] & 0xFFFF0000u), fmaf(e, y0[i + 1] + y1[i + 1], y2[i + 1]));
+							o[j] = pack_bf16(a0, a1);
 						}
-						*at = make_uint4(o[0], o[1], o[2], o[3]);
+						*reinterpret_cast<uint4 *>(own + unit(row, 2 * b + u)) = make_uint4(o[0], o[1], o[2], o[3]);
 					}
 				}
 				__syncwarp();
 #pragma unroll
-				for (int i = 0; i < 4; ++i)
-					if (ccol && t0 + cr + 8 * i < T)
-						*reinterpret_cast<uint4 *>(og + (size_t)(t0 + cr + 8 * i) * p.out_ld) = *reinterpret_cast<const uint4 *>(xt + (cr + 8 * i) * 128 + unit(cr + 8 * i, cu));
+				for (int i = 0; i < 4; ++i) {
+					const uint4 yv = *reinterpret_cast<const uint4 *>(xt + (cr + 8 * i) * 128 + unit(cr + 8 * i, cu));
+					const uint32_t ys[4] = {yv.x, yv.y, yv.z, yv.w};
+					uint32_t o[4];
+#pragma unroll
+					for (int j = 0; j < 4; ++j) o[j] = pack_bf16(__uint_as_float(ys[j] << 16) * gate[8 * i + 2 * j], __uint_as_float(ys[j] & 0xFFFF0000u) * gate[8 * i + 2 * j + 1]);
+					if (ccol && t0 + cr + 8 * i < T) *reinterpret_cast<uint4 *>(og + (size_t)(t0 + cr + 8 * i) * p.out_ld) = make_uint4(o[0], o[1], o[2], o[3]);
+				}
 				fence_proxy_async();                          // the tile is written by a copy next
 			}
 			tc_fence_before();
