@@ -1250,8 +1250,8 @@ def lifinex_kernels(G, engine, hbm: float, tflops: float, ctx: int = PROMPT, t: 
 			record('prompt rows (residual, norm)', graph_us([lambda: prepare_rows(st, ctl, bf, True, att.mixer_norm)] * 4), t * W * (4 + 4 + 4 + 2))
 		# ---- attention ----
 		mx, s = att.mixer, att.mixer.spec
-		raw = torch.randn((M, mx.w_in.shape[0]), device=dev)
-		gemm('attention in-projection', mx.w_in, epilogue(_dense.EPI_F32, raw), att.mixer_norm)
+		raw = torch.randn((M, mx.w_in.shape[0]), device=dev).to(torch.float32 if decode else bf)
+		gemm('attention in-projection', mx.w_in, epilogue(_dense.EPI_F32 if decode else _dense.EPI_T, raw), att.mixer_norm)
 		n = max(2, min(80, int(320e6 / (ctx * s.kv_heads * (s.maps * mx.D + mx.V) * 2)))) if decode else 2
 		caches = [{k: torch.randn_like(v.float()).to(bf) for k, v in StaticCache([s.cache_layout(engine.max_seq)], 1, bf, dev)[0].items()} for _ in range(n)]
 		o = torch.empty((M, s.heads * mx.V), dtype=bf, device=dev)

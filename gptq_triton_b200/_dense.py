@@ -52,7 +52,7 @@ class LatentPrefill(ctypes.Structure):
 class Gqa(ctypes.Structure):
 	_fields_ = [(n, _I) for n in ('M', 'rows_per_seq', 'heads', 'kv_heads', 'maps', 'dim', 'vdim', 'dim_true', 'vdim_true', 'max_seq', 'splits')] + [
 		(n, c_float) for n in ('scale', 'cap', 'eps', 'lambda_', 'out_mul', 'bound')] + [
-		('out_norm', _I), ('pos', _P), ('raw', _P), ('raw_ld', c_int64), ('q_norm', _P), ('k_norm', _P), ('k_cache', _P), ('v_cache', _P), ('q_hi', _P), ('q_lo', _P),
+		('out_norm', _I), ('pos', _P), ('raw', _P), ('raw_t', _I), ('raw_ld', c_int64), ('q_norm', _P), ('k_norm', _P), ('k_cache', _P), ('v_cache', _P), ('q_hi', _P), ('q_lo', _P),
 		('q_f32', _P), ('part_ml', _P), ('part_acc', _P), ('out', _P), ('out_ld', c_int64), ('status', _P)]
 
 

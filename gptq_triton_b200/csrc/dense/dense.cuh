@@ -158,6 +158,36 @@ __device__ void norm_parts(const RowPrep &p, const S *x, T *dst, float *inv) {
 	const int shares = p.fin_groups >= DN_WARPS ? 1 : DN_WARPS / p.fin_groups;
 	const bool quads = n % 4 == 0;                      // parts are whole groups of four entries (of the padded row, which is aligned)
 	const int per = quads ? ((n >> 2) + shares - 1) / shares * 4 : (n + shares - 1) / shares;
+	constexpr int KEEP = 8;                             // units of a share that a lane keeps in registers
+	if (quads && p.fin_groups * shares == DN_WARPS && per <= KEEP * 128) {
+		const int g = warp / shares, c0 = g * n + (warp - g * shares) * per, c1 = min(c0 + per, (g + 1) * n);
+		float4 v[KEEP];
+		float s = 0.f;
+#pragma unroll
+		for (int i = 0; i < KEEP; ++i) {
+			const int c = c0 + 4 * (lane + 32 * i);
+			v[i] = c < c1 ? Elem<S>::ldcg4(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+			s = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, s))));
+		}
+		s = warp_sum(s);
+		if (shares > 1) {
+			if (lane == 0) inv[warp] = s;
+			__syncthreads();
+			s = 0.f;
+			for (int i = 0; i < shares; ++i) s += inv[g * shares + i];
+		}
+		const float f = 1.f / sqrtf(s / (float)n + p.eps);
+#pragma unroll
+		for (int i = 0; i < KEEP; ++i) {
+			const int c = c0 + 4 * (lane + 32 * i);
+			if (c < c1) {
+				const float4 w = p.fin_w ? __ldg(reinterpret_cast<const float4 *>(p.fin_w + c)) : make_float4(1.f, 1.f, 1.f, 1.f);
+				Elem<T>::store4(dst + c, make_float4(v[i].x * f * w.x, v[i].y * f * w.y, v[i].z * f * w.z, v[i].w * f * w.w));
+			}
+		}
+		for (int c = p.width + tid; c < p.ld; c += DN_THREADS) Elem<T>::store(dst + c, 0.f);
+		return;
+	}
 	for (int i = warp; i < p.fin_groups * shares; i += DN_WARPS) {
 		const int g = i / shares, c0 = (i - g * shares) * per, c1 = min(c0 + per, n);
 		float s = 0.f;
@@ -497,8 +527,31 @@ int dense_rows_launch(const RowPrep &p, int M, void *h, long long ldh, int dtype
 int dn_sm_count();
 int dn_smem_opt_in(const void *kernel, size_t bytes);
 
+// ---- clusters: barriers, and stores into another CTA's shared memory -------------------------------------------------------------
+__device__ __forceinline__ uint32_t cluster_rank() {
+	uint32_t r;
+	asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
+	return r;
+}
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+__device__ __forceinline__ uint32_t cluster_map(uint32_t addr, uint32_t rank) {
+	uint32_t r;
+	asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
+	return r;
+}
+__device__ __forceinline__ void cluster_store2(uint32_t addr, float a, float b) {
+	asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(addr), "f"(a), "f"(b) : "memory");
+}
+__device__ __forceinline__ void cluster_store4(uint32_t addr, float a, float b, float c, float d) {
+	asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "f"(a), "f"(b), "f"(c), "f"(d) : "memory");
+}
+
+// cluster: CTAs per cluster; carveout: percentage of an SM's memory that is asked for as shared memory, or -1 (the driver's choice).
+// In a chain of dependent launches an SM never falls idle, so it keeps the largest split that a kernel of the chain asked for, and the
+// projections behind it lose the L1 that their loads in flight need: kernels of a decode step ask for no more than they use.
 template <typename... KArgs, typename... Args>
-static int dn_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args &&...args) {
+static int dn_launch_as(int cluster, int carveout, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args &&...args) {
 	if (smem > 16 * 1024)          // static shared memory comes on top (at most 32 KB)
 		if (int rc = dn_smem_opt_in(reinterpret_cast<const void *>(kernel), smem)) return rc;
 	cudaLaunchConfig_t cfg = {};
@@ -506,12 +559,27 @@ static int dn_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t sme
 	cfg.blockDim = block;
 	cfg.dynamicSmemBytes = smem;
 	cfg.stream = stream;
-	cudaLaunchAttribute attr[1];
+	cudaLaunchAttribute attr[3];
 	attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
 	attr[0].val.programmaticStreamSerializationAllowed = 1;
 	cfg.attrs = attr;
 	cfg.numAttrs = 1;
+	if (cluster > 1) {
+		cudaLaunchAttribute &a = attr[cfg.numAttrs++];
+		a.id = cudaLaunchAttributeClusterDimension;
+		a.val.clusterDim.x = cluster;
+		a.val.clusterDim.y = a.val.clusterDim.z = 1;
+	}
+	if (carveout >= 0) {
+		cudaLaunchAttribute &a = attr[cfg.numAttrs++];
+		a.id = cudaLaunchAttributePreferredSharedMemoryCarveout;
+		a.val.sharedMemCarveout = carveout;
+	}
 	return cuda_status(cudaLaunchKernelEx(&cfg, kernel, std::forward<Args>(args)...));
 }
 
+template <typename... KArgs, typename... Args>
+static int dn_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args &&...args) {
+	return dn_launch_as(1, -1, kernel, grid, block, smem, stream, std::forward<Args>(args)...);
+}
 }   // namespace gptq

@@ -5,6 +5,8 @@
 // are the A operand of mma.m16n8k16 and the activations the B operand.  A dot product does not care about the order of k, so
 // lane (gid, tig) feeds the eight consecutive k that its 16-byte loads deliver for rows gid and gid + 8 and the same eight k
 // of activation row gid: two MMAs per pair of loads, no shuffle.  fp32: the same layout on the FMA units.
+// Few tiles (a narrow projection) leave most SMs idle: then a cluster of CTAs shares a tile's K, the partial sums meet in the first
+// CTA's shared memory.
 // The prologue optionally prepares the rows itself (embedding lookup, residual, norm), the epilogue applies what
 // follows the projection (rotary queries / raw latent / gates, act(gate) * up, scaled logits with the greedy choice).
 #include <algorithm>
@@ -15,32 +17,36 @@ namespace gptq {
 
 namespace {
 
-constexpr int SK_M = 8, SK_U = 4, SK_REDLD = 17;
+constexpr int SK_M = 8, SK_U = 4, SK_REDLD = 17, SK_PARTS = 8;
 constexpr size_t SK_STATIC = (2 * DN_WARPS * SK_M * SK_REDLD + RP_SMEM) * sizeof(float) + 64;
 constexpr size_t SK_SMEM_MAX = 227 * 1024 - SK_STATIC - 1024;
 
-template <typename T>
-__global__ void __launch_bounds__(DN_THREADS, 2) dense_skinny_kernel(const DenseArgs p) {
+template <typename T, bool SPLIT>
+__global__ void __launch_bounds__(DN_THREADS, 2) dense_skinny_kernel(const DenseArgs p, int kparts) {
 	constexpr int E = 16 / sizeof(T);            // elements per 16-byte load
 	constexpr int STEP = 4 * E;                  // k per step of a warp
 	extern __shared__ __align__(16) unsigned char sk_smem[];
 	__shared__ float s_red[2][DN_WARPS][SK_M][SK_REDLD];
 	__shared__ float s_norm[RP_SMEM];
 	__shared__ int s_last;
+	__shared__ float2 s_part[SPLIT ? SK_PARTS : 1][SPLIT ? 8 * SK_M : 1];
+	if (SPLIT) cluster_arrive();                 // (every CTA of the cluster runs before its shared memory is written)
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
 	const int xs = p.K * (int)sizeof(T) + 16;    // bytes per staged row
-	const int nsteps = (p.K + STEP - 1) / STEP, spw = (nsteps + DN_WARPS - 1) / DN_WARPS;
-	const int s0 = warp * spw, s1 = min(s0 + spw, nsteps);
+	const int rank = SPLIT ? (int)cluster_rank() : 0, tile0 = SPLIT ? (int)blockIdx.x / kparts : (int)blockIdx.x, stride = SPLIT ? (int)gridDim.x / kparts : (int)gridDim.x;
+	const int slots = DN_WARPS * (SPLIT ? kparts : 1);
+	const int nsteps = (p.K + STEP - 1) / STEP, spw = (nsteps + slots - 1) / slots;
+	const int s0 = min((rank * DN_WARPS + warp) * spw, nsteps), s1 = min(s0 + spw, nsteps);
 	const int nbatch = (spw + SK_U - 1) / SK_U;
 	const int ntiles = (p.N + 15) >> 4;
-	const int mytiles = (ntiles - (int)blockIdx.x + (int)gridDim.x - 1) / (int)gridDim.x;
+	const int mytiles = (ntiles - tile0 + stride - 1) / stride;          // (SPLIT: one)
 	const int total = mytiles * nbatch;
 	const T *w = reinterpret_cast<const T *>(p.w);
 
 	uint4 wa[2][SK_U], wb[2][SK_U];
 	auto load = [&](int it, uint4 (&a)[SK_U], uint4 (&b)[SK_U]) {
 		const int ti = it / nbatch, bi = it - ti * nbatch;
-		const int row = ((int)blockIdx.x + ti * (int)gridDim.x) * 16 + gid;
+		const int row = (tile0 + ti * stride) * 16 + gid;
 		const T *pa = w + (size_t)min(row, p.N - 1) * p.ldw, *pb = w + (size_t)min(row + 8, p.N - 1) * p.ldw;
 #pragma unroll
 		for (int u = 0; u < SK_U; ++u) {
@@ -81,6 +87,19 @@ __global__ void __launch_bounds__(DN_THREADS, 2) dense_skinny_kernel(const Dense
 	const bool live = gid < p.M;
 	unsigned long long best = 0ull;              // LOGITS: running candidate of thread (m = tid / 8)
 
+	float part_a = 0.f, part_b = 0.f;            // SPLIT: this CTA's share of the results of threads below 8 M
+	auto finish = [&](int m, int j, int tile, float va, float vb) {
+		if (p.e.mode == DENSE_EPI_GATED) {
+			Elem<T>::store(reinterpret_cast<T *>(p.e.out) + (size_t)m * p.e.ldo + tile * 8 + j, activation(p.e.act, va) * vb);
+			return;
+		}
+		const int n = tile * 16 + 2 * j;
+		epi_pair<T>(p.e, m, n, va, vb);
+		if (p.e.mode == DENSE_EPI_LOGITS) {
+			if (n < p.N) best = max(best, argmax_key(va * p.e.scale, n));
+			if (n + 1 < p.N) best = max(best, argmax_key(vb * p.e.scale, n + 1));
+		}
+	};
 	auto compute = [&](int it, uint4 (&a)[SK_U], uint4 (&b)[SK_U]) {
 		const int ti = it / nbatch, bi = it - ti * nbatch;
 #pragma unroll
@@ -133,7 +152,7 @@ __global__ void __launch_bounds__(DN_THREADS, 2) dense_skinny_kernel(const Dense
 		}
 		__syncthreads();                         // the buffer is written again two tiles later, behind the next tile's barrier
 		if (tid < 8 * p.M) {
-			const int m = tid >> 3, j = tid & 7, tile = (int)blockIdx.x + ti * (int)gridDim.x;
+			const int m = tid >> 3, j = tid & 7, tile = tile0 + ti * stride;
 			const bool gated = p.e.mode == DENSE_EPI_GATED;
 			const int ra = gated ? j : 2 * j, rb = gated ? j + 8 : 2 * j + 1;
 			float va = 0.f, vb = 0.f;
@@ -142,15 +161,11 @@ __global__ void __launch_bounds__(DN_THREADS, 2) dense_skinny_kernel(const Dense
 				va += red[i][m][ra];
 				vb += red[i][m][rb];
 			}
-			if (gated) {
-				Elem<T>::store(reinterpret_cast<T *>(p.e.out) + (size_t)m * p.e.ldo + tile * 8 + j, activation(p.e.act, va) * vb);
+			if (SPLIT) {
+				part_a = va;
+				part_b = vb;
 			} else {
-				const int n = tile * 16 + 2 * j;
-				epi_pair<T>(p.e, m, n, va, vb);
-				if (p.e.mode == DENSE_EPI_LOGITS) {
-					if (n < p.N) best = max(best, argmax_key(va * p.e.scale, n));
-					if (n + 1 < p.N) best = max(best, argmax_key(vb * p.e.scale, n + 1));
-				}
+				finish(m, j, tile, va, vb);
 			}
 		}
 	};
@@ -162,6 +177,23 @@ __global__ void __launch_bounds__(DN_THREADS, 2) dense_skinny_kernel(const Dense
 		if (it + 1 < total) compute(it + 1, wa[1], wb[1]);
 	}
 
+	if (SPLIT) {
+		__syncwarp();
+		cluster_wait();
+		if (tid < 8 * p.M) cluster_store2(cluster_map(smem_u32(&s_part[rank][tid]), 0), part_a, part_b);
+		__syncwarp();
+		cluster_arrive();
+		cluster_wait();
+		if (rank == 0 && tid < 8 * p.M) {
+			float va = 0.f, vb = 0.f;
+			for (int i = 0; i < kparts; ++i) {
+				va += s_part[i][tid].x;
+				vb += s_part[i][tid].y;
+			}
+			finish(tid >> 3, tid & 7, tile0, va, vb);
+		}
+		return;
+	}
 	if (p.e.mode != DENSE_EPI_LOGITS || !p.e.best) return;
 	// ---- greedy choice: one candidate per CTA and row, the last CTA writes token and position ----------------------------
 	if (tid < 8 * SK_M) {                        // whole warps
@@ -188,8 +220,12 @@ template <typename T>
 int launch(const DenseArgs &a, cudaStream_t stream) {
 	const size_t smem = (size_t)a.M * ((size_t)a.K * sizeof(T) + 16);
 	const int ntiles = (a.N + 15) / 16, slots = dn_sm_count() * (smem + SK_STATIC > 110 * 1024 ? 1 : 2);
+	// few tiles: a cluster per tile, as long as every warp of it has a step of K
+	int kparts = SK_PARTS;
+	while (kparts > 1 && (ntiles * kparts > dn_sm_count() || a.K < kparts * DN_WARPS * 64 / (int)sizeof(T))) kparts >>= 1;
+	if (kparts > 1 && !a.e.best && smem <= 160 * 1024) return dn_launch_as(kparts, -1, dense_skinny_kernel<T, true>, dim3(ntiles * kparts), dim3(DN_THREADS), smem, stream, a, kparts);
 	const int waves = (ntiles + slots - 1) / slots;
-	return dn_launch(dense_skinny_kernel<T>, dim3((ntiles + waves - 1) / waves), dim3(DN_THREADS), smem, stream, a);
+	return dn_launch(dense_skinny_kernel<T, false>, dim3((ntiles + waves - 1) / waves), dim3(DN_THREADS), smem, stream, a, 1);
 }
 
 }   // namespace

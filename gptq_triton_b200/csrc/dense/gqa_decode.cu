@@ -19,56 +19,58 @@ namespace {
 constexpr int GQ_V = 4;                  // float4 units of a head vector per lane: dim, vdim <= 512
 constexpr int GQ_SPLITS = 64;
 
-// ---- norms and cache rows: a warp per head vector ------------------------------------------------------------------------
-template <typename T>
+// ---- norms and cache rows: LANES lanes per head vector, four entries per lane and unit ---------------------------------------------
+// R: type of the raw rows (fp32, or bf16 for prompts), T: of the cache
+template <typename R, typename T, int LANES, int UNITS>
 __global__ void __launch_bounds__(DN_THREADS) gqa_append_kernel(const GqaArgs p) {
-	const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+	constexpr int PER_CTA = DN_THREADS / LANES;
 	const int nq = p.heads * p.maps, nk = p.kv_heads * p.maps, rows = nq + nk + p.kv_heads;
-	const long long id = (long long)blockIdx.x * DN_WARPS + warp;
-	pdl_wait();
-	pdl_trigger();
+	const long long id = (long long)blockIdx.x * PER_CTA + threadIdx.x / LANES;
+	const int lane = threadIdx.x % LANES;
 	const int m = (int)(id / rows), r = (int)(id - (long long)m * rows);
-	if (m >= p.M) return;
-	const int pos = __ldcg(p.pos + m), seq = m / p.rows_per_seq;
-	if (pos < 0 || pos >= p.max_seq) {            // a position outside the cache is dropped
-		if (lane == 0) atomicExch(p.status, DN_BAD_POSITION);
-		return;
-	}
-	const float *raw = reinterpret_cast<const float *>(p.raw) + (size_t)m * p.raw_ld;
 	const bool value = r >= nq + nk, query = r < nq;
 	const int n = value ? p.vdim : p.dim;
-	const float *src = raw + (value ? (nq + nk) * p.dim + (r - nq - nk) * p.vdim : r * p.dim);
 	const float *gain = value ? nullptr : query ? p.q_norm : p.k_norm;
-	float4 v[GQ_V];
+	float4 g[UNITS];
+#pragma unroll
+	for (int i = 0; i < UNITS; ++i) {
+		const int c = (i * LANES + lane) * 4;
+		g[i] = gain && c < n ? __ldg(reinterpret_cast<const float4 *>(gain + c)) : make_float4(1.f, 1.f, 1.f, 1.f);
+	}
+	pdl_wait();
+	pdl_trigger();
+	const int pos = m < p.M ? __ldcg(p.pos + m) : -1, seq = m / p.rows_per_seq;
+	const bool live = pos >= 0 && pos < p.max_seq;
+	if (m < p.M && !live && lane == 0) atomicExch(p.status, DN_BAD_POSITION);      // a position outside the cache is dropped
+	const R *src = reinterpret_cast<const R *>(p.raw) + (size_t)m * p.raw_ld + (value ? (nq + nk) * p.dim + (r - nq - nk) * p.vdim : r * p.dim);
+	float4 v[UNITS];
 	float s = 0.f;
 #pragma unroll
-	for (int i = 0; i < GQ_V; ++i) {
-		const int c = (i * 32 + lane) * 4;
-		if (i * 128 < n) {
-			v[i] = c < n ? __ldcg(reinterpret_cast<const float4 *>(src + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
-			s = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, s))));
-		}
+	for (int i = 0; i < UNITS; ++i) {
+		const int c = (i * LANES + lane) * 4;
+		v[i] = live && c < n ? Elem<R>::ldcg4(src + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+		s = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, s))));
 	}
-	float f = 1.f;
-	if (gain) f = 1.f / sqrtf(warp_sum(s) / (float)p.dim_true + p.eps);
+#pragma unroll
+	for (int d = LANES / 2; d > 0; d >>= 1) s += __shfl_xor_sync(0xffffffffu, s, d);
+	if (!live) return;
+	float f = gain ? 1.f / sqrtf(s / (float)p.dim_true + p.eps) : 1.f;
 	if (query) f *= gqa_query_factor(p);
 	const size_t cache_row = (size_t)seq * p.max_seq + pos;
 	T *dst = query ? nullptr : value ? reinterpret_cast<T *>(p.v_cache) + (cache_row * p.kv_heads + (r - nq - nk)) * p.vdim
 									 : reinterpret_cast<T *>(p.k_cache) + (cache_row * nk + (r - nq)) * p.dim;
 	const size_t qo = ((size_t)m * nq + r) * p.dim;
 #pragma unroll
-	for (int i = 0; i < GQ_V; ++i) {
-		const int c = (i * 32 + lane) * 4;
+	for (int i = 0; i < UNITS; ++i) {
+		const int c = (i * LANES + lane) * 4;
 		if (c < n) {
-			const float4 g = gain ? __ldg(reinterpret_cast<const float4 *>(gain + c)) : make_float4(1.f, 1.f, 1.f, 1.f);
-			const float4 o = make_float4(v[i].x * f * g.x, v[i].y * f * g.y, v[i].z * f * g.z, v[i].w * f * g.w);
+			const float4 o = make_float4(v[i].x * f * g[i].x, v[i].y * f * g[i].y, v[i].z * f * g[i].z, v[i].w * f * g[i].w);
 			if (!query) {
 				Elem<T>::store4(dst + c, o);
 			} else if (sizeof(T) == 4) {
 				*reinterpret_cast<float4 *>(p.q_f32 + qo + c) = o;
 			} else {
-				bf16 *hi = reinterpret_cast<bf16 *>(p.q_hi) + qo + c;
-				Elem<bf16>::store4(hi, o);
+				Elem<bf16>::store4(reinterpret_cast<bf16 *>(p.q_hi) + qo + c, o);
 				if (p.q_lo) {
 					auto rest = [](float a) { return a - __bfloat162float(__float2bfloat16_rn(a)); };
 					Elem<bf16>::store4(reinterpret_cast<bf16 *>(p.q_lo) + qo + c, make_float4(rest(o.x), rest(o.y), rest(o.z), rest(o.w)));
@@ -81,6 +83,7 @@ __global__ void __launch_bounds__(DN_THREADS) gqa_append_kernel(const GqaArgs p)
 // ---- attention over a range of keys, bf16 -----------------------------------------------------------------------------
 constexpr int GA_KEYS = 32;              // keys per tile
 constexpr int GA_ROWS = 16;              // (map, query head) rows per CTA
+constexpr size_t GA_STATIC = 8 * 1024;   // more than its static shared memory and what the system keeps
 
 struct GaPlan {
 	int kd, krow, vrow, stages;          // key entries; bytes of a staged key / value row (padded against bank conflicts)
@@ -405,10 +408,20 @@ __global__ void __launch_bounds__(DN_THREADS) gqa_merge_kernel(const GqaArgs p) 
 
 }   // namespace
 
-int gqa_append_launch(const GqaArgs &p, int dtype, cudaStream_t stream) {
+template <typename R, typename T>
+static int append_launch(const GqaArgs &p, cudaStream_t stream) {
 	const long long rows = (long long)p.M * (p.heads * p.maps + p.kv_heads * (p.maps + 1));
-	const dim3 grid((unsigned)((rows + DN_WARPS - 1) / DN_WARPS));
-	return dtype ? dn_launch(gqa_append_kernel<float>, grid, dim3(DN_THREADS), 0, stream, p) : dn_launch(gqa_append_kernel<bf16>, grid, dim3(DN_THREADS), 0, stream, p);
+	const int widest = std::max(p.dim, p.vdim);
+	auto go = [&](auto kernel, int lanes) { return dn_launch(kernel, dim3((unsigned)((rows * lanes + DN_THREADS - 1) / DN_THREADS)), dim3(DN_THREADS), 0, stream, p); };
+	if (widest <= 64) return go(gqa_append_kernel<R, T, 16, 1>, 16);
+	if (widest <= 128) return go(gqa_append_kernel<R, T, 16, 2>, 16);
+	if (widest <= 256) return go(gqa_append_kernel<R, T, 32, 2>, 32);
+	return go(gqa_append_kernel<R, T, 32, GQ_V>, 32);
+}
+
+int gqa_append_launch(const GqaArgs &p, int dtype, cudaStream_t stream) {
+	if (dtype) return append_launch<float, float>(p, stream);
+	return p.raw_t ? append_launch<bf16, bf16>(p, stream) : append_launch<float, bf16>(p, stream);
 }
 
 bool gqa_attend_ok(int maps, int dim, int vdim) { return dim <= GQ_V * 128 && vdim <= GQ_V * 128 && ga_plan(maps, dim, vdim).smem <= 220 * 1024; }
@@ -424,10 +437,11 @@ int gqa_attend_launch(const GqaArgs &p, int dtype, cudaStream_t stream) {
 	const GaPlan g = ga_plan(p.maps, p.dim, p.vdim);
 	const int rtiles = (p.heads / p.kv_heads * p.maps + GA_ROWS - 1) / GA_ROWS;
 	const dim3 grid(p.splits, p.kv_heads * rtiles, p.M), block(DN_THREADS);
-	if (p.vdim <= 64) return dn_launch(gqa_attend_kernel<1>, grid, block, g.smem, stream, p);
-	if (p.vdim <= 128) return dn_launch(gqa_attend_kernel<2>, grid, block, g.smem, stream, p);
-	if (p.vdim <= 256) return dn_launch(gqa_attend_kernel<4>, grid, block, g.smem, stream, p);
-	return dn_launch(gqa_attend_kernel<8>, grid, block, g.smem, stream, p);
+	auto go = [&](auto kernel) { return dn_launch_as(1, (int)((g.smem + GA_STATIC) * 100 / (228 * 1024)) + 1, kernel, grid, block, g.smem, stream, p); };
+	if (p.vdim <= 64) return go(gqa_attend_kernel<1>);
+	if (p.vdim <= 128) return go(gqa_attend_kernel<2>);
+	if (p.vdim <= 256) return go(gqa_attend_kernel<4>);
+	return go(gqa_attend_kernel<8>);
 }
 
 int gqa_merge_launch(const GqaArgs &p, int dtype, cudaStream_t stream) {

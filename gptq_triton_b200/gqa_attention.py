@@ -68,12 +68,12 @@ class GroupedAttention(nn.Module):
 		(residual stream x, sublayer output y), both fp32."""
 		s, dev, dt = self.spec, control.device, self.w_in.dtype
 		M, max_seq = stream.rows, cache['k'].shape[1]
-		raw = torch.empty((M, self.w_in.shape[0]), dtype=torch.float32, device=dev)
-		x = project_stream(stream, self.w_in, epilogue(_dense.EPI_F32, raw), control, final=norm)
+		maps = 0 if start is None or dt == torch.float32 or rows_per_seq <= DECODE_MAX_ROWS else _dense.lib().dense_gqa_prefill_maps(s.maps, self.D, self.V)
+		raw = torch.empty((M, self.w_in.shape[0]), dtype=dt if maps else torch.float32, device=dev)
+		x = project_stream(stream, self.w_in, epilogue(_dense.EPI_T if maps else _dense.EPI_F32, raw), control, final=norm)
 		a = self.arguments(raw, cache, pos, rows_per_seq, stream.eps, control)
 		lib, code, st = _dense.lib(), _dense.DTYPE_CODE[dt], stream_ptr(dev)
 		out = torch.empty((M, s.heads * self.V), dtype=dt, device=dev)
-		maps = 0 if start is None or dt == torch.float32 or rows_per_seq <= DECODE_MAX_ROWS else lib.dense_gqa_prefill_maps(s.maps, self.D, self.V)
 		if maps:
 			self._prompt(a, out, rows_per_seq, start, maps, cache)
 		else:
@@ -89,7 +89,7 @@ class GroupedAttention(nn.Module):
 		a.dim, a.vdim, a.dim_true, a.vdim_true, a.max_seq, a.splits = self.D, self.V, s.dim, s.vdim, cache['k'].shape[1], 1
 		a.scale, a.cap, a.eps, a.lambda_, a.bound = s.scale, s.softcap or 0.0, eps, self.lam, self.bound
 		a.out_norm, a.out_mul = int(s.maps == 2), 1.0 - s.diff if s.maps == 2 else 1.0
-		a.pos, a.raw, a.raw_ld, a.q_norm, a.k_norm = ptr(pos), ptr(raw), raw.stride(0), ptr(self.q_norm), ptr(self.k_norm)
+		a.pos, a.raw, a.raw_t, a.raw_ld, a.q_norm, a.k_norm = ptr(pos), ptr(raw), int(raw.dtype != torch.float32), raw.stride(0), ptr(self.q_norm), ptr(self.k_norm)
 		a.k_cache, a.v_cache, a.status = ptr(cache['k']), ptr(cache['v']), _dense.status_ptr(control)
 		return a
 

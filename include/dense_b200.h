@@ -147,7 +147,8 @@ typedef struct {
 	float bound;                       /* |q . k * scale / cap| is known to be at most this (0: nothing known); used by the prompt kernel */
 	int out_norm;
 	const int32_t *pos;                /* [M] */
-	const void *raw;                   /* [M, raw_ld] fp32 */
+	const void *raw;                   /* [M, raw_ld] fp32, or (raw_t) in the activation dtype */
+	int raw_t;
 	int64_t raw_ld;
 	const float *q_norm, *k_norm;      /* [dim] or NULL */
 	void *k_cache;                     /* [sequences, max_seq, kv_heads * maps * dim] */

@@ -44,7 +44,8 @@ def close(got, want, rel):
 # ---- the kernels alone ---------------------------------------------------------------------------------------------------
 
 @pytest.mark.parametrize('dtype', [F32, B16])
-@pytest.mark.parametrize('M,K,N', [(1, 48, 80), (2, 1040, 33), (5, 272, 528), (8, 2080, 16), (9, 64, 48), (130, 336, 515), (300, 1088, 272)])
+@pytest.mark.parametrize('M,K,N', [(1, 48, 80), (2, 1040, 33), (5, 272, 528), (8, 2080, 16), (9, 64, 48), (130, 336, 515), (300, 1088, 272),
+									 (1, 4112, 40), (3, 8208, 256), (6, 2064, 144), (1200, 2064, 200), (2500, 1040, 500), (9, 1040, 16)])
 def test_projection(control, dtype, M, K, N):
 	from gptq_triton_b200 import _dense
 	from gptq_triton_b200.dense import epilogue, linear, matmul
