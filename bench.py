@@ -710,6 +710,40 @@ def kernel_case(args):
 		torch.cuda.synchronize()
 		print(json.dumps({'kernel_case': args.kernel_case}))
 		return
+	if args.kernel_case in ('gqa-prefill', 'ssm-prefill', 'lifinex-decode'):
+		# 2048 tokens through the tensor-core kernels of the differential attention / the state-space recurrence alone, or decode steps
+		# of two layers (at most 2 GB on the device)
+		import ctypes
+		from gptq_triton_b200 import _dense
+		from gptq_triton_b200.cache import StaticCache
+		bf, t = torch.bfloat16, PROMPT
+		cfg = lifinex_config(G, 2, args.heads * 128, 11008 if args.kernel_case == 'lifinex-decode' else 256, vocab=2048)
+		e = G.LifinexEngine(G.synthetic_lifinex(cfg, device=dev), 1, PROMPT + 16, use_graph=False)
+		if args.kernel_case == 'lifinex-decode':
+			e.feed(torch.randint(0, cfg.vocab_size, (1, t), generator=torch.Generator().manual_seed(3)))
+			for _ in range(3):
+				e.step()
+		elif args.kernel_case == 'gqa-prefill':
+			mx, s = e.model.layers[0].mixer, cfg.layers[0].mixer
+			raw, o = torch.randn((t, mx.w_in.shape[0]), device=dev).to(bf), torch.empty((t, s.heads * mx.V), dtype=bf, device=dev)
+			pos = torch.arange(t, dtype=torch.int32, device=dev)
+			a = mx.arguments(raw, e.cache[0], pos, t, cfg.norm_eps, e.control)
+			keep = mx.buffers(a, o, 1)
+			_dense.check(_dense.lib().dense_gqa_append(ctypes.byref(a), 0, None), 'dense_gqa_append')
+			for _ in range(3):
+				_dense.check(_dense.lib().dense_gqa_prefill(ctypes.byref(a), 0, None), 'dense_gqa_prefill')
+		else:
+			mx, s = e.model.layers[1].mixer, cfg.layers[1].mixer
+			raw, steps = torch.randn((t, mx.dt_at), device=dev).to(bf), torch.randn((t, mx.w_in.shape[0] - mx.dt_at), device=dev)
+			o, pos = torch.empty((t, s.inner), dtype=bf, device=dev), torch.arange(t, dtype=torch.int32, device=dev)
+			a = mx.arguments(raw, steps, e.cache[1], pos, t, o, e.control)
+			keep = mx.portion_buffers(a, bf, True)
+			_dense.check(_dense.lib().dense_ssm_conv(ctypes.byref(a), 0, None), 'dense_ssm_conv')
+			for _ in range(3):
+				_dense.check(_dense.lib().dense_ssm_chunked(ctypes.byref(a), None), 'dense_ssm_chunked')
+		torch.cuda.synchronize()
+		print(json.dumps({'kernel_case': args.kernel_case}))
+		return
 	if args.kernel_case == 'chain':
 		# the persistent decode-step kernel on four layers of the 7B architecture after a 2048-token prompt (about 1 GB on
 		# the device): a few steps, nothing else; also prints the step time of both engines
@@ -1381,9 +1415,9 @@ def main():
 						 'differential attention and state-space layers beside befalix at equal sizes')
 	ap.add_argument('--case', default='', help='befalix, lifinex: sizes to run (2048, 4096, 8192), separated by commas')
 	ap.add_argument('--no-graph', action='store_true', help='do not capture the decode step in a CUDA graph')
-	ap.add_argument('--kernel-case', default=None, choices=['gateup', 'qkv', 'o', 'down', 'prefill', 'attn', 'lmhead', 'chain', 'qkvattn', 'latent-prefill', 'latent-decode'], help='profiling aid: run a few launches of one kernel and exit')
+	ap.add_argument('--kernel-case', default=None, choices=['gateup', 'qkv', 'o', 'down', 'prefill', 'attn', 'lmhead', 'chain', 'qkvattn', 'latent-prefill', 'latent-decode', 'gqa-prefill', 'ssm-prefill', 'lifinex-decode'], help='profiling aid: run a few launches of one kernel and exit')
 	ap.add_argument('--m', type=int, default=1, help='batch rows for --kernel-case')
-	ap.add_argument('--heads', type=int, default=32, help='heads for --kernel-case attn and latent-prefill')
+	ap.add_argument('--heads', type=int, default=32, help='heads for --kernel-case attn, latent-prefill and gqa-prefill')
 	args = ap.parse_args()
 	if args.kernel_case:
 		kernel_case(args)

@@ -65,7 +65,8 @@ class Ssm(ctypes.Structure):
 _SIGNATURES = {
 	'dense_version': (c_int, []),
 	'dense_last_cuda_error': (c_int, []),
-	'dense_matmul': (c_int, [_P, c_int64, _P, c_int64, _I, _I, _I, _I, _P, _P, _P, _P]),
+	'dense_matmul': (c_int, [_P, c_int64, _P, c_int64, _I, _I, _I, _I, _P, _P, _P, _P, _P]),
+	'dense_matmul_scratch': (c_int64, [_I, _I, _I, _I]),
 	'dense_decode_rows_ok': (c_int, [_I, _I, _I]),
 	'dense_prepare_rows': (c_int, [_P, _I, _P, c_int64, _I, _P]),
 	'dense_latent_splits': (c_int, [_I, _I, _I, _I]),

@@ -514,11 +514,14 @@ struct DenseArgs {
 	RowPrep rp;
 	DenseEpi e;
 	int *status;
+	float *ws;                       // scratch of a split K: [parts, M, N to 16], or NULL
+	int parts;
 };
 
 // launchers (dense_skinny.cu, dense_tc.cu, dense_simt.cu)
 int dense_skinny_launch(const DenseArgs &a, int dtype, cudaStream_t stream);
 bool dense_skinny_ok(int M, int K, int dtype);
+int dense_tc_parts(int M, int K, int N);
 int dense_tc_launch(const DenseArgs &a, cudaStream_t stream);
 int dense_simt_launch(const DenseArgs &a, cudaStream_t stream);
 
@@ -542,9 +545,6 @@ __device__ __forceinline__ uint32_t cluster_map(uint32_t addr, uint32_t rank) {
 }
 __device__ __forceinline__ void cluster_store2(uint32_t addr, float a, float b) {
 	asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(addr), "f"(a), "f"(b) : "memory");
-}
-__device__ __forceinline__ void cluster_store4(uint32_t addr, float a, float b, float c, float d) {
-	asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "f"(a), "f"(b), "f"(c), "f"(d) : "memory");
 }
 
 // cluster: CTAs per cluster; carveout: percentage of an SM's memory that is asked for as shared memory, or -1 (the driver's choice).

@@ -88,8 +88,8 @@ int dense_version(void) { return 100; }
 int dense_last_cuda_error(void) { return g_last_cuda_error; }
 int dense_decode_rows_ok(int M, int K, int dtype) { return dense_skinny_ok(M, K, dtype) ? 1 : 0; }
 
-int dense_matmul(const void *x, int64_t ldx, const void *w, int64_t ldw, int M, int K, int N, int dtype, const dense_rows_t *rows, const dense_epilogue_t *epi, int *status,
-				 void *stream) {
+int dense_matmul(const void *x, int64_t ldx, const void *w, int64_t ldw, int M, int K, int N, int dtype, const dense_rows_t *rows, const dense_epilogue_t *epi, float *scratch,
+				 int *status, void *stream) {
 	if (!w || !epi || !status || M < 0 || K < 16 || N < 1 || (dtype != 0 && dtype != 1) || (!rows && !x)) return GPTQ_ERR_INVALID;
 	if (M == 0) return GPTQ_OK;
 	if (K % 16) return GPTQ_ERR_SHAPE;
@@ -134,6 +134,8 @@ int dense_matmul(const void *x, int64_t ldx, const void *w, int64_t ldw, int M, 
 	a.N = N;
 	a.e = *epi;
 	a.status = status;
+	a.ws = scratch;
+	if (!aligned16(scratch)) return GPTQ_ERR_ALIGN;
 	if (rows) {
 		if (rows_bad(*rows, dtype) || rows->ld != K) return GPTQ_ERR_INVALID;
 		a.prep = 1;
@@ -143,6 +145,12 @@ int dense_matmul(const void *x, int64_t ldx, const void *w, int64_t ldw, int M, 
 	if (dense_skinny_ok(M, K, dtype)) return dense_skinny_launch(a, dtype, st);
 	if (rows || epi->best) return GPTQ_ERR_UNSUPPORTED;
 	return dtype ? dense_simt_launch(a, st) : dense_tc_launch(a, st);
+}
+
+int64_t dense_matmul_scratch(int M, int K, int N, int dtype) {
+	if (dtype || M < 1 || K < 16 || N < 1 || dense_skinny_ok(M, K, dtype)) return 0;
+	const int parts = dense_tc_parts(M, K, N);
+	return parts > 1 ? (int64_t)parts * M * ((N + 15) / 16 * 16) : 0;
 }
 
 int dense_prepare_rows(const dense_rows_t *rows, int M, void *h, int64_t ldh, int dtype, void *stream) {

@@ -220,8 +220,9 @@ template <typename T>
 int launch(const DenseArgs &a, cudaStream_t stream) {
 	const size_t smem = (size_t)a.M * ((size_t)a.K * sizeof(T) + 16);
 	const int ntiles = (a.N + 15) / 16, slots = dn_sm_count() * (smem + SK_STATIC > 110 * 1024 ? 1 : 2);
-	// few tiles: a cluster per tile, as long as every warp of it has a step of K
-	int kparts = SK_PARTS;
+	// few tiles with long rows: a cluster per tile, as long as every warp of it has a step of K (with shorter rows the launch of a
+	// cluster costs more than it saves)
+	int kparts = a.K * (int)sizeof(T) > 8192 ? SK_PARTS : 1;
 	while (kparts > 1 && (ntiles * kparts > dn_sm_count() || a.K < kparts * DN_WARPS * 64 / (int)sizeof(T))) kparts >>= 1;
 	if (kparts > 1 && !a.e.best && smem <= 160 * 1024) return dn_launch_as(kparts, -1, dense_skinny_kernel<T, true>, dim3(ntiles * kparts), dim3(DN_THREADS), smem, stream, a, kparts);
 	const int waves = (ntiles + slots - 1) / slots;

@@ -32,7 +32,7 @@ template <int BN> struct TdShape {
 	static constexpr uint32_t TMEM = 2 * BN < 32 ? 32 : 2 * BN;
 };
 
-template <int BN>
+template <int BN, bool SPLIT>
 __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_constant__ CUtensorMap tmx, const __grid_constant__ CUtensorMap tmw, const DenseArgs p,
 																 int mt, int nt) {
 	extern __shared__ unsigned char td_raw[];
@@ -45,7 +45,9 @@ __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_co
 	uint32_t *s_tmem = reinterpret_cast<uint32_t *>(bars + 2 * S + 4);
 	volatile int *s_abort = reinterpret_cast<volatile int *>(s_tmem + 1);
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-	const int nkb = (p.K + TD_BK - 1) / TD_BK, ntiles = mt * nt;
+	const int nkb = (p.K + TD_BK - 1) / TD_BK, parts = SPLIT ? p.parts : 1, ntiles = mt * nt * parts;
+	auto k_first = [&](int t) { return SPLIT ? t % parts * nkb / parts : 0; };          // (SPLIT: consecutive CTAs share a tile)
+	auto k_last = [&](int t) { return SPLIT ? (t % parts + 1) * nkb / parts : nkb; };
 
 	if (tid == 0) {
 		for (int s = 0; s < S; ++s) {
@@ -80,8 +82,8 @@ __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_co
 		if (lane == 0) {
 			int it = 0;
 			for (int t = blockIdx.x; t < ntiles && !*s_abort; t += gridDim.x) {
-				const int m0 = (t % mt) * TD_BM, n0 = (t / mt) * BN;
-				for (int kb = 0; kb < nkb; ++kb, ++it) {
+				const int tile = t / parts, m0 = (tile % mt) * TD_BM, n0 = (tile / mt) * BN;
+				for (int kb = k_first(t); kb < k_last(t); ++kb, ++it) {
 					const int s = it % S;
 					if (*s_abort || !mbar_wait_bounded(bar_empty + 8 * s, ((it / S) & 1) ^ 1, TD_SPIN)) { fail(); break; }
 					mbar_arrive_expect_tx(bar_full + 8 * s, Sh::STAGE);
@@ -100,14 +102,15 @@ __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_co
 				const int b = lt & 1;
 				if (!mbar_wait_bounded(bar_free + 8 * b, ((lt >> 1) & 1) ^ 1, TD_SPIN)) { fail(); break; }
 				tc_fence_after();
-				for (int kb = 0; kb < nkb; ++kb, ++it) {
+				const int k0 = k_first(t);
+				for (int kb = k0; kb < k_last(t); ++kb, ++it) {
 					const int s = it % S;
 					if (*s_abort || !mbar_wait_bounded(bar_full + 8 * s, (it / S) & 1, TD_SPIN)) { fail(); break; }
 					tc_fence_after();
 					const uint32_t a = smem_u32(smem + (size_t)s * Sh::STAGE), w = a + TD_A_BYTES;
 #pragma unroll
 					for (int k = 0; k < TD_BK / 16; ++k)
-						umma_f16(tmem + b * BN, smem_desc_sw128(a + k * 32), smem_desc_sw128(w + k * 32), IDESC, (kb > 0 || k > 0) ? 1u : 0u);
+						umma_f16(tmem + b * BN, smem_desc_sw128(a + k * 32), smem_desc_sw128(w + k * 32), IDESC, (kb > k0 || k > 0) ? 1u : 0u);
 					umma_commit(bar_empty + 8 * s);
 				}
 				umma_commit(bar_acc + 8 * b);
@@ -121,7 +124,7 @@ __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_co
 		int lt = 0;
 		bool ok = true;
 		for (int t = blockIdx.x; t < ntiles && ok; t += gridDim.x, ++lt) {
-			const int b = lt & 1, m = (t % mt) * TD_BM + q * 32 + lane, n0 = (t / mt) * BN;
+			const int tile = t / parts, b = lt & 1, m = (tile % mt) * TD_BM + q * 32 + lane, n0 = (tile / mt) * BN;
 			ok = !*s_abort && mbar_wait_bounded(bar_acc + 8 * b, (lt >> 1) & 1, TD_SPIN);
 			ok = __all_sync(0xffffffffu, ok);
 			if (!ok) {
@@ -138,7 +141,16 @@ __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_co
 				tmem_ld_wait();
 #pragma unroll
 				for (int i = 0; i < 16; ++i) asm volatile("" : "+f"(v[0][i]), "+f"(v[1][i]));
-				if (m < p.M) {
+				if (SPLIT) {
+					const int n16 = (p.N + 15) & ~15;
+					float *ws = p.ws + ((size_t)(t % parts) * p.M + m) * n16 + n0 + c;
+#pragma unroll
+					for (int h = 0; h < 2; ++h)
+						if (m < p.M && n0 + c + 16 * h < p.N) {
+							Elem<float>::store8(ws + 16 * h, v[h]);
+							Elem<float>::store8(ws + 16 * h + 8, v[h] + 8);
+						}
+				} else if (m < p.M) {
 					if (n0 + c < p.N) epi_16<bf16>(p.e, m, n0 + c, v[0]);
 					if (n0 + c + 16 < p.N) epi_16<bf16>(p.e, m, n0 + c + 16, v[1]);
 				}
@@ -152,142 +164,33 @@ __global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_kernel(const __grid_co
 	if (warp == 1) tmem_dealloc(tmem, Sh::TMEM);
 }
 
-// ---- narrow outputs: a cluster of CTAs shares the K range of one output tile -------------------------------------------------------
-// Every CTA accumulates its K blocks in its own tensor memory; then each gets a share of the tile's columns from all of them
-// through distributed shared memory (the ring's stages, idle by then), adds the parts in rank order and runs the epilogue.
-constexpr int TK_BN = 256, TK_STAGE = TD_A_BYTES + TK_BN * TD_BK * 2, TK_S = 4;
-constexpr size_t TK_SMEM = (size_t)TK_S * TK_STAGE + 2048;
-
-__global__ void __launch_bounds__(TD_THREADS, 1) dense_tc_cluster_kernel(const __grid_constant__ CUtensorMap tmx, const __grid_constant__ CUtensorMap tmw, const DenseArgs p,
-																		 int mt, int parts) {
-	extern __shared__ unsigned char tk_raw[];
-	constexpr uint32_t IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(TK_BN >> 3) << 17) | ((uint32_t)(TD_BM >> 4) << 24);
-	unsigned char *smem = tk_raw + ((1024u - (smem_u32(tk_raw) & 1023u)) & 1023u);
-	uint64_t *bars = reinterpret_cast<uint64_t *>(smem + (size_t)TK_S * TK_STAGE);
-	const uint32_t bar_full = smem_u32(bars), bar_empty = smem_u32(bars + TK_S), bar_acc = smem_u32(bars + 2 * TK_S);
-	uint32_t *s_tmem = reinterpret_cast<uint32_t *>(bars + 2 * TK_S + 1);
-	volatile int *s_abort = reinterpret_cast<volatile int *>(s_tmem + 1);
-	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rank = (int)cluster_rank(), tile = blockIdx.x / parts;
-	const int m0 = (tile % mt) * TD_BM, n0 = (tile / mt) * TK_BN;
-	const int nkb = (p.K + TD_BK - 1) / TD_BK, k_lo = rank * nkb / parts, n = (rank + 1) * nkb / parts - k_lo;      // (nkb >= parts)
-	if (tid == 0) {
-		for (int s = 0; s < TK_S; ++s) {
-			mbar_init(bar_full + 8 * s, 1);
-			mbar_init(bar_empty + 8 * s, 1);
-		}
-		mbar_init(bar_acc, 1);
-		*s_abort = 0;
-		fence_mbar_init();
-		tma_prefetch_desc(&tmx);
-		tma_prefetch_desc(&tmw);
-	}
-	if (warp == 1) {
-		tmem_alloc(smem_u32(s_tmem), TK_BN);
-		tmem_relinquish();
-	}
-	tc_fence_before();
-	__syncthreads();
-	tc_fence_after();
-	const uint32_t tmem = *s_tmem;
-	auto fail = [&]() {
-		*s_abort = 1;
-		atomicExch(p.status, 3);
-	};
+// ---- narrow outputs: the K range of a tile split over CTAs, fp32 parts in scratch memory, summed in order by a second kernel ---------
+__global__ void __launch_bounds__(DN_THREADS) dense_finish_kernel(const DenseArgs p, int n16) {
+	const int groups = n16 >> 4, i = blockIdx.x * DN_THREADS + threadIdx.x, m = i / groups, n = (i - m * groups) * 16;
 	pdl_wait();
 	pdl_trigger();
-	if (warp == 0) {
-		if (lane == 0) {
-			int it = 0;
-			for (; it < n; ++it) {
-				const int s = it % TK_S;
-				if (*s_abort || !mbar_wait_bounded(bar_empty + 8 * s, ((it / TK_S) & 1) ^ 1, TD_SPIN)) { fail(); break; }
-				mbar_arrive_expect_tx(bar_full + 8 * s, TK_STAGE);
-				unsigned char *st = smem + (size_t)s * TK_STAGE;
-				tma_load_2d(smem_u32(st), &tmx, (k_lo + it) * TD_BK, m0, bar_full + 8 * s);              // rows and columns outside are zero-filled
-				tma_load_2d(smem_u32(st + TD_A_BYTES), &tmw, (k_lo + it) * TD_BK, n0, bar_full + 8 * s);
-			}
-			for (int i = max(0, it - TK_S); i < it; ++i) mbar_wait_bounded(bar_full + 8 * (i % TK_S), (i / TK_S) & 1, TD_SPIN);
-		}
-		__syncwarp();
-	} else if (warp == 1) {
-		if (lane == 0) {
-			for (int it = 0; it < n; ++it) {
-				const int s = it % TK_S;
-				if (*s_abort || !mbar_wait_bounded(bar_full + 8 * s, (it / TK_S) & 1, TD_SPIN)) { fail(); break; }
-				tc_fence_after();
-				const uint32_t a = smem_u32(smem + (size_t)s * TK_STAGE), w = a + TD_A_BYTES;
+	if (m >= p.M) return;
+	float v[16] = {};
+	for (int r = 0; r < p.parts; ++r) {
+		const float4 *f = reinterpret_cast<const float4 *>(p.ws + ((size_t)r * p.M + m) * n16 + n);
 #pragma unroll
-				for (int k = 0; k < TD_BK / 16; ++k) umma_f16(tmem, smem_desc_sw128(a + k * 32), smem_desc_sw128(w + k * 32), IDESC, (it > 0 || k > 0) ? 1u : 0u);
-				umma_commit(bar_empty + 8 * s);
-			}
-			umma_commit(bar_acc);
-		}
-		__syncwarp();
-	}
-	// every warp waits for the CTA's own products; then the ring may be overwritten, here and (behind the barrier) by the others
-	const bool ok = __all_sync(0xffffffffu, mbar_wait_bounded(bar_acc, 0, TD_SPIN)) && !*s_abort;
-	if (!ok) fail();
-	tc_fence_after();
-	__syncwarp();
-	cluster_arrive();
-	cluster_wait();
-	const int cols = TK_BN / parts, ld = cols + 4;                   // columns per rank; padded rows
-	if (warp >= 2) {
-		const int q = warp & 3, half = (warp - 2) >> 2, row = q * 32 + lane;
-		const uint32_t src = smem_u32(smem) + (uint32_t)(rank * TD_BM + row) * ld * 4;
-#pragma unroll 1
-		for (int c = half * (TK_BN / 2); c < (half + 1) * (TK_BN / 2); c += 16) {
-			float v[16];
-			tmem_ld16(tmem + ((uint32_t)(q * 32) << 16) + c, v);
-			tmem_ld_wait();
-#pragma unroll
-			for (int i = 0; i < 16; ++i) asm volatile("" : "+f"(v[i]));
-			const int to = c / cols;
-			const uint32_t dst = cluster_map(src + (uint32_t)(c - to * cols) * 4, (uint32_t)to);
-#pragma unroll
-			for (int i = 0; i < 4; ++i) cluster_store4(dst + 16 * i, v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
+		for (int k = 0; k < 4; ++k) {
+			const float4 x = __ldcg(f + k);
+			v[4 * k] += x.x;
+			v[4 * k + 1] += x.y;
+			v[4 * k + 2] += x.z;
+			v[4 * k + 3] += x.w;
 		}
 	}
-	__syncwarp();
-	cluster_arrive();
-	cluster_wait();
-	if (warp >= 2 && ok) {
-		const int t = tid - 64, row = t & (TD_BM - 1);
-		for (int c = (t >> 7) * 16; c < cols; c += 32) {
-			float v[16] = {};
-			for (int r = 0; r < parts; ++r) {
-				const float4 *f = reinterpret_cast<const float4 *>(reinterpret_cast<const float *>(smem) + (size_t)(r * TD_BM + row) * ld + c);
-#pragma unroll
-				for (int i = 0; i < 4; ++i) {
-					const float4 x = f[i];
-					v[4 * i] += x.x;
-					v[4 * i + 1] += x.y;
-					v[4 * i + 2] += x.z;
-					v[4 * i + 3] += x.w;
-				}
-			}
-			const int col = n0 + rank * cols + c;
-			if (m0 + row < p.M && col < p.N) epi_16<bf16>(p.e, m0 + row, col, v);
-		}
-	}
-	tc_fence_before();
-	__syncthreads();
-	if (warp == 1) tmem_dealloc(tmem, TK_BN);
+	epi_16<bf16>(p.e, m, n, v);
 }
 
-int launch_cluster(const CUtensorMap &tmx, const DenseArgs &a, int parts, cudaStream_t stream) {
-	alignas(64) CUtensorMap tmw;
-	if (int rc = dense_tensor_map(a.w, a.N, a.K, a.ldw, TK_BN, TD_BK, &tmw)) return rc;
-	const int mt = (a.M + TD_BM - 1) / TD_BM, nt = (a.N + TK_BN - 1) / TK_BN;
-	return dn_launch_as(parts, -1, dense_tc_cluster_kernel, dim3(mt * nt * parts), dim3(TD_THREADS), TK_SMEM, stream, tmx, tmw, a, mt, parts);
-}
-
-template <int BN>
+template <int BN, bool SPLIT = false>
 int launch(const CUtensorMap &tmx, const DenseArgs &a, cudaStream_t stream) {
 	alignas(64) CUtensorMap tmw;
 	if (int rc = dense_tensor_map(a.w, a.N, a.K, a.ldw, BN, TD_BK, &tmw)) return rc;
 	const int mt = (a.M + TD_BM - 1) / TD_BM, nt = (a.N + BN - 1) / BN;
-	return dn_launch(dense_tc_kernel<BN>, dim3(std::min(mt * nt, dn_sm_count())), dim3(TD_THREADS), TdShape<BN>::SMEM, stream, tmx, tmw, a, mt, nt);
+	return dn_launch(dense_tc_kernel<BN, SPLIT>, dim3(std::min(mt * nt * (SPLIT ? a.parts : 1), dn_sm_count())), dim3(TD_THREADS), TdShape<BN>::SMEM, stream, tmx, tmw, a, mt, nt);
 }
 
 }   // namespace
@@ -321,17 +224,24 @@ int dense_tensor_map(const void *base, long long rows, long long cols, long long
 	return GPTQ_OK;
 }
 
+// An MMA with its first operand in shared memory takes as long for 32 columns as for 256, so a narrow output wants wide tiles and a
+// split K: parts per tile, 1 where the plain kernel is better.
+int dense_tc_parts(int M, int K, int N) {
+	const int wide = (M + TD_BM - 1) / TD_BM * ((N + 255) / 256), most = std::min(dn_sm_count() / std::max(1, wide), K / (16 * TD_BK));
+	return N <= 512 && most >= 2 ? std::min(most, 8) : 1;
+}
+
 int dense_tc_launch(const DenseArgs &a, cudaStream_t stream) {
 	alignas(64) CUtensorMap tmx;
 	if (int rc = dense_tensor_map(a.x, a.M, a.K, a.ldx, TD_BM, TD_BK, &tmx)) return rc;
 	// column tile: whole waves of tiles, each costing its columns plus a fixed part (smaller tiles feed the tensor cores worse)
 	const int sms = dn_sm_count(), mt = (a.M + TD_BM - 1) / TD_BM;
-	// an output of few wide tiles and a long K: clusters that share K read the rows once instead of once per narrow tile
-	const int wide = mt * ((a.N + TK_BN - 1) / TK_BN);
-	if (a.N <= 2 * TK_BN && a.K >= 1024 && wide * 2 <= sms) {
-		int parts = 8;
-		while (wide * parts > sms) parts >>= 1;
-		return launch_cluster(tmx, a, parts, stream);
+	if (a.ws && dense_tc_parts(a.M, a.K, a.N) > 1) {
+		DenseArgs d = a;
+		d.parts = dense_tc_parts(a.M, a.K, a.N);
+		if (int rc = launch<256, true>(tmx, d, stream)) return rc;
+		const int n16 = (a.N + 15) / 16 * 16;
+		return dn_launch(dense_finish_kernel, dim3((unsigned)(((long long)a.M * (n16 / 16) + DN_THREADS - 1) / DN_THREADS)), dim3(DN_THREADS), 0, stream, d, n16);
 	}
 	const int bns[4] = {256, 128, 64, 32};
 	int pick = 0;

@@ -97,9 +97,13 @@ def matmul(x, w: torch.Tensor, epi: '_dense.Epilogue', control: torch.Tensor, ro
 	require_cuda(w, control, *([] if x is None else [x]))
 	assert w.stride(1) == 1 and (x is None or x.stride(1) == 1 and x.dtype == w.dtype)
 	N, K = w.shape
-	rc = _dense.lib().dense_matmul(ptr(x), 0 if x is None else x.stride(0), ptr(w), w.stride(0), x.shape[0] if x is not None else M, K, N, _dense.DTYPE_CODE[w.dtype],
-								   None if rows is None else ctypes.byref(rows), ctypes.byref(epi), _dense.status_ptr(control), stream_ptr(w.device))
-	_dense.check(rc, 'dense_matmul')
+	rows_n = x.shape[0] if x is not None else M
+	lib, code = _dense.lib(), _dense.DTYPE_CODE[w.dtype]
+	need = lib.dense_matmul_scratch(rows_n, K, N, code)
+	scratch = torch.empty(need, dtype=torch.float32, device=w.device) if need else None
+	rc = lib.dense_matmul(ptr(x), 0 if x is None else x.stride(0), ptr(w), w.stride(0), rows_n, K, N, code, None if rows is None else ctypes.byref(rows),
+						  ctypes.byref(epi), ptr(scratch), _dense.status_ptr(control), stream_ptr(w.device))
+	_dense.check(rc, 'dense_matmul', 2 if need else 1)
 
 
 def project_stream(stream: Stream, w: torch.Tensor, epi: '_dense.Epilogue', control: torch.Tensor, keep: bool = True, final=None) -> Optional[torch.Tensor]:

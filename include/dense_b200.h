@@ -194,7 +194,10 @@ int dense_last_cuda_error(void);
 /* y = epilogue(rows x W^T).  With `rows` the kernel prepares its input rows itself (few rows only, see dense_decode_rows_ok),
  * else x is [M, ldx].  w is [N, ldw].  Chooses the decode kernel, the tensor-core kernel or the fp32 kernel by shape. */
 int dense_matmul(const void *x, int64_t ldx, const void *w, int64_t ldw, int M, int K, int N, int dtype, const dense_rows_t *rows, const dense_epilogue_t *epi,
-				 int *status, void *stream);
+				 float *scratch, int *status, void *stream);
+/* fp32 values of scratch with which dense_matmul splits the K range of a narrow output (two kernels); 0: it would not.  scratch may be
+ * NULL. */
+int64_t dense_matmul_scratch(int M, int K, int N, int dtype);
 int dense_decode_rows_ok(int M, int K, int dtype);      /* the decode kernel (and row preparation inside it) covers M rows of K */
 int dense_prepare_rows(const dense_rows_t *rows, int M, void *h, int64_t ldh, int dtype, void *stream);
 

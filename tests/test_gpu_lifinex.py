@@ -99,10 +99,11 @@ def test_norm_of_equal_parts(control, dtype, M, n, parts):
 
 
 @pytest.mark.parametrize('dtype', [F32, B16])
-@pytest.mark.parametrize('M', [1, 2, 3, 8, 40, 200])
-def test_gated_mlp_and_token_side(control, dtype, M):
+@pytest.mark.parametrize('M,width', [(1, 90), (2, 90), (3, 90), (8, 90), (40, 90), (200, 90), (1, 4200), (2, 6200), (5, 4200), (140, 4200)])
+def test_gated_mlp_and_token_side(control, dtype, M, width):
+	"""Also rows so long that the narrow projections share them over several CTAs."""
 	from gptq_triton_b200.dense import DenseMLP, RMSNorm, Stream, TokenSide, padded, pad_to
-	width, ff, dim, V, L, eps = 90, 77, 21, 31, 3, 1e-4
+	ff, dim, V, L, eps = 77, 21, 31, 3, 1e-4
 	g, u, d = (rnd(*s, seed=i, dtype=B16) * 2 * s[1] ** -0.5 for i, s in enumerate([(ff, width), (ff, width), (width, ff)]))
 	x, y = rnd(M, width, seed=8), rnd(M, width, seed=9)
 	w = 0.2 * rnd(width, seed=5)

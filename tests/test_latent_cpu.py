@@ -50,11 +50,11 @@ def test_struct_layouts_match_the_header(tmp_path):
 def test_arguments_are_refused_on_the_host(lib):
 	e, r, a = _dense.Epilogue(), _dense.Rows(), _dense.Latent()
 	p = ctypes.c_void_p(0x1000)
-	assert lib.dense_matmul(None, 64, p, 64, 1, 64, 16, 0, None, ctypes.byref(e), p, None) == -1          # neither rows nor x
-	assert lib.dense_matmul(p, 64, p, 64, 1, 60, 16, 0, None, ctypes.byref(e), p, None) == -2             # K not a multiple of 16
-	assert lib.dense_matmul(p, 64, ctypes.c_void_p(0x1004), 64, 1, 64, 16, 0, None, ctypes.byref(e), p, None) == -4
-	assert lib.dense_matmul(p, 64, p, 64, 1, 64, 16, 0, None, ctypes.byref(e), p, None) == -1             # no output
-	assert lib.dense_matmul(p, 64, p, 64, 0, 64, 16, 0, None, ctypes.byref(e), p, None) == 0              # no rows: nothing to do
+	assert lib.dense_matmul(None, 64, p, 64, 1, 64, 16, 0, None, ctypes.byref(e), None, p, None) == -1          # neither rows nor x
+	assert lib.dense_matmul(p, 64, p, 64, 1, 60, 16, 0, None, ctypes.byref(e), None, p, None) == -2             # K not a multiple of 16
+	assert lib.dense_matmul(p, 64, ctypes.c_void_p(0x1004), 64, 1, 64, 16, 0, None, ctypes.byref(e), None, p, None) == -4
+	assert lib.dense_matmul(p, 64, p, 64, 1, 64, 16, 0, None, ctypes.byref(e), None, p, None) == -1             # no output
+	assert lib.dense_matmul(p, 64, p, 64, 0, 64, 16, 0, None, ctypes.byref(e), None, p, None) == 0              # no rows: nothing to do
 	assert lib.dense_prepare_rows(ctypes.byref(r), 1, p, 64, 0, None) == -1
 	assert lib.dense_latent_absorb(ctypes.byref(a), 0, None) == -1
 	assert lib.dense_latent_prefill(None, None) == -1

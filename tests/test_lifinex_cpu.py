@@ -162,9 +162,9 @@ def test_arguments_are_refused_on_the_host(lib):
 	e = _dense.Epilogue()
 	e.mode, e.out, e.ldo, e.tab, e.tab_token, e.tab_rows, e.tab_ld, e.tab_col = _dense.EPI_TABLE, p, 16, p, p, 4, 32, 24
 	v = ctypes.c_void_p(p)
-	assert lib.dense_matmul(v, 64, v, 64, 1, 64, 16, 0, None, ctypes.byref(e), v, None) == -4          # columns beyond the table's row
+	assert lib.dense_matmul(v, 64, v, 64, 1, 64, 16, 0, None, ctypes.byref(e), None, v, None) == -4          # columns beyond the table's row
 	e.mode, e.act = _dense.EPI_F32, 7
-	assert lib.dense_matmul(v, 64, v, 64, 1, 64, 16, 0, None, ctypes.byref(e), v, None) == -1
+	assert lib.dense_matmul(v, 64, v, 64, 1, 64, 16, 0, None, ctypes.byref(e), None, v, None) == -1
 	assert lib.dense_gqa_splits(1, 32, 8, 2, 4096, 0) > 1 and lib.dense_gqa_splits(4096, 32, 8, 2, 4096, 0) == 1
 	with pytest.raises(ValueError):
 		RMSNorm(torch.ones(12), parts=5)
