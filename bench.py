@@ -1203,7 +1203,7 @@ def lifinex_config(G, runs, hid, inter, vocab=32000, max_positions=4096):
 	"""`runs` layer runs, attention and state-space layers in turn (runs = 8: six layers, two of them run twice)."""
 	ff = {'kind': 'dense', 'ff': inter}
 	H = hid // 128
-	att = {'type': 'attention', 'mlp': ff, 'mixer': {'heads': H, 'kv_heads': H // 4, 'dim': 64, 'vdim': 128, 'scale': 0.125, 'softcap': 30.0, 'diff': 0.3}}
+	att = {'type': 'attention', 'mlp': ff, 'mixer': {'heads': H, 'kv_heads': H // 4, 'dim': 64, 'vdim': 128, 'scale': 0.125, 'softcap': 25.0, 'diff': 0.4}}
 	ssm = {'type': 'mamba2', 'mlp': ff, 'mixer': {'heads': hid // 32, 'vdim': 64, 'state': 128, 'groups': 8, 'conv': 4, 'norm_groups': 8}}
 	layers, loop = {8: ([att, ssm] * 3, (2, 4, 2)), 4: ([ssm, att, ssm], (1, 2, 2)), 2: ([att, ssm], (0, 1, 1))}[runs]
 	return G.LifinexConfig.from_dict({'vocab': vocab, 'width': hid, 'layers': layers, 'norm': {'eps': 1e-6}, 'max_positions': max_positions, 'token_side': {'dim': 256},

@@ -275,7 +275,7 @@ def build_ssm(spec, W, dtype):
 	return StateSpaceMixer(spec, W['in'].to(dtype), *(W[k] for k in ('conv', 'conv.b', 'dt_bias', 'A_log', 'D', 'norm')), W['o'].to(dtype)).cuda()
 
 
-SSM_SHAPES = [(2, 16, 16, 1, 1, 1), (6, 20, 24, 3, 4, 5), (5, 7, 40, 1, 2, 7), (4, 64, 128, 2, 4, 4), (3, 33, 200, 3, 3, 1), (8, 48, 32, 2, 3, 2), (2, 80, 256, 1, 7, 2), (1, 5, 3, 1, 16, 1),
+SSM_SHAPES = [(2, 16, 16, 1, 1, 1), (6, 20, 24, 3, 4, 5), (5, 7, 40, 1, 2, 7), (4, 64, 128, 2, 4, 4), (3, 33, 200, 3, 3, 1), (6, 48, 32, 3, 3, 4), (2, 80, 256, 1, 7, 2), (1, 5, 3, 1, 16, 1),
 			  (4, 128, 64, 4, 4, 1), (16, 32, 64, 2, 4, 16)]
 
 
